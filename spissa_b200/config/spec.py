@@ -50,11 +50,14 @@ class ScheduleEntry:
     entry of the same step has written. ``adds_embedding``: the embedding's output of
     the step's tokens is added to the residual stream right before this run (how a group
     of layers that runs several times takes its input in again at every pass but the first).
+    ``adds_row``: this row of ``ModelSpec.pass_rows`` is added to the stream right before this
+    run (a learned vector per pass).
     """
     layer: int
     cache: int
     writes_cache: bool = True
     adds_embedding: bool = False
+    adds_row: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -69,6 +72,7 @@ class ModelSpec:
     head: PartSpec
     max_position: int
     extras: dict = field(default_factory=dict)
+    pass_rows: Optional[PartSpec] = None      # a table of learned rows that schedule entries add to the stream
     streams: int = 1          # copies of the residual stream side by side in a token's row (hyper-connections): the
     #                           embedding's output fills them all, the layers' blocks mix them, the final norm reads their sum
 
@@ -79,6 +83,8 @@ class ModelSpec:
             raise ValueError("a model needs a non-empty layer schedule")
         if self.streams < 1 or (self.streams > 1 and any(e.adds_embedding for e in self.schedule)):
             raise ValueError("several residual streams and layers that take the embedding in again do not go together")
+        if any(e.adds_row is not None for e in self.schedule) and (self.pass_rows is None or self.streams > 1):
+            raise ValueError("schedule entries that add a row need a table of rows and one residual stream")
         writers = {}
         for pos, e in enumerate(self.schedule):
             if not (0 <= e.layer < len(self.layers)):

@@ -58,6 +58,7 @@ MODULES = {
     "hybrid": "hybrid_kernels.cu",
     "latent": "latent_kernels.cu",
     "sandwich": "sandwich_kernels.cu",
+    "rglru": "rglru_kernels.cu",
 }
 
 

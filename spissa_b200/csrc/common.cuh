@@ -48,6 +48,23 @@ __device__ __forceinline__ void sp_st_dt(void* p, int dt, size_t i, float v) {
     else ((__nv_bfloat16*)p)[i] = __float2bfloat16_rn(v);
 }
 
+// ---------------------------------------------------------------- activations of gated units
+// What a product's epilogue applies: silu(gate)·up, gelu(gate)·up, or (plain rows) the square of relu.
+enum { SP_ACT_SILU = 0, SP_ACT_GELU = 1, SP_ACT_RELU2 = 2 };
+
+// The tanh form of gelu, ½ z (1 + tanh(a)) with a = √(2/π)(z + 0.044715 z³), written with the logistic function:
+// ½ (1 + tanh(a)) = 1 / (1 + e^{−2a}).
+__device__ __forceinline__ float sp_gelu_tanh(float z) {
+    return z / (1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+}
+__device__ __forceinline__ float sp_gated(float gate, float up, int act) {
+    return (act == SP_ACT_GELU ? sp_gelu_tanh(gate) : gate / (1.0f + expf(-gate))) * up;
+}
+__device__ __forceinline__ float sp_relu2(float z) {
+    const float r = fmaxf(z, 0.0f);
+    return r * r;
+}
+
 // ---------------------------------------------------------------- reductions
 __device__ __forceinline__ float sp_warp_sum(float v) {
 #pragma unroll

@@ -50,17 +50,18 @@ SP_API int sp_embed_gather(const void* table, int table_dt, const int* ids, floa
 // ============================================================== rms norm
 // One block per output row. ``rows`` (optional) gathers input rows: out row r is the
 // norm of x row rows[r]. Statistics and the product are 32-bit; the result is rounded
-// once, on the store.
-__global__ void rmsnorm_kernel(const float* __restrict__ x, const void* __restrict__ w, int w_dt,
+// once, on the store. ``add`` (optional, [H], without ``rows``): added to every row of x first, in place.
+__global__ void rmsnorm_kernel(float* x, const void* __restrict__ w, int w_dt,
                                void* __restrict__ out, int out_dt, const int* __restrict__ rows,
-                               int n_rows, int H, float eps) {
+                               int n_rows, int H, float eps, const float* __restrict__ add) {
     __shared__ float scratch[32];
     const int r = blockIdx.x;
     if (r >= n_rows) return;
     const size_t src = (size_t)(rows ? rows[r] : r) * H;
     float ss = 0.0f;
     for (int c = threadIdx.x; c < H; c += blockDim.x) {
-        const float v = x[src + c];
+        float v = x[src + c];
+        if (add) x[src + c] = v = v + add[c];               // this thread reads the entry back below
         ss = fmaf(v, v, ss);
     }
     ss = sp_block_sum(ss, scratch);
@@ -73,12 +74,12 @@ __global__ void rmsnorm_kernel(const float* __restrict__ x, const void* __restri
 
 // The same with each row held in registers: one read of x. For H a multiple of 4 up to 4096.
 __global__ void __launch_bounds__(256)
-rmsnorm_row_kernel(const float* __restrict__ x, const void* __restrict__ w, int w_dt, void* __restrict__ out,
-                   int out_dt, const int* __restrict__ rows, int n_rows, int H, float eps) {
+rmsnorm_row_kernel(float* x, const void* __restrict__ w, int w_dt, void* __restrict__ out,
+                   int out_dt, const int* __restrict__ rows, int n_rows, int H, float eps, const float* __restrict__ add) {
     __shared__ float scratch[32];
     const int r = blockIdx.x;
     if (r >= n_rows) return;
-    const float4* src = (const float4*)(x + (size_t)(rows ? rows[r] : r) * H);
+    float4* src = (float4*)(x + (size_t)(rows ? rows[r] : r) * H);
     const int n4 = H >> 2;
     float4 v[4];
     float ss = 0.0f;
@@ -86,6 +87,11 @@ rmsnorm_row_kernel(const float* __restrict__ x, const void* __restrict__ w, int 
     for (int i = 0; i < 4; ++i) {
         const int c = threadIdx.x + i * 256;
         v[i] = c < n4 ? src[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+        if (add && c < n4) {
+            const float4 e = ((const float4*)add)[c];
+            v[i].x += e.x; v[i].y += e.y; v[i].z += e.z; v[i].w += e.w;
+            src[c] = v[i];
+        }
         ss = fmaf(v[i].x, v[i].x, ss); ss = fmaf(v[i].y, v[i].y, ss);
         ss = fmaf(v[i].z, v[i].z, ss); ss = fmaf(v[i].w, v[i].w, ss);
     }
@@ -116,17 +122,25 @@ rmsnorm_row_kernel(const float* __restrict__ x, const void* __restrict__ w, int 
 // in flight at once and the row sum needs no shared memory. For H = 128·NV.
 template <int NV, bool WBF16>
 __global__ void __launch_bounds__(256)
-rmsnorm_warp_kernel(const float* __restrict__ x, const void* __restrict__ w, int w_dt, void* __restrict__ out,
-                    int out_dt, const int* __restrict__ rows, int n_rows, int H, float eps) {
+rmsnorm_warp_kernel(float* x, const void* __restrict__ w, int w_dt, void* __restrict__ out,
+                    int out_dt, const int* __restrict__ rows, int n_rows, int H, float eps, const float* __restrict__ add) {
     sp_allow_dependents();
     sp_wait_for_predecessor();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int r = blockIdx.x * 8 + warp;
     if (r >= n_rows) return;
-    const float4* src = (const float4*)(x + (size_t)(rows ? rows[r] : r) * H);
+    float4* src = (float4*)(x + (size_t)(rows ? rows[r] : r) * H);
     float4 v[NV];
 #pragma unroll
     for (int i = 0; i < NV; ++i) v[i] = src[lane + 32 * i];
+    if (add) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const float4 e = ((const float4*)add)[lane + 32 * i];
+            v[i].x += e.x; v[i].y += e.y; v[i].z += e.z; v[i].w += e.w;
+            src[lane + 32 * i] = v[i];
+        }
+    }
     // bfloat16 weights are asked for before the row's sum is known: one trip to memory instead of two in a row
     // (float32 weights would not fit the registers next to the row)
     uint2 wb[WBF16 ? NV : 1];
@@ -167,30 +181,42 @@ rmsnorm_warp_kernel(const float* __restrict__ x, const void* __restrict__ w, int
     }
 }
 
-SP_API int sp_rmsnorm(const float* x, const void* w, int w_dt, void* out, int out_dt, const int* rows,
-                      int n_rows, int H, float eps, cudaStream_t stream) {
+static int rmsnorm_any(float* x, const void* w, int w_dt, void* out, int out_dt, const int* rows, int n_rows, int H,
+                       float eps, const float* add, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
+    if (add && rows) SP_FAIL("rmsnorm: a row is added to every row of the stream, not to gathered ones");
     if ((w_dt | out_dt) & ~1) SP_FAIL("rmsnorm: unsupported dtype code");
     // fixed block sizes: the order of the row sum must not depend on the batch
-    const bool aligned = ((((uintptr_t)x | (uintptr_t)out | (uintptr_t)w) & 15) == 0);
+    const bool aligned = ((((uintptr_t)x | (uintptr_t)out | (uintptr_t)w | (uintptr_t)add) & 15) == 0);
 #define SP_NORM_WARP(NV)                                                                                        \
     if (aligned && H == 128 * NV) {                                                                             \
         if (w_dt == SP_DT_BF16)                                                                                 \
-            sp_launch_dependent(rmsnorm_warp_kernel<NV, true>, dim3((n_rows + 7) / 8), dim3(256), 0, stream, x, w, w_dt, out, out_dt, rows, n_rows, H, eps); \
+            sp_launch_dependent(rmsnorm_warp_kernel<NV, true>, dim3((n_rows + 7) / 8), dim3(256), 0, stream, x, w, w_dt, out, out_dt, rows, n_rows, H, eps, add); \
         else                                                                                                    \
-            sp_launch_dependent(rmsnorm_warp_kernel<NV, false>, dim3((n_rows + 7) / 8), dim3(256), 0, stream, x, w, w_dt, out, out_dt, rows, n_rows, H, eps); \
+            sp_launch_dependent(rmsnorm_warp_kernel<NV, false>, dim3((n_rows + 7) / 8), dim3(256), 0, stream, x, w, w_dt, out, out_dt, rows, n_rows, H, eps, add); \
         SP_CHECK_LAUNCH("rmsnorm");                                                                             \
         return 0;                                                                                               \
     }
     SP_NORM_WARP(4) SP_NORM_WARP(8) SP_NORM_WARP(16) SP_NORM_WARP(24) SP_NORM_WARP(32)
 #undef SP_NORM_WARP
-    if ((H & 3) == 0 && H <= 4096 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0)
+    if ((H & 3) == 0 && H <= 4096 && (((uintptr_t)x | (uintptr_t)out | (uintptr_t)add) & 15) == 0)
         SP_CHECK_CALL("rmsnorm", sp_launch_cluster(rmsnorm_row_kernel, dim3(n_rows), dim3(256), 0, stream, 1, x, w, w_dt, out,
-                                              out_dt, rows, n_rows, H, eps));
+                                              out_dt, rows, n_rows, H, eps, add));
     else
         SP_CHECK_CALL("rmsnorm", sp_launch_cluster(rmsnorm_kernel, dim3(n_rows), dim3(256), 0, stream, 1, x, w, w_dt, out,
-                                              out_dt, rows, n_rows, H, eps));
+                                              out_dt, rows, n_rows, H, eps, add));
     return 0;
+}
+
+SP_API int sp_rmsnorm(const float* x, const void* w, int w_dt, void* out, int out_dt, const int* rows,
+                      int n_rows, int H, float eps, cudaStream_t stream) {
+    return rmsnorm_any(const_cast<float*>(x), w, w_dt, out, out_dt, rows, n_rows, H, eps, nullptr, stream);
+}
+
+// x[r, :] += add, then the norm of the new rows, in one pass
+SP_API int sp_rmsnorm_add_row(float* x, const float* add, const void* w, int w_dt, void* out, int out_dt, int n_rows, int H,
+                              float eps, cudaStream_t stream) {
+    return rmsnorm_any(x, w, w_dt, out, out_dt, nullptr, n_rows, H, eps, add, stream);
 }
 
 // ============================================================== matrix product
@@ -763,29 +789,34 @@ SP_API int sp_attention_generic(const void* q, int q_dt, const void* kpool, cons
     return 0;
 }
 
-// ============================================================== silu(gate) * up
-// gu row = [gate(0..I) | up(0..I)]; out row = silu(gate) ⊙ up, silu(z) = z / (1 + e^-z).
+// ============================================================== act(gate) * up
+// gu row = [gate(0..I) | up(0..I)]; out row = act(gate) ⊙ up · mult (SP_ACT_SILU, SP_ACT_GELU).
 template <typename T>
-__global__ void silu_mul_kernel(const T* __restrict__ gu, T* __restrict__ out, size_t rows, int I) {
+__global__ void gated_mul_kernel(const T* __restrict__ gu, T* __restrict__ out, size_t rows, int I, int act, float mult) {
     const size_t n = rows * (size_t)I;
     for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < n; e += (size_t)gridDim.x * blockDim.x) {
         const size_t r = e / I;
         const int c = (int)(e % I);
         const float g = sp_ld(gu, r * 2 * I + c);
         const float u = sp_ld(gu, r * 2 * I + I + c);
-        sp_st(out, e, (g / (1.0f + expf(-g))) * u);
+        sp_st(out, e, sp_gated(g, u, act) * mult);
     }
 }
 
-SP_API int sp_silu_mul(const void* gu, void* out, int dt, int rows, int I, cudaStream_t stream) {
+SP_API int sp_gated_mul(const void* gu, void* out, int dt, int rows, int I, int act, float mult, cudaStream_t stream) {
     if (rows <= 0 || I <= 0) return 0;
+    if (act != SP_ACT_SILU && act != SP_ACT_GELU) SP_FAIL("gated_mul: activation code %d is not built", act);
     const size_t n = (size_t)rows * I;
     const int blocks = (int)((n + 255) / 256 > 148 * 16 ? 148 * 16 : (n + 255) / 256);
-    if (dt == SP_DT_F32) silu_mul_kernel<float><<<blocks, 256, 0, stream>>>((const float*)gu, (float*)out, rows, I);
-    else if (dt == SP_DT_BF16) silu_mul_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>((const __nv_bfloat16*)gu, (__nv_bfloat16*)out, rows, I);
-    else SP_FAIL("silu_mul: unsupported dtype code %d", dt);
-    SP_CHECK_LAUNCH("silu_mul");
+    if (dt == SP_DT_F32) gated_mul_kernel<float><<<blocks, 256, 0, stream>>>((const float*)gu, (float*)out, rows, I, act, mult);
+    else if (dt == SP_DT_BF16) gated_mul_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>((const __nv_bfloat16*)gu, (__nv_bfloat16*)out, rows, I, act, mult);
+    else SP_FAIL("gated_mul: unsupported dtype code %d", dt);
+    SP_CHECK_LAUNCH("gated_mul");
     return 0;
+}
+
+SP_API int sp_silu_mul(const void* gu, void* out, int dt, int rows, int I, cudaStream_t stream) {
+    return sp_gated_mul(gu, out, dt, rows, I, SP_ACT_SILU, 1.0f, stream);
 }
 
 // ============================================================== cap of the logits, a gate per row
@@ -849,6 +880,56 @@ SP_API int sp_scale_rows_sigmoid(void* x, int dt, const float* z, int rows, int 
     return 0;
 }
 
+// x[t, c] ← x[t, c] · sigmoid(z[t·ldz + c]) · mult: a gate with a number of its own for every element
+template <typename T>
+__global__ void gate_elements_kernel(T* __restrict__ x, const float* __restrict__ z, size_t rows, int C, int ldz, float mult) {
+    const size_t n = rows * (size_t)C;
+    for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < n; e += (size_t)gridDim.x * blockDim.x) {
+        const float g = mult / (1.0f + expf(-z[e / C * ldz + e % C]));
+        sp_st(x, e, sp_ld(x, e) * g);
+    }
+}
+
+// the same, eight bfloat16 at a time (C a multiple of 8, the gates' rows on 16-byte boundaries)
+__global__ void __launch_bounds__(256)
+gate_elements_vec_kernel(uint4* __restrict__ x, const float* __restrict__ z, size_t groups, int groups_per_row, int ldz, float mult) {
+    sp_allow_dependents();
+    sp_wait_for_predecessor();
+    for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < groups; e += (size_t)gridDim.x * blockDim.x) {
+        const size_t t = e / groups_per_row;
+        const float4* zr = (const float4*)(z + t * ldz + (e - t * groups_per_row) * 8);
+        const float4 z0 = zr[0], z1 = zr[1];
+        uint4 w = x[e];
+        const float g[8] = {z0.x, z0.y, z0.z, z0.w, z1.x, z1.y, z1.z, z1.w};
+        __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&w);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float2 f = __bfloat1622float2(p[i]);
+            p[i] = __floats2bfloat162_rn(f.x * (mult / (1.0f + expf(-g[2 * i]))), f.y * (mult / (1.0f + expf(-g[2 * i + 1]))));
+        }
+        x[e] = w;
+    }
+}
+
+SP_API int sp_gate_elements(void* x, int dt, const float* z, int rows, int C, int ldz, float mult, cudaStream_t stream) {
+    if (rows <= 0 || C <= 0) return 0;
+    if (ldz < C) SP_FAIL("gate_elements: rows of %d gates for %d columns", ldz, C);
+    const size_t n = (size_t)rows * C;
+    if (dt == SP_DT_BF16 && C % 8 == 0 && ldz % 4 == 0 && (((uintptr_t)x | (uintptr_t)z) & 15) == 0) {
+        const size_t groups = n / 8;
+        const int blocks = (int)((groups + 255) / 256 > 148 * 16 ? 148 * 16 : (groups + 255) / 256);
+        SP_CHECK_CALL("gate_elements", sp_launch_dependent(gate_elements_vec_kernel, dim3(blocks), dim3(256), 0, stream, (uint4*)x, z,
+                                                           groups, C / 8, ldz, mult));
+        return 0;
+    }
+    const int blocks = (int)((n + 255) / 256 > 148 * 16 ? 148 * 16 : (n + 255) / 256);
+    if (dt == SP_DT_F32) gate_elements_kernel<float><<<blocks, 256, 0, stream>>>((float*)x, z, rows, C, ldz, mult);
+    else if (dt == SP_DT_BF16) gate_elements_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>((__nv_bfloat16*)x, z, rows, C, ldz, mult);
+    else SP_FAIL("gate_elements: unsupported dtype code %d", dt);
+    SP_CHECK_LAUNCH("gate_elements");
+    return 0;
+}
+
 // ============================================================== residual add
 __global__ void add_inplace_kernel(float* __restrict__ dst, const void* __restrict__ src, int src_dt, size_t n) {
     for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < n; e += (size_t)gridDim.x * blockDim.x)
@@ -861,6 +942,19 @@ SP_API int sp_add_inplace(float* dst, const void* src, int src_dt, long long n, 
     const int blocks = (int)(want > 148 * 16 ? 148 * 16 : want);
     add_inplace_kernel<<<blocks, 256, 0, stream>>>(dst, src, src_dt, (size_t)n);
     SP_CHECK_LAUNCH("add_inplace");
+    return 0;
+}
+
+// x[r, :] += row, 32-bit
+__global__ void add_row_kernel(float* __restrict__ x, const float* __restrict__ row, size_t n, int W) {
+    for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < n; e += (size_t)gridDim.x * blockDim.x) x[e] += row[e % W];
+}
+
+SP_API int sp_add_row(float* x, const float* row, int T, int W, cudaStream_t stream) {
+    if (T <= 0 || W <= 0) return 0;
+    const size_t n = (size_t)T * W, want = (n + 255) / 256;
+    add_row_kernel<<<(unsigned)(want > 148 * 16 ? 148 * 16 : want), 256, 0, stream>>>(x, row, n, W);
+    SP_CHECK_LAUNCH("add_row");
     return 0;
 }
 

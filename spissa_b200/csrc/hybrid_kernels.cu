@@ -1012,7 +1012,7 @@ SP_API int sp_gla(const float* proj, int ld, float* state, int n_slots, const vo
 __global__ void gelu_tanh_kernel(const void* __restrict__ z, int z_dt, void* __restrict__ out, int out_dt, size_t n) {
     for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < n; e += (size_t)gridDim.x * blockDim.x) {
         const float v = sp_ld_dt(z, z_dt, e);
-        sp_st_dt(out, out_dt, e, 0.5f * v * (1.0f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v))));
+        sp_st_dt(out, out_dt, e, sp_gelu_tanh(v));
     }
 }
 
@@ -1058,7 +1058,8 @@ SP_API int sp_clamped_glu(const void* gu, int gu_dt, void* out, int out_dt, int 
 // the row's E logits; choice c = s + correction (none: s). The weights leave times ``weight_scale``. The experts form ``n_groups`` equal groups of
 // neighbours; a group's score is the sum of its two largest c; only experts of the ``keep`` best groups can be chosen
 // (n_groups ≤ 1: all). The ``top`` largest allowed c are chosen (among equals the lowest index); their weights are
-// their s divided by the sum of those s (+ 1e-20). One warp per token; lane l holds experts l, l+32, ...
+// their s divided by the sum of those s (+ 1e-20), or with ``normalize`` 0 their s as it is. One warp per token; lane l
+// holds experts l, l+32, ...
 #define MS_MAX_E 512
 #define MS_WARPS 4
 __device__ __forceinline__ void ms_take(float& bv, int& bi, float ov, int oi) {
@@ -1068,7 +1069,7 @@ __device__ __forceinline__ void ms_take(float& bv, int& bi, float ov, int oi) {
 __global__ void __launch_bounds__(MS_WARPS * 32)
 moe_select_kernel(const float* __restrict__ z, const void* __restrict__ corr, int corr_dt, int* __restrict__ ids,
                   float* __restrict__ wts, int T, int E, int ldz, int top, int n_groups, int keep, int softmax,
-                  float weight_scale, float* __restrict__ extra) {
+                  float weight_scale, int normalize, float* __restrict__ extra) {
     __shared__ float ch[MS_WARPS][MS_MAX_E];        // choice scores; −inf once chosen or not allowed
     __shared__ float sc[MS_WARPS][MS_MAX_E];
     __shared__ float gs[MS_WARPS][MS_MAX_E];        // group scores
@@ -1147,12 +1148,12 @@ moe_select_kernel(const float* __restrict__ z, const void* __restrict__ corr, in
         __syncwarp();
     }
     __syncwarp();
-    const float den = sum + 1e-20f;
+    const float den = normalize ? sum + 1e-20f : 1.0f;
     for (int k = lane; k < top; k += 32) wts[(size_t)t * top + k] = wts[(size_t)t * top + k] / den * weight_scale;
 }
 
 SP_API int sp_moe_select(const float* z, const void* corr, int corr_dt, int* ids, float* wts, int T, int E, int ldz,
-                         int top, int n_groups, int keep, int softmax, float weight_scale, float* extra,
+                         int top, int n_groups, int keep, int softmax, float weight_scale, int normalize, float* extra,
                          cudaStream_t stream) {
     if (T <= 0) return 0;
     if (E <= 0 || E > MS_MAX_E) SP_FAIL("moe_select: %d experts, this kernel takes up to %d", E, MS_MAX_E);
@@ -1162,7 +1163,7 @@ SP_API int sp_moe_select(const float* z, const void* corr, int corr_dt, int* ids
     if (n_groups > 1 && (keep < 1 || keep > n_groups)) SP_FAIL("moe_select: %d of %d groups cannot be kept", keep, n_groups);
     const int allowed = n_groups > 1 ? keep * (E / n_groups) : E;
     if (top < 1 || top > allowed) SP_FAIL("moe_select: %d experts cannot be chosen among %d allowed", top, allowed);
-    moe_select_kernel<<<(T + MS_WARPS - 1) / MS_WARPS, MS_WARPS * 32, 0, stream>>>(z, corr, corr_dt, ids, wts, T, E, ldz, top, n_groups, keep, softmax, weight_scale, extra);
+    moe_select_kernel<<<(T + MS_WARPS - 1) / MS_WARPS, MS_WARPS * 32, 0, stream>>>(z, corr, corr_dt, ids, wts, T, E, ldz, top, n_groups, keep, softmax, weight_scale, normalize, extra);
     SP_CHECK_LAUNCH("moe_select");
     return 0;
 }
@@ -1170,7 +1171,9 @@ SP_API int sp_moe_select(const float* z, const void* corr, int corr_dt, int* ids
 // ============================================================== the chosen experts' products
 // A pair p = token · top + k names one chosen expert of one token. ``moe_plan`` sorts the pairs by expert (pairs of
 // one expert in ascending order) and cuts every expert's list into tiles of ME_TM rows: (expert, first place in the
-// sorted list, rows); unused entries of the tile table (it is sized for the worst case) say expert −1.
+// sorted list, rows); unused entries of the tile table (it is sized for the worst case) say expert −1. An id of E or
+// more names an identity expert, whose output is the token's input: such a pair is in no list and no product, the
+// combining kernel adds the input times the pair's weight.
 #define ME_TM 32
 __global__ void moe_count_kernel(const int* __restrict__ ids, int n_pairs, int* __restrict__ counts) {
     __shared__ int red[32];
@@ -1284,9 +1287,11 @@ SP_API int sp_moe_plan_tiles(const void* x, const int* ids, int T, int top, int 
     return 0;
 }
 
-// y[t] += Σ_k weight[t·top + k] · rows[pos[t·top + k]] in the order of k
+// y[t] += Σ_k weight[t·top + k] · rows[pos[t·top + k]] in the order of k; with ``ids`` (E experts have products) a pair
+// whose id is E or more adds weight · x[t]
 __global__ void moe_combine_rows_kernel(const float* __restrict__ rows, const int* __restrict__ pos, const float* __restrict__ wts,
-                                        float* __restrict__ y, size_t T, int top, int W) {
+                                        float* __restrict__ y, size_t T, int top, int W, const int* __restrict__ ids, int E,
+                                        const __nv_bfloat16* __restrict__ x) {
     const size_t n = T * (size_t)(W / 4);
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
         const size_t t = i / (W / 4);
@@ -1294,7 +1299,14 @@ __global__ void moe_combine_rows_kernel(const float* __restrict__ rows, const in
         float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         for (int k = 0; k < top; ++k) {
             const float wt = wts[t * top + k];
-            const float4 r = ((const float4*)(rows + (size_t)pos[t * top + k] * W))[c];
+            float4 r;
+            if (ids && ids[t * top + k] >= E) {
+                const uint2 q = ((const uint2*)(x + t * W))[c];
+                const float2 lo = __bfloat1622float2(*(const __nv_bfloat162*)&q.x), hi = __bfloat1622float2(*(const __nv_bfloat162*)&q.y);
+                r = make_float4(lo.x, lo.y, hi.x, hi.y);
+            } else {
+                r = ((const float4*)(rows + (size_t)pos[t * top + k] * W))[c];
+            }
             v.x += r.x * wt; v.y += r.y * wt; v.z += r.z * wt; v.w += r.w * wt;
         }
         float4 o = ((float4*)(y + t * W))[c];
@@ -1304,12 +1316,13 @@ __global__ void moe_combine_rows_kernel(const float* __restrict__ rows, const in
 }
 
 SP_API int sp_moe_combine_rows(const float* rows, const int* pos, const float* wts, float* y, int T, int top, int W,
-                               cudaStream_t stream) {
+                               const int* ids, int E, const void* x, cudaStream_t stream) {
     if (T <= 0) return 0;
-    if (W % 4 || (((uintptr_t)rows | (uintptr_t)y) & 15)) SP_FAIL("moe_combine_rows: rows of %d do not move in 16-byte pieces", W);
+    if (W % 4 || (((uintptr_t)rows | (uintptr_t)y | (uintptr_t)x) & 15)) SP_FAIL("moe_combine_rows: rows of %d do not move in 16-byte pieces", W);
     const size_t n = (size_t)T * (W / 4);
     const size_t want = (n + 255) / 256;
-    moe_combine_rows_kernel<<<(unsigned)(want > 148 * 16 ? 148 * 16 : want), 256, 0, stream>>>(rows, pos, wts, y, (size_t)T, top, W);
+    moe_combine_rows_kernel<<<(unsigned)(want > 148 * 16 ? 148 * 16 : want), 256, 0, stream>>>(rows, pos, wts, y, (size_t)T, top, W, ids, E,
+                                                                                                       (const __nv_bfloat16*)x);
     SP_CHECK_LAUNCH("moe_combine_rows");
     return 0;
 }
@@ -1318,7 +1331,9 @@ SP_API int sp_moe_combine_rows(const float* rows, const int* pos, const float* w
 // 4tx … 4tx+3. Every output adds its products in the order of k, whatever tile it falls into.
 #define ME_BN 64
 #define ME_BK 32
-template <typename TA, typename TW>
+// GLU: an expert's rows are gate and up, the store is the gated activation; else up rows alone, the store is the square
+// of their relu.
+template <typename TA, typename TW, bool GLU>
 __global__ void __launch_bounds__(256)
 moe_up_kernel(const TA* __restrict__ x, const TW* __restrict__ wgu, const int* __restrict__ sorted,
               const int* __restrict__ tiles, TA* __restrict__ act, int top, int W, int F, float limit, float slope) {
@@ -1331,8 +1346,8 @@ moe_up_kernel(const TA* __restrict__ x, const TW* __restrict__ wgu, const int* _
     const int n0 = blockIdx.y * ME_BN;
     if (threadIdx.x < ME_TM) tok[threadIdx.x] = threadIdx.x < rows ? sorted[first + threadIdx.x] / top : -1;
     __syncthreads();
-    const TW* wg = wgu + (size_t)e * 2 * F * W;
-    const TW* wu = wg + (size_t)F * W;
+    const TW* wg = wgu + (size_t)e * (GLU ? 2 : 1) * F * W;
+    const TW* wu = wg + (GLU ? (size_t)F * W : 0);
     const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
     float ag[2][4] = {}, au[2][4] = {};
     for (int k0 = 0; k0 < W; k0 += ME_BK) {
@@ -1348,7 +1363,7 @@ moe_up_kernel(const TA* __restrict__ x, const TW* __restrict__ wgu, const int* _
             for (int u = 0; u < 8; ++u) {
                 const bool ok = in && k0 + k8 + u < W;
                 Bg[k8 + u][n] = ok ? sp_ld(wg, (size_t)(n0 + n) * W + k0 + k8 + u) : 0.0f;
-                Bu[k8 + u][n] = ok ? sp_ld(wu, (size_t)(n0 + n) * W + k0 + k8 + u) : 0.0f;
+                if (GLU) Bu[k8 + u][n] = ok ? sp_ld(wu, (size_t)(n0 + n) * W + k0 + k8 + u) : 0.0f;
             }
         }
         __syncthreads();
@@ -1356,12 +1371,12 @@ moe_up_kernel(const TA* __restrict__ x, const TW* __restrict__ wgu, const int* _
         for (int k = 0; k < ME_BK; ++k) {
             const float a0 = As[k][2 * ty], a1 = As[k][2 * ty + 1];
             const float4 g4 = *(const float4*)&Bg[k][4 * tx];
-            const float4 u4 = *(const float4*)&Bu[k][4 * tx];
+            const float4 u4 = GLU ? *(const float4*)&Bu[k][4 * tx] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
             const float g[4] = {g4.x, g4.y, g4.z, g4.w}, uu[4] = {u4.x, u4.y, u4.z, u4.w};
 #pragma unroll
             for (int c = 0; c < 4; ++c) {
                 ag[0][c] = fmaf(a0, g[c], ag[0][c]); ag[1][c] = fmaf(a1, g[c], ag[1][c]);
-                au[0][c] = fmaf(a0, uu[c], au[0][c]); au[1][c] = fmaf(a1, uu[c], au[1][c]);
+                if (GLU) { au[0][c] = fmaf(a0, uu[c], au[0][c]); au[1][c] = fmaf(a1, uu[c], au[1][c]); }
             }
         }
         __syncthreads();
@@ -1373,7 +1388,7 @@ moe_up_kernel(const TA* __restrict__ x, const TW* __restrict__ wgu, const int* _
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
             const int n = n0 + 4 * tx + c;
-            if (n < F) sp_st(act, (size_t)(first + m) * F + n, hy_clamped_glu(ag[r][c], au[r][c], limit, slope));
+            if (n < F) sp_st(act, (size_t)(first + m) * F + n, GLU ? hy_clamped_glu(ag[r][c], au[r][c], limit, slope) : sp_relu2(ag[r][c]));
         }
     }
 }
@@ -1435,23 +1450,25 @@ moe_down_kernel(const TA* __restrict__ act, const TW* __restrict__ wd, const int
 // blocks of 32 through three shared-memory stages filled by cp.async (two in flight while one is multiplied: a decode
 // step's tiles are bound by how many bytes a CTA has asked for); four warps, each 32 rows x all columns with
 // mma.sync m16n8k16 (A and B fragments by ldmatrix from rows padded to 80 bytes); a group of 16 rows beyond the tile's
-// rows (a decode step's tiles hold a row or two) is skipped. GLU: the tile holds the gate and the
-// up columns of the same outputs and stores the activation; else the result times the pair's weight goes to the
-// pair's row of ``out``. A row's sum runs over k in the same order whatever tile or batch the row is in.
+// rows (a decode step's tiles hold a row or two) is skipped. MM_GLU: the tile holds the gate and the
+// up columns of the same outputs and stores the activation; MM_UP: up columns alone, the store is the square of their
+// relu; MM_DOWN: the result times the pair's weight goes to the pair's row of ``out``. A row's sum runs over k in the same order whatever tile or batch the row is in.
 #define MM_TM 128
 #define MM_BN 64
 #define MM_BK 32
 #define MM_ROW 40
 #define MM_STAGES 3
-template <bool GLU>
-constexpr size_t mm_smem_bytes() { return (size_t)MM_STAGES * (MM_TM + (GLU ? 2 : 1) * MM_BN) * MM_ROW * sizeof(__nv_bfloat16); }
-template <bool GLU>
+enum { MM_DOWN = 0, MM_GLU = 1, MM_UP = 2 };
+template <int KIND>
+constexpr size_t mm_smem_bytes() { return (size_t)MM_STAGES * (MM_TM + (KIND == MM_GLU ? 2 : 1) * MM_BN) * MM_ROW * sizeof(__nv_bfloat16); }
+template <int KIND>
 __global__ void __launch_bounds__(128, 3)
 moe_mma_kernel(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bfloat16* __restrict__ Wt, long long w_stride,
                int N, int K, const int* __restrict__ sorted, const int* __restrict__ tiles, int top,
                __nv_bfloat16* __restrict__ act, float* __restrict__ out, const float* __restrict__ wts, float limit,
                float slope, int blk) {
-    // ``blk`` (GLU): 0 = an expert's N gate rows, then its N up rows; else blocks of ``blk`` gate rows, each followed by
+    constexpr bool GLU = KIND == MM_GLU, DOWN = KIND == MM_DOWN;
+    // ``blk`` (MM_GLU): 0 = an expert's N gate rows, then its N up rows; else blocks of ``blk`` gate rows, each followed by
     // the ``blk`` up rows of the same outputs (the layout the tcgen05 tile kernel's gated epilogue reads)
     extern __shared__ __align__(16) unsigned char mm_smem[];
     typedef __nv_bfloat16 (*ATile)[MM_TM][MM_ROW];
@@ -1465,7 +1482,7 @@ moe_mma_kernel(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bfloat16
     const int n0 = blockIdx.y * MM_BN;
     if (threadIdx.x < MM_TM) {
         const int m = (int)threadIdx.x;
-        src_row[m] = m < rows ? (GLU ? sorted[first + m] / top : first + m) : -1;
+        src_row[m] = m < rows ? (DOWN ? first + m : sorted[first + m] / top) : -1;
     }
     __syncthreads();
     const __nv_bfloat16* w0 = Wt + (size_t)e * w_stride;
@@ -1559,8 +1576,8 @@ moe_mma_kernel(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bfloat16
         for (int half = 0; half < 2; ++half) {
             const int m = (lane >> 2) + 8 * half;
             if (m >= rows) continue;
-            const int p = GLU ? 0 : sorted[first + m];
-            const float wt = GLU ? 0.0f : wts[p];
+            const int p = DOWN ? sorted[first + m] : 0;
+            const float wt = DOWN ? wts[p] : 0.0f;
 #pragma unroll
             for (int j = 0; j < 2; ++j) {
                 const int n = n0 + (2 * warp + j) * 8 + (lane & 3) * 2;
@@ -1568,7 +1585,8 @@ moe_mma_kernel(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bfloat16
                 for (int u = 0; u < 2; ++u) {
                     if (n + u >= N) continue;
                     if (GLU) act[(size_t)(first + m) * N + n + u] = __float2bfloat16_rn(hy_clamped_glu(acc[0][0][j][2 * half + u], acc[0][GLU ? 1 : 0][j][2 * half + u], limit, slope));
-                    else out[(size_t)p * N + n + u] = acc[0][0][j][2 * half + u] * wt;
+                    else if (DOWN) out[(size_t)p * N + n + u] = acc[0][0][j][2 * half + u] * wt;
+                    else act[(size_t)(first + m) * N + n + u] = __float2bfloat16_rn(sp_relu2(acc[0][0][j][2 * half + u]));
                 }
             }
         }
@@ -1580,8 +1598,8 @@ moe_mma_kernel(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bfloat16
         for (int half = 0; half < 2; ++half) {
             const int m = warp * 32 + f * 16 + (lane >> 2) + 8 * half;
             if (m >= rows) continue;
-            const int p = GLU ? 0 : sorted[first + m];
-            const float wt = GLU ? 0.0f : wts[p];
+            const int p = DOWN ? sorted[first + m] : 0;
+            const float wt = DOWN ? wts[p] : 0.0f;
 #pragma unroll
             for (int nt = 0; nt < 8; ++nt) {
                 const int n = n0 + nt * 8 + (lane & 3) * 2;
@@ -1589,34 +1607,43 @@ moe_mma_kernel(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bfloat16
                 for (int u = 0; u < 2; ++u) {
                     if (n + u >= N) continue;
                     if (GLU) act[(size_t)(first + m) * N + n + u] = __float2bfloat16_rn(hy_clamped_glu(acc[f][0][nt][2 * half + u], acc[f][GLU ? 1 : 0][nt][2 * half + u], limit, slope));
-                    else out[(size_t)p * N + n + u] = acc[f][0][nt][2 * half + u] * wt;
+                    else if (DOWN) out[(size_t)p * N + n + u] = acc[f][0][nt][2 * half + u] * wt;
+                    else act[(size_t)(first + m) * N + n + u] = __float2bfloat16_rn(sp_relu2(acc[f][0][nt][2 * half + u]));
                 }
             }
         }
 }
 
-// y[t] += Σ_k out[t·top + k] in the order of k
-__global__ void moe_combine_kernel(const float* __restrict__ out, float* __restrict__ y, size_t T, int top, int W) {
+// y[t] += Σ_k out[t·top + k] in the order of k; with ``ids`` a pair whose id is E or more adds its weight · x[t]
+template <typename TX>
+__global__ void moe_combine_kernel(const float* __restrict__ out, float* __restrict__ y, size_t T, int top, int W,
+                                   const int* __restrict__ ids, int E, const float* __restrict__ wts, const TX* __restrict__ x) {
     const size_t n = T * (size_t)W;
     for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < n; e += (size_t)gridDim.x * blockDim.x) {
         const size_t t = e / W;
         const int c = (int)(e % W);
         float v = 0.0f;
-        for (int k = 0; k < top; ++k) v += out[(t * top + k) * W + c];
+        for (int k = 0; k < top; ++k) {
+            const size_t p = t * top + k;
+            v += (ids && ids[p] >= E) ? wts[p] * sp_ld(x, t * W + c) : out[p * W + c];
+        }
         y[e] += v;
     }
 }
 
 SP_API int sp_moe_experts(const void* x, int x_dt, const int* ids, const void* wgu, const void* wd, int w_dt, int E,
                           int* counts, int* sorted, int* tiles, int max_tiles, const float* wts, void* act, float* out_pairs,
-                          float* y, int T, int top, int W, int F, float limit, float slope, int glu_block,
-                          cudaStream_t stream) {
+                          float* y, int T, int top, int W, int F, float limit, float slope, int glu_block, int act_kind,
+                          int identities, cudaStream_t stream) {
+    // ``act_kind`` SP_ACT_RELU2: ``wgu`` holds up rows alone, F per expert; ``identities``: ids of E and more are in use
     if (T <= 0) return 0;
     const int n_pairs = T * top;
     if (glu_block && (x_dt != SP_DT_BF16 || w_dt != SP_DT_BF16 || F % glu_block))
         SP_FAIL("moe_experts: gate and up rows in blocks of %d are a bfloat16 layout for sizes that are multiples of it", glu_block);
     const bool mma = x_dt == SP_DT_BF16 && w_dt == SP_DT_BF16 && W % 8 == 0 && F % 8 == 0 &&
                      (((uintptr_t)x | (uintptr_t)wgu | (uintptr_t)wd | (uintptr_t)act) & 15) == 0;
+    const bool glu = act_kind != SP_ACT_RELU2;
+    if (!glu && glu_block) SP_FAIL("moe_experts: experts without a gate have no blocks of gate and up rows");
     if (mma && ((long long)T * W >= (1LL << 31) || (long long)n_pairs * F >= (1LL << 31) || 2LL * F * W >= (1LL << 31)))
         SP_FAIL("moe_experts: operands beyond 2^31 elements");
     const int tm = mma ? MM_TM : ME_TM;
@@ -1626,16 +1653,22 @@ SP_API int sp_moe_experts(const void* x, int x_dt, const int* ids, const void* w
         const int used = (n_pairs + tm - 1) / tm + E;           // entries beyond the tiles in use say expert -1
         static SpPerDevice mma_ready;
         if (!mma_ready.done()) {
-            if (cudaFuncSetAttribute(moe_mma_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)mm_smem_bytes<true>()) != cudaSuccess ||
-                cudaFuncSetAttribute(moe_mma_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)mm_smem_bytes<false>()) != cudaSuccess)
+            if (cudaFuncSetAttribute(moe_mma_kernel<MM_GLU>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)mm_smem_bytes<MM_GLU>()) != cudaSuccess ||
+                cudaFuncSetAttribute(moe_mma_kernel<MM_UP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)mm_smem_bytes<MM_UP>()) != cudaSuccess ||
+                cudaFuncSetAttribute(moe_mma_kernel<MM_DOWN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)mm_smem_bytes<MM_DOWN>()) != cudaSuccess)
                 SP_FAIL("moe_experts: cannot raise the shared memory limit");
             mma_ready.mark();
         }
-        moe_mma_kernel<true><<<dim3(used, (F + MM_BN - 1) / MM_BN), 128, mm_smem_bytes<true>(), stream>>>(
-            (const __nv_bfloat16*)x, W, (const __nv_bfloat16*)wgu, 2LL * F * W, F, W, sorted, tiles, top,
-            (__nv_bfloat16*)act, nullptr, nullptr, limit, slope, glu_block);
+        if (glu)
+            moe_mma_kernel<MM_GLU><<<dim3(used, (F + MM_BN - 1) / MM_BN), 128, mm_smem_bytes<MM_GLU>(), stream>>>(
+                (const __nv_bfloat16*)x, W, (const __nv_bfloat16*)wgu, 2LL * F * W, F, W, sorted, tiles, top,
+                (__nv_bfloat16*)act, nullptr, nullptr, limit, slope, glu_block);
+        else
+            moe_mma_kernel<MM_UP><<<dim3(used, (F + MM_BN - 1) / MM_BN), 128, mm_smem_bytes<MM_UP>(), stream>>>(
+                (const __nv_bfloat16*)x, W, (const __nv_bfloat16*)wgu, (long long)F * W, F, W, sorted, tiles, top,
+                (__nv_bfloat16*)act, nullptr, nullptr, 0.0f, 0.0f, 0);
         SP_CHECK_LAUNCH("moe_up (tensor cores)");
-        moe_mma_kernel<false><<<dim3(used, (W + MM_BN - 1) / MM_BN), 128, mm_smem_bytes<false>(), stream>>>(
+        moe_mma_kernel<MM_DOWN><<<dim3(used, (W + MM_BN - 1) / MM_BN), 128, mm_smem_bytes<MM_DOWN>(), stream>>>(
             (const __nv_bfloat16*)act, F, (const __nv_bfloat16*)wd, (long long)W * F, W, F, sorted, tiles, top, nullptr,
             out_pairs, wts, 0.0f, 0.0f, 0);
         SP_CHECK_LAUNCH("moe_down (tensor cores)");
@@ -1644,7 +1677,8 @@ SP_API int sp_moe_experts(const void* x, int x_dt, const int* ids, const void* w
         const dim3 g_up(max_tiles, (F + ME_BN - 1) / ME_BN), g_down(max_tiles, (W + ME_BN - 1) / ME_BN);
 #define ME_LAUNCH(TA, TW)                                                                                             \
     do {                                                                                                              \
-        moe_up_kernel<TA, TW><<<g_up, 256, 0, stream>>>((const TA*)x, (const TW*)wgu, sorted, tiles, (TA*)act, top, W, F, limit, slope); \
+        if (glu) moe_up_kernel<TA, TW, true><<<g_up, 256, 0, stream>>>((const TA*)x, (const TW*)wgu, sorted, tiles, (TA*)act, top, W, F, limit, slope); \
+        else moe_up_kernel<TA, TW, false><<<g_up, 256, 0, stream>>>((const TA*)x, (const TW*)wgu, sorted, tiles, (TA*)act, top, W, F, limit, slope); \
         SP_CHECK_LAUNCH("moe_up");                                                                                    \
         moe_down_kernel<TA, TW><<<g_down, 256, 0, stream>>>((const TA*)act, (const TW*)wd, sorted, tiles, wts, out_pairs, W, F); \
         SP_CHECK_LAUNCH("moe_down");                                                                                  \
@@ -1657,7 +1691,10 @@ SP_API int sp_moe_experts(const void* x, int x_dt, const int* ids, const void* w
     }
     const size_t n = (size_t)T * W;
     const size_t want = (n + 255) / 256;
-    moe_combine_kernel<<<(unsigned)(want > 148 * 16 ? 148 * 16 : want), 256, 0, stream>>>(out_pairs, y, (size_t)T, top, W);
+    const unsigned blocks = (unsigned)(want > 148 * 16 ? 148 * 16 : want);
+    const int* same = identities ? ids : nullptr;
+    if (x_dt == SP_DT_F32) moe_combine_kernel<float><<<blocks, 256, 0, stream>>>(out_pairs, y, (size_t)T, top, W, same, E, wts, (const float*)x);
+    else moe_combine_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>(out_pairs, y, (size_t)T, top, W, same, E, wts, (const __nv_bfloat16*)x);
     SP_CHECK_LAUNCH("moe_combine");
     return 0;
 }

@@ -130,13 +130,21 @@ def embed_gather(table, ids, out, status=None, scale: float = 1.0):
         T, H, table.shape[0], c_void_p(_ptr(status)), c_float(scale), c_void_p(_stream())))
 
 
-def rmsnorm(x, weight, out, eps, rows=None):
-    """out[r,:] = x[rows[r] or r,:] / sqrt(mean(x²)+eps) · weight; ``x`` is float32."""
+def rmsnorm(x, weight, out, eps, rows=None, add=None):
+    """out[r,:] = x[rows[r] or r,:] / sqrt(mean(x²)+eps) · weight; ``x`` is float32. ``add`` (float32 [H], without
+    ``rows``): x[r,:] += add first, in place and in the same pass."""
     lib = load("generic")
     if x.dtype != torch.float32:
         raise KernelError("rmsnorm reads the 32-bit residual stream")
-    _need_contig(x, weight, out, rows)
+    _need_contig(x, weight, out, rows, add)
     n_rows, H = out.shape
+    if add is not None:
+        if rows is not None or add.dtype != torch.float32 or add.numel() != H or x.shape != out.shape:
+            raise KernelError("rmsnorm: the row added to the whole stream is float32 and as wide as the stream")
+        _check("generic", lib.sp_rmsnorm_add_row(
+            c_void_p(_ptr(x)), c_void_p(_ptr(add)), c_void_p(_ptr(weight)), dt_code(weight), c_void_p(_ptr(out)), dt_code(out),
+            n_rows, H, c_float(eps), c_void_p(_stream())))
+        return
     _check("generic", lib.sp_rmsnorm(
         c_void_p(_ptr(x)), c_void_p(_ptr(weight)), dt_code(weight), c_void_p(_ptr(out)), dt_code(out),
         c_void_p(_ptr(rows)), n_rows, H, c_float(eps), c_void_p(_stream())))
@@ -226,15 +234,33 @@ def scale_rows_sigmoid(x, z):
                                                 c_void_p(_stream())))
 
 
-def silu_mul(gu, out):
-    """out[r,:] = silu(gu[r,:I]) ⊙ gu[r,I:]."""
+def gate_elements(x, z, mult: float = 1.0):
+    """x[t, c] ← x[t, c] · sigmoid(z[t, c]) · mult in place; ``z`` float32, possibly columns of wider rows."""
+    lib = load("generic")
+    if z.dtype != torch.float32 or z.shape != x.shape or z.stride(1) != 1 or not z.is_cuda:
+        raise KernelError("gate_elements takes one float32 gate per element, rows of unit stride")
+    _need_contig(x)
+    _check("generic", lib.sp_gate_elements(c_void_p(_ptr(x)), dt_code(x), c_void_p(z.data_ptr()), x.shape[0], x.shape[1],
+                                           z.stride(0), c_float(mult), c_void_p(_stream())))
+
+
+ACT_SILU, ACT_GELU, ACT_RELU2 = 0, 1, 2       # the kernels' activation codes (common.cuh)
+
+
+def gated_mul(gu, out, act=ACT_SILU, mult: float = 1.0):
+    """out[r,:] = act(gu[r,:I]) ⊙ gu[r,I:] · mult."""
     lib = load("generic")
     rows, I = out.shape
     _need_contig(gu, out)
     if gu.dtype != out.dtype or gu.shape[1] != 2 * I:
-        raise KernelError("silu_mul wants gu [rows, 2·I] and out [rows, I] of one dtype")
-    _check("generic", lib.sp_silu_mul(c_void_p(_ptr(gu)), c_void_p(_ptr(out)), dt_code(out), rows, I,
-                                      c_void_p(_stream())))
+        raise KernelError("gated_mul wants gu [rows, 2·I] and out [rows, I] of one dtype")
+    _check("generic", lib.sp_gated_mul(c_void_p(_ptr(gu)), c_void_p(_ptr(out)), dt_code(out), rows, I, int(act),
+                                       c_float(mult), c_void_p(_stream())))
+
+
+def silu_mul(gu, out):
+    """out[r,:] = silu(gu[r,:I]) ⊙ gu[r,I:]."""
+    gated_mul(gu, out)
 
 
 def add_inplace(dst, src):
@@ -245,6 +271,15 @@ def add_inplace(dst, src):
         raise KernelError("add_inplace wants a float32 destination and equal sizes")
     _check("generic", lib.sp_add_inplace(c_void_p(_ptr(dst)), c_void_p(_ptr(src)), dt_code(src),
                                          c_longlong(dst.numel()), c_void_p(_stream())))
+
+
+def add_row(x, row):
+    """Every row of ``x`` (float32 [T, W]) += ``row`` (float32 [W])."""
+    lib = load("generic")
+    _need_contig(x, row)
+    if x.dtype != torch.float32 or row.dtype != torch.float32 or row.numel() != x.shape[1]:
+        raise KernelError("add_row wants a float32 matrix and a float32 row of its width")
+    _check("generic", lib.sp_add_row(c_void_p(_ptr(x)), c_void_p(_ptr(row)), x.shape[0], x.shape[1], c_void_p(_stream())))
 
 
 def gather_i32(src, idx, dst):
@@ -416,12 +451,12 @@ def tc_gemm_supported(a: torch.Tensor, w: torch.Tensor) -> bool:
 TC_STORE, TC_ACCUMULATE, TC_SILU_MUL = 0, 1, 2
 
 
-def tc_gemm(a, w, out, mode=TC_STORE, bn=128):
+def tc_gemm(a, w, out, mode=TC_STORE, bn=128, act=ACT_SILU, mult: float = 1.0):
     """out = a · wᵀ on the tcgen05 tensor cores (bfloat16 operands, float32 accumulation).
 
     ``mode`` TC_STORE writes ``out`` (bfloat16 or float32), TC_ACCUMULATE adds into a float32 ``out``,
     TC_SILU_MUL takes a weight whose rows interleave gate and up in blocks of ``bn``/2 and writes
-    silu(gate)·up into ``out`` [M, N/2].
+    silu(gate)·up into ``out`` [M, N/2] (``act`` ACT_GELU: gelu(gate)·up; times ``mult``).
     """
     lib = load("tc_gemm")
     M, K = a.shape
@@ -431,6 +466,11 @@ def tc_gemm(a, w, out, mode=TC_STORE, bn=128):
         raise KernelError(f"tc_gemm: out {tuple(out.shape)} does not fit a {tuple(a.shape)}, w {tuple(w.shape)}")
     if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise KernelError("tc_gemm takes bfloat16 operands")
+    if mode == TC_SILU_MUL and (act != ACT_SILU or mult != 1.0):
+        _check("tc_gemm", lib.sp_tc_gemm_gated(
+            c_void_p(_ptr(a)), c_void_p(_ptr(w)), c_void_p(_ptr(out)), dt_code(out), M, N, K, a.stride(0), w.stride(0),
+            out.stride(0), int(bn), int(act), c_float(mult), c_void_p(_ptr(status_word(a.device))), c_void_p(_stream())))
+        return
     _check("tc_gemm", lib.sp_tc_gemm(
         c_void_p(_ptr(a)), c_void_p(_ptr(w)), c_void_p(_ptr(out)), dt_code(out), M, N, K,
         a.stride(0), w.stride(0), out.stride(0), int(mode), int(bn), c_void_p(_ptr(status_word(a.device))),
@@ -668,7 +708,7 @@ def gemv_supported(x: torch.Tensor, w: torch.Tensor) -> bool:
             and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
-def gemv(x, w, out, mode=TC_STORE, pair=0):
+def gemv(x, w, out, mode=TC_STORE, pair=0, act=ACT_SILU, mult: float = 1.0):
     """out = x · wᵀ for up to 64 tokens, streaming ``w`` once. Modes as ``tc_gemm``; for TC_SILU_MUL
     ``pair`` is the number of gate rows before the matching up rows in the interleaved weight."""
     lib = load("gemv")
@@ -677,6 +717,11 @@ def gemv(x, w, out, mode=TC_STORE, pair=0):
     want_cols = N // 2 if mode == TC_SILU_MUL else N
     if out.shape[0] != M or out.shape[1] != want_cols or out.stride(1) != 1:
         raise KernelError(f"gemv: out {tuple(out.shape)} does not fit x {tuple(x.shape)}, w {tuple(w.shape)}")
+    if mode == TC_SILU_MUL and (act != ACT_SILU or mult != 1.0):
+        _check("gemv", lib.sp_gemv_gated(
+            c_void_p(_ptr(x)), c_void_p(_ptr(w)), c_void_p(_ptr(out)), dt_code(out), M, N, K, x.stride(0), w.stride(0),
+            out.stride(0), int(pair), int(act), c_float(mult), c_void_p(_stream())))
+        return
     _check("gemv", lib.sp_gemv(
         c_void_p(_ptr(x)), c_void_p(_ptr(w)), c_void_p(_ptr(out)), dt_code(out), M, N, K,
         x.stride(0), w.stride(0), out.stride(0), int(mode), int(pair), c_void_p(_stream())))
@@ -873,7 +918,7 @@ def tc_stream_supported(x: torch.Tensor, w: torch.Tensor, mode=TC_STORE, pair: i
         int(mode), int(pair)) == 0
 
 
-def tc_stream(x, w, out, mode=TC_STORE, pair=0):
+def tc_stream(x, w, out, mode=TC_STORE, pair=0, act=ACT_SILU, mult: float = 1.0):
     """out = x · wᵀ for up to 128 tokens on the tensor cores with the rows of ``w`` as the instruction's M: every SM
     streams its share of ``w``; K is cut over the CTAs of a cluster, whose pieces are added in a fixed order. Modes as ``tc_gemm``; for
     TC_SILU_MUL ``pair`` is the number of gate rows before the matching up rows in the interleaved weight."""
@@ -883,6 +928,11 @@ def tc_stream(x, w, out, mode=TC_STORE, pair=0):
     want_cols = N // 2 if mode == TC_SILU_MUL else N
     if out.shape[0] != M or out.shape[1] != want_cols or out.stride(1) != 1:
         raise KernelError(f"tc_stream: out {tuple(out.shape)} does not fit x {tuple(x.shape)}, w {tuple(w.shape)}")
+    if mode == TC_SILU_MUL and (act != ACT_SILU or mult != 1.0):
+        _check("tc_stream", lib.sp_tc_stream_gated(
+            c_void_p(_ptr(x)), c_void_p(_ptr(w)), c_void_p(_ptr(out)), dt_code(out), M, N, K, x.stride(0), w.stride(0),
+            out.stride(0), int(pair), int(act), c_float(mult), c_void_p(_ptr(status_word(x.device))), c_void_p(_stream())))
+        return
     _check("tc_stream", lib.sp_tc_stream(
         c_void_p(_ptr(x)), c_void_p(_ptr(w)), c_void_p(_ptr(out)), dt_code(out), M, N, K, x.stride(0), w.stride(0),
         out.stride(0), int(mode), int(pair), c_void_p(_ptr(status_word(x.device))), c_void_p(_stream())))
@@ -1191,10 +1241,10 @@ def clamped_glu(gu, out, limit, slope=1.702):
 
 
 def moe_select(z, correction, ids, weights, top, n_groups=1, keep=1, softmax=False, weight_scale=1.0, experts=None,
-               extra=None):
+               extra=None, normalize=True):
     """From router logits ``z`` (float32 [T, E]): the ``top`` experts per token by s + correction (s = sigmoid(z), or
     with ``softmax`` the softmax over the row's experts) among the ``keep`` best of ``n_groups`` groups (a group's
-    score: its two largest), and their weights s / Σ s · ``weight_scale``. ``experts`` < z's columns: the row's other
+    score: its two largest), and their weights s / Σ s · ``weight_scale`` (``normalize`` False: s · ``weight_scale``). ``experts`` < z's columns: the row's other
     columns are copied to ``extra`` (float32 [T, columns − experts])."""
     lib = load("hybrid")
     if z.dtype != torch.float32 or ids.dtype != torch.int32 or weights.dtype != torch.float32:
@@ -1208,7 +1258,7 @@ def moe_select(z, correction, ids, weights, top, n_groups=1, keep=1, softmax=Fal
     _check("hybrid", lib.sp_moe_select(
         c_void_p(_ptr(z)), c_void_p(_ptr(correction)), dt_code(correction) if correction is not None else 0,
         c_void_p(_ptr(ids)), c_void_p(_ptr(weights)), T, E, ldz, int(top), int(n_groups or 1), int(keep or 1),
-        int(bool(softmax)), c_float(weight_scale), c_void_p(_ptr(extra)), c_void_p(_stream())))
+        int(bool(softmax)), c_float(weight_scale), int(bool(normalize)), c_void_p(_ptr(extra)), c_void_p(_stream())))
 
 
 def moe_tile_rows() -> int:
@@ -1218,23 +1268,28 @@ def moe_tile_rows() -> int:
 TC_EXPERT_PAIRS = 512        # from this many (token, expert) pairs on, and 8 per expert, whole 128-row tiles pay off
 
 
-def moe_experts(x, ids, weights, w_gate_up, w_down, y, top, limit, slope=1.702, glu_block=0):
+def moe_experts(x, ids, weights, w_gate_up, w_down, y, top, limit, slope=1.702, glu_block=0, act=ACT_SILU, identities=False):
     """y (float32 [T, W]) += Σ_k weights[t,k] · expert_{ids[t,k]}(x[t]) with clamped-GLU experts: ``w_gate_up``
     [E, 2F, W] (an expert's gate rows, then its up rows; with ``glu_block`` = b: blocks of b gate rows, each followed by
-    the b up rows of the same outputs), ``w_down`` [E, W, F]. The (token, expert) pairs are sorted by expert on the
+    the b up rows of the same outputs), ``w_down`` [E, W, F]. ``act`` ACT_RELU2: experts without a gate, ``w_gate_up`` is
+    [E, F, W] and an expert is w_down · relu(w_up · x)². ``identities``: an id of E or more names an expert that returns
+    its input (no product; the combining kernel adds weight · x). The (token, expert) pairs are sorted by expert on the
     device; nothing comes back to the host. Many pairs in the block layout: the products run as grouped products of the
     tcgen05 tile kernel over rows gathered into 128-row tiles of one expert each."""
     lib = load("hybrid")
     _need_contig(x, ids, weights, w_gate_up, w_down, y)
     T, W = x.shape
     E, F2, _ = w_gate_up.shape
-    F = F2 // 2
+    glu = act != ACT_RELU2
+    F = F2 // 2 if glu else F2
     n_pairs = T * top
     dev = x.device
     if ids.dtype != torch.int32 or weights.dtype != torch.float32 or y.dtype != torch.float32:
         raise KernelError("moe_experts takes int32 ids, float32 weights and adds into a float32 matrix")
     global launches
-    if (glu_block and n_pairs >= max(TC_EXPERT_PAIRS, 8 * E) and W % 128 == 0 and F % 8 == 0 and W % 4 == 0
+    if w_down.shape != (E, W, F):
+        raise KernelError(f"moe_experts: w_down {tuple(w_down.shape)} does not fit up rows {tuple(w_gate_up.shape)}")
+    if ((glu_block or not glu) and n_pairs >= max(TC_EXPERT_PAIRS, 8 * E) and W % 128 == 0 and F % 8 == 0 and W % 4 == 0
             and tc_gemm_supported(x, w_gate_up[0]) and w_down.dtype == torch.bfloat16):
         tc = load("tc_gemm")
         max_tiles = (n_pairs + 127) // 128 + E
@@ -1244,36 +1299,38 @@ def moe_experts(x, ids, weights, w_gate_up, w_down, y, top, limit, slope=1.702, 
         rest = book[E + rows + n_pairs:]
         tiles, tab_up, tab_down = rest[:3 * max_tiles], rest[3 * max_tiles:4 * max_tiles], rest[4 * max_tiles:]
         xs = torch.empty(rows, W, dtype=torch.bfloat16, device=dev)
-        act = torch.empty(rows, F, dtype=torch.bfloat16, device=dev)
+        hidden = torch.empty(rows, F, dtype=torch.bfloat16, device=dev)
         out_rows = torch.empty(rows, W, dtype=torch.float32, device=dev)
         launches += 6
         _check("hybrid", lib.sp_moe_plan_tiles(
-            c_void_p(_ptr(x)), c_void_p(_ptr(ids)), T, int(top), W, E, 2 * F, W, c_void_p(_ptr(counts)), c_void_p(_ptr(order)),
+            c_void_p(_ptr(x)), c_void_p(_ptr(ids)), T, int(top), W, E, F2, W, c_void_p(_ptr(counts)), c_void_p(_ptr(order)),
             c_void_p(_ptr(pos)), c_void_p(_ptr(tiles)), c_void_p(_ptr(tab_up)), c_void_p(_ptr(tab_down)), max_tiles,
             c_void_p(_ptr(xs)), c_void_p(_stream())))
         status = c_void_p(_ptr(status_word(dev)))
         _check("tc_gemm", tc.sp_tc_gemm_grouped(
-            c_void_p(_ptr(xs)), c_void_p(_ptr(w_gate_up)), c_void_p(_ptr(act)), dt_code(act), rows, 2 * F, W, W, W, E * 2 * F, F,
-            TC_SILU_MUL, 2 * int(glu_block), c_void_p(_ptr(tab_up)), c_float(limit), c_float(slope), status, c_void_p(_stream())))
+            c_void_p(_ptr(xs)), c_void_p(_ptr(w_gate_up)), c_void_p(_ptr(hidden)), dt_code(hidden), rows, F2, W, W, W, E * F2, F,
+            TC_SILU_MUL if glu else TC_STORE, 2 * int(glu_block) if glu else (256 if F % 256 == 0 else 128),
+            c_void_p(_ptr(tab_up)), c_float(limit), c_float(slope), int(act), status, c_void_p(_stream())))
         _check("tc_gemm", tc.sp_tc_gemm_grouped(
-            c_void_p(_ptr(act)), c_void_p(_ptr(w_down)), c_void_p(_ptr(out_rows)), dt_code(out_rows), rows, W, F, F, F, E * W, W,
-            TC_STORE, 256 if W % 256 == 0 else 128, c_void_p(_ptr(tab_down)), c_float(0.0), c_float(0.0), status,
+            c_void_p(_ptr(hidden)), c_void_p(_ptr(w_down)), c_void_p(_ptr(out_rows)), dt_code(out_rows), rows, W, F, F, F, E * W, W,
+            TC_STORE, 256 if W % 256 == 0 else 128, c_void_p(_ptr(tab_down)), c_float(0.0), c_float(0.0), ACT_SILU, status,
             c_void_p(_stream())))
-        _check("hybrid", lib.sp_moe_combine_rows(c_void_p(_ptr(out_rows)), c_void_p(_ptr(pos)), c_void_p(_ptr(weights)),
-                                                 c_void_p(_ptr(y)), T, int(top), W, c_void_p(_stream())))
+        _check("hybrid", lib.sp_moe_combine_rows(
+            c_void_p(_ptr(out_rows)), c_void_p(_ptr(pos)), c_void_p(_ptr(weights)), c_void_p(_ptr(y)), T, int(top), W,
+            c_void_p(_ptr(ids) if identities else None), E, c_void_p(_ptr(x)), c_void_p(_stream())))
         return
     tm = moe_tile_rows()
     max_tiles = (n_pairs + tm - 1) // tm + E
     book = torch.empty(E + n_pairs + 3 * max_tiles, dtype=torch.int32, device=dev)
     counts, order, tiles = book[:E], book[E:E + n_pairs], book[E + n_pairs:]
-    act = torch.empty(n_pairs, F, dtype=x.dtype, device=dev)
+    hidden = torch.empty(n_pairs, F, dtype=x.dtype, device=dev)
     out_pairs = torch.empty(n_pairs, W, dtype=torch.float32, device=dev)
     launches += 4
     _check("hybrid", lib.sp_moe_experts(
         c_void_p(_ptr(x)), dt_code(x), c_void_p(_ptr(ids)), c_void_p(_ptr(w_gate_up)), c_void_p(_ptr(w_down)),
         _w_dt(w_gate_up, w_down), E, c_void_p(_ptr(counts)), c_void_p(_ptr(order)), c_void_p(_ptr(tiles)), max_tiles,
-        c_void_p(_ptr(weights)), c_void_p(_ptr(act)), c_void_p(_ptr(out_pairs)), c_void_p(_ptr(y)), T, int(top), W, F,
-        c_float(limit), c_float(slope), int(glu_block), c_void_p(_stream())))
+        c_void_p(_ptr(weights)), c_void_p(_ptr(hidden)), c_void_p(_ptr(out_pairs)), c_void_p(_ptr(y)), T, int(top), W, F,
+        c_float(limit), c_float(slope), int(glu_block), int(act), int(bool(identities)), c_void_p(_stream())))
 
 
 # ------------------------------------------------------------------ latent: attention through a cached low-rank latent
@@ -1400,11 +1457,11 @@ def gated_qkv_store(proj, bias, q_out, k_pool, v_pool, meta, gates, freq, nh, nk
         c_float(rot_mult), c_float(temp_coef), int(temp_every), c_void_p(_stream())))
 
 
-def latent_rot_store(proj, wc, q_out, pool, meta, gates, freq, H, d, rd, rank, rot_mult, eps, rows_out=None):
+def latent_rot_store(proj, wc, q_out, pool, meta, gates, freq, H, d, rd, rank, rot_mult, eps, rows_out=None, halves=False):
     """``proj`` rows (float32) = [q: H·(d + rd) | row: rank | key part: rd | gates: H] (``pool`` None: no row and no key
     part). The row's RMS norm with ``wc`` and the key part with its neighbouring pairs rotated go into ONE page row
     [rank + rd] of ``pool``; every head's last ``rd`` query dims are rotated the same way; q to ``q_out``, the gates'
-    arguments to ``gates`` (float32 [T, H]). ``rows_out`` [T, rank + rd] also receives the page rows token by token."""
+    arguments to ``gates`` (float32 [T, H], or None). ``halves``: dim i pairs with dim i + rd/2 instead. ``rows_out`` [T, rank + rd] also receives the page rows token by token."""
     lib = load("sandwich")
     if proj.dtype != torch.float32:
         raise KernelError("latent_rot_store reads 32-bit projections")
@@ -1417,7 +1474,7 @@ def latent_rot_store(proj, wc, q_out, pool, meta, gates, freq, H, d, rd, rank, r
         dt_code(q_out), c_void_p(_ptr(pool)), dt_code(pool) if pool is not None else 0, c_void_p(_ptr(rows_out)),
         c_void_p(_ptr(gates)), c_void_p(_ptr(freq)), c_void_p(_ptr(meta.token_seq)), c_void_p(_ptr(meta.positions)),
         c_void_p(_ptr(meta.seq_slot)), c_void_p(_ptr(pt)), pt.shape[1], meta.page_size, proj.shape[0], int(H), int(d), int(rd),
-        int(rank), c_float(rot_mult), c_float(eps), c_void_p(_stream())))
+        int(rank), int(bool(halves)), c_float(rot_mult), c_float(eps), c_void_p(_stream())))
 
 
 def gelu_gather_mul(z, table, ids, out, offset):
@@ -1429,3 +1486,36 @@ def gelu_gather_mul(z, table, ids, out, offset):
     _check("sandwich", lib.sp_gelu_gather_mul(
         c_void_p(_ptr(z)), dt_code(z), c_void_p(_ptr(table)), dt_code(table), c_void_p(_ptr(ids)), c_void_p(_ptr(out)),
         z.shape[0], z.shape[1], table.shape[1], int(offset), table.shape[0], c_void_p(_stream())))
+
+
+# ------------------------------------------------------------------ rglru: a gated linear recurrence behind a short convolution
+def rglru(proj, w: dict, ring, state, out, step, width, taps, parts, mult=1.0):
+    """``proj`` rows [y: width | x: width] (float32, without biases); ``w``: float32 ``yb``, ``xb``, ``conv`` [width, taps],
+    ``convb``, ``rab``, ``rib``, ``decay`` (the positive factor of the gate in −log a) and the gate matrices ``ra``, ``ri``
+    [parts, width/parts, width/parts] in their storage type; ``ring`` float32 [slots, taps, width] (None with one tap),
+    ``state`` float32 [slots, width]; ``out`` [T, width] = state ⊙ gelu(y) · mult."""
+    lib = load("rglru")
+    if proj.dtype != torch.float32 or state.dtype != torch.float32 or (ring is not None and ring.dtype != torch.float32):
+        raise KernelError("rglru runs on 32-bit projections and states")
+    small = [w[k] for k in ("yb", "xb", "conv", "convb", "rab", "rib", "decay")]
+    if any(t.dtype != torch.float32 for t in small) or w["ra"].dtype != w["ri"].dtype or (ring is None and taps > 1):
+        raise KernelError("rglru: vectors are float32, both gates share a storage type, a convolution needs its ring")
+    _need_contig(proj, ring, state, out, w["ra"], w["ri"], *small)
+    T = proj.shape[0]
+    head = [c_void_p(_ptr(proj)), proj.shape[1], c_void_p(_ptr(w["yb"])), c_void_p(_ptr(w["xb"])), c_void_p(_ptr(w["conv"])),
+            c_void_p(_ptr(w["convb"])), c_void_p(_ptr(w["ra"])), c_void_p(_ptr(w["ri"])), dt_code(w["ra"]),
+            c_void_p(_ptr(w["rab"])), c_void_p(_ptr(w["rib"])), c_void_p(_ptr(w["decay"])), c_void_p(_ptr(ring)),
+            c_void_p(_ptr(state)), state.shape[0], c_void_p(_ptr(step.seq_start)), c_void_p(_ptr(step.seq_slot)),
+            c_void_p(_ptr(step.positions))]
+    if step.all_single:
+        _check("rglru", lib.sp_rglru_step(*head, c_void_p(_ptr(out)), dt_code(out), step.n_seqs, int(width), int(taps), int(parts),
+                                          c_float(mult), c_void_p(_stream())))
+        return
+    global launches
+    launches += 2
+    n_chunks = query_tiles(step.host["new_counts"], int(lib.sp_rglru_chunk_tokens()))
+    av = torch.empty(T, width, 2, dtype=torch.float32, device=proj.device)
+    cells = torch.empty(n_chunks, width, 2, dtype=torch.float32, device=proj.device)
+    _check("rglru", lib.sp_rglru_chunked(
+        *head, c_void_p(_ptr(av)), c_void_p(_ptr(cells)), n_chunks, c_void_p(_ptr(out)), dt_code(out), T, step.n_seqs, int(width),
+        int(taps), int(parts), c_float(mult), int(out.dtype == torch.bfloat16), c_void_p(_stream())))

@@ -10,7 +10,8 @@
 //                       q out, k and v into their page rows, the gates out as 32-bit numbers
 //   latent_rot_store    a projected row [q (per head: plain | rotated part) | low-rank row | shared key part | gates]:
 //                       RMS norm of the low-rank row, rotation of the shared key part and of the queries' rotated
-//                       parts, [normed row | rotated key part] into ONE page row, q and the gates out
+//                       parts (neighbouring dims or dims half the part apart form a pair), [normed row | rotated key
+//                       part] into ONE page row, q and the gates out
 //   gelu_gather_mul     out[t, j] = gelu_tanh(z[t, j]) · S[id_t, off + j]
 //
 // Norm statistics, angles (position · frequency, cosf / sinf), gates and sums are 32-bit; stores round to the
@@ -304,7 +305,7 @@ struct LatentRotArgs {
     float* gates;                        // [T][H]
     const float* freq;                   // [rd/2]
     RowPlace pl;
-    int T, H, d, rd, rank;
+    int T, H, d, rd, rank, halves;       // halves: dim i pairs with dim i + rd/2, else dim 2i with dim 2i + 1
     float rot_mult, eps;
 };
 
@@ -321,6 +322,7 @@ __global__ void __launch_bounds__(256) latent_rot_store_kernel(LatentRotArgs a) 
     __syncthreads();
     const float* src = a.proj + (size_t)t * a.ld;
     const int qd = a.d + a.rd, nq = a.H * qd;
+    const int first = a.halves ? 1 : 2, apart = a.halves ? half : 1;      // pair i: dims first·i and first·i + apart
     // queries: the plain part passes, the rotated part turns pair by pair
     for (int e = threadIdx.x; e < a.H * a.d; e += blockDim.x) {
         const int h = e / a.d, i = e - h * a.d;
@@ -328,10 +330,10 @@ __global__ void __launch_bounds__(256) latent_rot_store_kernel(LatentRotArgs a) 
     }
     for (int e = threadIdx.x; e < a.H * half; e += blockDim.x) {
         const int h = e / half, i = e - h * half;
-        const int c = h * qd + a.d + 2 * i;
-        const float u = src[c], v = src[c + 1], co = cs[i], si = cs[half + i];
+        const int c = h * qd + a.d + first * i;
+        const float u = src[c], v = src[c + apart], co = cs[i], si = cs[half + i];
         sp_st_dt(a.q_out, a.q_dt, (size_t)t * nq + c, u * co - v * si);
-        sp_st_dt(a.q_out, a.q_dt, (size_t)t * nq + c + 1, v * co + u * si);
+        sp_st_dt(a.q_out, a.q_dt, (size_t)t * nq + c + apart, v * co + u * si);
     }
     int g0 = nq;
     if (a.pool) {
@@ -350,15 +352,16 @@ __global__ void __launch_bounds__(256) latent_rot_store_kernel(LatentRotArgs a) 
             if (a.rows) sp_st_dt(a.rows, a.q_dt, (size_t)t * R + i, c);
         }
         for (int i = threadIdx.x; i < half; i += blockDim.x) {
-            const float u = lat[a.rank + 2 * i], v = lat[a.rank + 2 * i + 1], co = cs[i], si = cs[half + i];
+            const int c = a.rank + first * i;
+            const float u = lat[c], v = lat[c + apart], co = cs[i], si = cs[half + i];
             const float ru = u * co - v * si, rv = v * co + u * si;
             if (place_ok) {
-                sp_st_dt(a.pool, a.c_dt, base + a.rank + 2 * i, ru);
-                sp_st_dt(a.pool, a.c_dt, base + a.rank + 2 * i + 1, rv);
+                sp_st_dt(a.pool, a.c_dt, base + c, ru);
+                sp_st_dt(a.pool, a.c_dt, base + c + apart, rv);
             }
             if (a.rows) {
-                sp_st_dt(a.rows, a.q_dt, (size_t)t * R + a.rank + 2 * i, ru);
-                sp_st_dt(a.rows, a.q_dt, (size_t)t * R + a.rank + 2 * i + 1, rv);
+                sp_st_dt(a.rows, a.q_dt, (size_t)t * R + c, ru);
+                sp_st_dt(a.rows, a.q_dt, (size_t)t * R + c + apart, rv);
             }
         }
         g0 += R;
@@ -370,7 +373,7 @@ __global__ void __launch_bounds__(256) latent_rot_store_kernel(LatentRotArgs a) 
 SP_API int sp_latent_rot_store(const float* proj, int ld, const void* wc, int w_dt, void* q_out, int q_dt, void* pool, int c_dt,
                                void* rows, float* gates, const float* freq, const int* token_seq, const int* positions,
                                const int* seq_row, const int* page_table, int max_pages, int page_size, int T, int H, int d,
-                               int rd, int rank, float rot_mult, float eps, cudaStream_t stream) {
+                               int rd, int rank, int halves, float rot_mult, float eps, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (H <= 0 || d <= 0 || rank <= 0 || rd < 0 || (rd & 1)) SP_FAIL("latent_rot_store: sizes %d heads x (%d + %d), rank %d", H, d, rd, rank);
     if (rd > 0 && !freq) SP_FAIL("latent_rot_store: a frequency table is needed");
@@ -378,7 +381,7 @@ SP_API int sp_latent_rot_store(const float* proj, int ld, const void* wc, int w_
     if (pool && !wc) SP_FAIL("latent_rot_store: the row's norm needs its weight");
     LatentRotArgs a{proj, ld, wc, w_dt, q_out, q_dt, pool, c_dt, rows, gates, freq,
                     RowPlace{token_seq, positions, seq_row, page_table, max_pages, page_size, sp_range_host},
-                    T, H, d, rd, rank, rot_mult, eps};
+                    T, H, d, rd, rank, halves, rot_mult, eps};
     const size_t smem = (size_t)(rd > 0 ? rd : 2) * sizeof(float);
     SP_CHECK_CALL("latent_rot_store", sp_launch_dependent(latent_rot_store_kernel, dim3(T), dim3(256), smem, stream, a));
     return 0;

@@ -175,11 +175,13 @@ __global__ void __launch_bounds__(192, 1)
 tc_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                void* __restrict__ C, int c_dt, int M, int N, int K, int ldc, int mode, int* status,
                const __grid_constant__ EpiArgs ep, const SpRange rg, const int* __restrict__ group, float glu_limit,
-               float glu_slope) {
+               float glu_slope, int act, float mult) {
     // ``group`` (single CTAs only): a grouped product. The rows of A lie sorted by group in tiles of 128 rows; entry
     // t of the table is the row of W at which the weights of row tile t's group begin (W stacks the groups' matrices,
     // N rows each), or -1 for a row tile that is not in use, which all three roles pass over alike. ``glu_slope``
     // non-zero: the gated epilogue is g·sigmoid(slope·g)·(u + 1) with g = min(gate, limit), u = clamp(up, ±limit).
+    // ``act`` (SP_ACT_*): the gate's activation otherwise, with ``mult`` on the outputs; SP_ACT_RELU2 squares the relu of
+    // a plain store.
     using L = SmemLayout<BN, STAGES, CG>;
     extern __shared__ uint8_t smem_raw[];
     __shared__ __align__(8) uint64_t bar_full[STAGES];
@@ -525,13 +527,17 @@ tc_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                             const float up = fminf(fmaxf(__uint_as_float(u[j]) * rstd, -glu_limit), glu_limit);
                             v[j] = (g / (1.0f + expf(-glu_slope * g))) * (up + 1.0f);
                         } else {
-                            v[j] = (g / (1.0f + expf(-g))) * (__uint_as_float(u[j]) * rstd);
+                            v[j] = sp_gated(g, __uint_as_float(u[j]) * rstd, act) * mult;
                         }
                     }
                 } else {
                     tc_ld_wait();
 #pragma unroll
                     for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]) * rstd;
+                    if (act == SP_ACT_RELU2) {
+#pragma unroll
+                        for (int j = 0; j < 32; ++j) v[j] = sp_relu2(v[j]);
+                    }
                 }
                 if (c0 + SPAN >= c_end) {            // all of this tile has left tensor memory: hand the buffer back
                     tc_fence_before();
@@ -587,7 +593,7 @@ __device__ __forceinline__ uint32_t part_addr(uint32_t part, int col, int row) {
 template <int BN, int STAGES>
 __global__ void __launch_bounds__(192, 1)
 tc_gemm_splitk_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
-                      void* __restrict__ C, int c_dt, int M, int N, int K, int ldc, int mode, int splits, int* status) {
+                      void* __restrict__ C, int c_dt, int M, int N, int K, int ldc, int mode, int splits, int* status, int act, float mult) {
     using L = SmemLayout<BN, STAGES>;
     static_assert(STAGES * L::STAGE_BYTES >= BM * BN * 4, "the partial tile must fit over the pipeline stages");
     extern __shared__ uint8_t smem_raw[];
@@ -714,10 +720,7 @@ tc_gemm_splitk_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_co
                     }
                 }
 #pragma unroll
-                for (int j = 0; j < 32; ++j) {
-                    const float g = v[j];
-                    v[j] = (g / (1.0f + expf(-g))) * b[j];
-                }
+                for (int j = 0; j < 32; ++j) v[j] = sp_gated(v[j], b[j], act) * mult;
                 if (grow < M) store_row32(C, c_dt, (size_t)grow * ldc + n0 / 2 + c0, n0 / 2 + c0, N / 2, v, false);
             } else if (grow < M) {
                 store_row32(C, c_dt, (size_t)grow * ldc + n0 + c0, n0 + c0, N, v, mode == MODE_ACCUMULATE);
@@ -796,7 +799,7 @@ int make_map(CUtensorMap* map, const void* ptr, int rows, int K, int ld, int box
 
 template <int BN, int STAGES>
 int launch(const CUtensorMap& ma, const CUtensorMap& mw, void* C, int c_dt, int M, int N, int K, int ldc, int mode,
-           int* status, cudaStream_t stream, const EpiArgs& ep) {
+           int* status, cudaStream_t stream, const EpiArgs& ep, int act, float mult) {
     using L = SmemLayout<BN, STAGES>;
     static SpPerDevice configured;
     if (!configured.done()) {
@@ -810,14 +813,14 @@ int launch(const CUtensorMap& ma, const CUtensorMap& mw, void* C, int c_dt, int 
     const int grid = (int)(tiles < sm_count ? tiles : sm_count);
     SP_CHECK_CALL("tc_gemm", sp_launch_dependent(tc_gemm_kernel<BN, STAGES>, dim3(grid), dim3(192), (size_t)L::TOTAL, stream, ma, mw,
                                                  C, c_dt, M, N, K, ldc, mode, status, ep, sp_range_host, (const int*)nullptr,
-                                                 0.0f, 0.0f));
+                                                 0.0f, 0.0f, act, mult));
     return 0;
 }
 
 // A grouped product (see the kernel's ``group``): every row tile takes its own group's weights
 template <int BN, int STAGES>
 int launch_grouped(const CUtensorMap& ma, const CUtensorMap& mw, void* C, int c_dt, int M, int N, int K, int ldc, int mode,
-                   int* status, cudaStream_t stream, const int* group, float limit, float slope) {
+                   int* status, cudaStream_t stream, const int* group, float limit, float slope, int act) {
     using L = SmemLayout<BN, STAGES>;
     static SpPerDevice configured;
     if (!configured.done()) {
@@ -833,14 +836,14 @@ int launch_grouped(const CUtensorMap& ma, const CUtensorMap& mw, void* C, int c_
     memset(&ep, 0, sizeof(ep));
     SP_CHECK_CALL("tc_gemm (grouped)", sp_launch_dependent(tc_gemm_kernel<BN, STAGES>, dim3(grid), dim3(192), (size_t)L::TOTAL, stream,
                                                            ma, mw, C, c_dt, M, N, K, ldc, mode, status, ep, sp_range_host, group,
-                                                           limit, slope));
+                                                           limit, slope, act, 1.0f));
     return 0;
 }
 
 // The same tiles by pairs of CTAs (tcgen05 cta_group::2): tiles of 256 rows, one pair per two SMs.
 template <int BN, int STAGES>
 int launch_pair(const CUtensorMap& ma, const CUtensorMap& mw_half, void* C, int c_dt, int M, int N, int K, int ldc, int mode,
-                int* status, cudaStream_t stream, const EpiArgs& ep) {
+                int* status, cudaStream_t stream, const EpiArgs& ep, int act, float mult) {
     using L = SmemLayout<BN, STAGES, 2>;
     static_assert(L::TOTAL <= 232448, "a CTA's shared memory");
     static SpPerDevice configured;
@@ -855,13 +858,13 @@ int launch_pair(const CUtensorMap& ma, const CUtensorMap& mw_half, void* C, int 
     const int pairs = (int)(tiles < sm_count / 2 ? tiles : sm_count / 2);
     SP_CHECK_CALL("tc_gemm", sp_launch_cluster(tc_gemm_kernel<BN, STAGES, 2>, dim3(2 * pairs), dim3(192), (size_t)L::TOTAL, stream,
                                                -2, ma, mw_half, C, c_dt, M, N, K, ldc, mode, status, ep, sp_range_host,
-                                               (const int*)nullptr, 0.0f, 0.0f));
+                                               (const int*)nullptr, 0.0f, 0.0f, act, mult));
     return 0;
 }
 
 template <int BN, int STAGES>
 int launch_splitk(const CUtensorMap& ma, const CUtensorMap& mw, void* C, int c_dt, int M, int N, int K, int ldc,
-                  int mode, int splits, int* status, cudaStream_t stream) {
+                  int mode, int splits, int* status, cudaStream_t stream, int act, float mult) {
     using L = SmemLayout<BN, STAGES>;
     static SpPerDevice configured;
     if (!configured.done()) {
@@ -872,7 +875,7 @@ int launch_splitk(const CUtensorMap& ma, const CUtensorMap& mw, void* C, int c_d
     const int n_tiles = ((N + BN - 1) / BN) * ((M + BM - 1) / BM);
     SP_CHECK_CALL("tc_gemm_splitk", sp_launch_cluster(tc_gemm_splitk_kernel<BN, STAGES>, dim3(n_tiles * splits), dim3(192),
                                                      (size_t)L::TOTAL, stream, splits, ma, mw, C, c_dt, M, N, K, ldc,
-                                                     mode, splits, status));
+                                                     mode, splits, status, act, mult));
     return 0;
 }
 
@@ -909,7 +912,8 @@ SP_API int sp_tc_gemm_supported(const void* A, const void* W, int K, int lda, in
 SP_API int sp_tc_gemm_n_tiles(int N, int bn) { return bn > 0 ? (N + bn - 1) / bn : 0; }
 
 static int tc_gemm_any(const void* A, const void* W, void* C, int c_dt, int M, int N, int K, int lda, int ldw, int ldc,
-                       int mode, int bn, const EpiArgs* epp, int* status, cudaStream_t stream);
+                       int mode, int bn, const EpiArgs* epp, int* status, cudaStream_t stream, int act = SP_ACT_SILU,
+                       float mult = 1.0f);
 
 // CTAs that would share a tile along K in sp_tc_gemm for these sizes (1: none): the host asks before it chooses
 // between a fused epilogue (never split) and the plain one followed by a small kernel.
@@ -932,29 +936,38 @@ SP_API int sp_tc_gemm(const void* A, const void* W, void* C, int c_dt, int M, in
     return tc_gemm_any(A, W, C, c_dt, M, N, K, lda, ldw, ldc, mode, bn, nullptr, status, stream);
 }
 
+// mode 2 with another activation of the gate (SP_ACT_*) and a factor on the outputs
+SP_API int sp_tc_gemm_gated(const void* A, const void* W, void* C, int c_dt, int M, int N, int K, int lda, int ldw, int ldc,
+                            int bn, int act, float mult, int* status, cudaStream_t stream) {
+    if (act != SP_ACT_SILU && act != SP_ACT_GELU) SP_FAIL("tc_gemm: activation code %d is not built for gated rows", act);
+    return tc_gemm_any(A, W, C, c_dt, M, N, K, lda, ldw, ldc, MODE_SILU_MUL, bn, nullptr, status, stream, act, mult);
+}
+
 // A grouped product on 128-row tiles of A (M a multiple of 128): row tile t multiplies with the N rows of W that begin
 // at row group[t] (W [w_rows, K] stacks the groups' matrices), or is passed over when group[t] < 0. mode 0: C [M, N];
 // mode 2: the groups' gate and up rows interleaved in blocks of bn/2, C [M, N/2] = the gated activation, clamped when
-// ``slope`` is non-zero. Nothing about the groups is known to the host.
+// ``slope`` is non-zero. ``act`` SP_ACT_RELU2 (mode 0): C is the square of the products' relu. Nothing about the groups
+// is known to the host.
 SP_API int sp_tc_gemm_grouped(const void* A, const void* W, void* C, int c_dt, int M, int N, int K, int lda, int ldw,
-                              int w_rows, int ldc, int mode, int bn, const int* group, float limit, float slope,
+                              int w_rows, int ldc, int mode, int bn, const int* group, float limit, float slope, int act,
                               int* status, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (sp_tc_gemm_supported(A, W, K, lda, ldw)) return 1;
     if (M % BM) SP_FAIL("tc_gemm (grouped): the rows (%d) come in tiles of %d", M, BM);
     if (mode != MODE_STORE && mode != MODE_SILU_MUL) SP_FAIL("tc_gemm (grouped): mode %d is not built", mode);
     if (bn != 128 && bn != 256) SP_FAIL("tc_gemm (grouped): tile width %d is not built (128 or 256)", bn);
-    if (N % bn) SP_FAIL("tc_gemm (grouped): a group's %d rows of W are no multiple of the tile width %d", N, bn);
+    if (act == SP_ACT_RELU2 && mode != MODE_STORE) SP_FAIL("tc_gemm (grouped): the squared relu belongs to the plain store");
+    if (mode == MODE_SILU_MUL && (N % bn)) SP_FAIL("tc_gemm (grouped): a group's %d rows of W are no multiple of the tile width %d", N, bn);
     if (!group) SP_FAIL("tc_gemm (grouped): the table of the row tiles' groups is missing");
     CUtensorMap ma, mw;
     if (make_map(&ma, A, M, K, lda, BM)) return 1;
     if (make_map(&mw, W, w_rows, K, ldw, bn)) return 1;
-    if (bn == 128) return launch_grouped<128, 6>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, group, limit, slope);
-    return launch_grouped<256, 4>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, group, limit, slope);
+    if (bn == 128) return launch_grouped<128, 6>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, group, limit, slope, act);
+    return launch_grouped<256, 4>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, group, limit, slope, act);
 }
 
 static int tc_gemm_any(const void* A, const void* W, void* C, int c_dt, int M, int N, int K, int lda, int ldw, int ldc,
-                       int mode, int bn, const EpiArgs* epp, int* status, cudaStream_t stream) {
+                       int mode, int bn, const EpiArgs* epp, int* status, cudaStream_t stream, int act, float mult) {
     EpiArgs ep;
     memset(&ep, 0, sizeof(ep));
     if (epp) ep = *epp;
@@ -982,17 +995,17 @@ static int tc_gemm_any(const void* A, const void* W, void* C, int c_dt, int M, i
     // a prompt's worth of rows: pairs of CTAs on tiles of 256 rows, each fetching half of the W tile
     if (pairs_from > 0 && M >= pairs_from) {
         if (make_map(&mw, W, N, K, ldw, bn / 2)) return 1;
-        if (bn == 128) return launch_pair<128, 8>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep);
-        if (bn == 192) return launch_pair<192, 7>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep);
-        return launch_pair<256, 6>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep);
+        if (bn == 128) return launch_pair<128, 8>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep, act, mult);
+        if (bn == 192) return launch_pair<192, 7>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep, act, mult);
+        return launch_pair<256, 6>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep, act, mult);
     }
     if (make_map(&mw, W, N, K, ldw, bn)) return 1;
     const int splits = fused ? 1 : pick_splits(M, N, K, bn);
     if (splits > 1) {
-        if (bn == 128) return launch_splitk<128, 6>(ma, mw, C, c_dt, M, N, K, ldc, mode, splits, status, stream);
-        return launch_splitk<256, 4>(ma, mw, C, c_dt, M, N, K, ldc, mode, splits, status, stream);
+        if (bn == 128) return launch_splitk<128, 6>(ma, mw, C, c_dt, M, N, K, ldc, mode, splits, status, stream, act, mult);
+        return launch_splitk<256, 4>(ma, mw, C, c_dt, M, N, K, ldc, mode, splits, status, stream, act, mult);
     }
-    if (bn == 128) return launch<128, 6>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep);
-    if (bn == 192) return launch<192, 5>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep);
-    return launch<256, 4>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep);
+    if (bn == 128) return launch<128, 6>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep, act, mult);
+    if (bn == 192) return launch<192, 5>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep, act, mult);
+    return launch<256, 4>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep, act, mult);
 }

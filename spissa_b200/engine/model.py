@@ -33,10 +33,12 @@ class Model:
                 raise ValueError(f"no block arrangement registered as {layer.block!r}; "
                                  f"known: {part_registry.known_parts('block')}") from None
             self.layers.append(cls(mixer=layer.mixer, ffn=layer.ffn, norms=layer.norms, **layer.params))
+        self.pass_rows = part_registry.build_part("embedding", spec.pass_rows) if spec.pass_rows is not None else None
         # a block that ends with a pass over the stream can write the first norm of the block that always follows it
         runs = [e.layer for e in spec.schedule]
         for a, b in zip(spec.schedule, spec.schedule[1:]):
-            if (runs.count(a.layer) == 1 and runs.count(b.layer) == 1 and not b.adds_embedding and spec.streams == 1
+            if (runs.count(a.layer) == 1 and runs.count(b.layer) == 1 and not b.adds_embedding and b.adds_row is None
+                    and spec.streams == 1
                     and hasattr(self.layers[a.layer], "feeds")):
                 self.layers[a.layer].feeds(self.layers[b.layer])
         self.final_norm = part_registry.build_part("norm", spec.final_norm)
@@ -77,7 +79,7 @@ class Model:
 
     # ------------------------------------------------------------------ weights
     def parts(self) -> list:
-        return [self.embedding] + self.layers + [self.final_norm, self.head]
+        return [self.embedding] + ([self.pass_rows] if self.pass_rows is not None else []) + self.layers + [self.final_norm, self.head]
 
     def weight_specs(self) -> list:
         out = []
@@ -156,7 +158,14 @@ class Model:
             for e in self.spec.schedule:
                 if e.adds_embedding:
                     K.add_inplace(h, h0)
-                self.layers[e.layer].forward(h, step, cache.view(e.cache, step, e.writes_cache))
+                layer, view = self.layers[e.layer], cache.view(e.cache, step, e.writes_cache)
+                if e.adds_row is None:
+                    layer.forward(h, step, view)
+                elif getattr(layer, "takes_row", False):
+                    layer.forward(h, step, view, row=self.pass_rows.row(e.adds_row))      # inside the layer's first norm
+                else:
+                    K.add_row(h, self.pass_rows.row(e.adds_row))
+                    layer.forward(h, step, view)
         if step.n_want == 0:
             if greedy:
                 return torch.empty(0, dtype=torch.int32, device=h.device)

@@ -38,9 +38,14 @@ class PreNormBlock(Block):
                  ffn_norm=self.ffn_norm.fused_fields(), ffn=self.ffn.fused_fields())
         return None if any(v is None for v in f.values()) else f
 
-    def forward(self, h, step, cache):
+    @property
+    def takes_row(self) -> bool:
+        return getattr(self.mixer_norm, "takes_row", False)
+
+    def forward(self, h, step, cache, row=None):
+        """``row`` (float32 [hidden], only where ``takes_row``): joins every row of the stream in front of the layer."""
         with phase("attention_norm_ms"):
-            x = self.mixer_norm.forward(h)
+            x = self.mixer_norm.forward(h) if row is None else self.mixer_norm.forward(h, add=row)
         self.mixer.forward(x, step, cache, h)
         if self.ffn is None:
             return

@@ -94,6 +94,29 @@ class PairEmbedding(TokenEmbedding):
         return out
 
 
+@register_part("embedding", "row_table")
+class RowTable(Part):
+    """Learned rows [rows, hidden] that are added to the whole stream at places of the layer schedule
+    (``ScheduleEntry.adds_row``), one row per pass of a group of layers that runs several times (not in the reference)."""
+    graph_safe = True
+
+    def __init__(self, rows: int, hidden_size: int, prefix: str = "", weight_name: str = "rows"):
+        super().__init__(prefix)
+        self.rows, self.hidden_size = int(rows), int(hidden_size)
+        self.weight_name = prefix + weight_name
+        self.table = None
+
+    def weight_specs(self):
+        return [WeightSpec(self.weight_name, (self.rows, self.hidden_size))]
+
+    def bind(self, tensors, rt):
+        super().bind(tensors, rt)
+        self.table = tensors[self.weight_name].float().contiguous()        # they join the 32-bit stream
+
+    def row(self, i: int) -> torch.Tensor:
+        return self.table[i]
+
+
 @register_part("head", "lm_head")
 class LMHead(Part):
     graph_safe = True

@@ -186,14 +186,17 @@ class LatentAttention(Mixer):
 
 @register_part("mixer", "rotary_latent_attention")
 class RotaryLatentAttention(Mixer):
-    """Attention through a cached low-rank row plus ONE rotated key part that all heads share, with a gate per head
-    (not in the reference).
+    """Attention through a cached low-rank row plus ONE rotated key part that all heads share, with a gate per head or
+    per element (not in the reference).
 
-        q_h = [q_h° (dim) | q_h^r (rot_dim)] = W_q,h x,   q_h^r rotated (neighbouring pairs, the position part's
-                                                           frequencies, cos and sin times its amplitude)
+        q_h = [q_h° (dim) | q_h^r (rot_dim)] = W_q,h x,   q_h^r rotated (the position part's pairs and frequencies, cos
+                                                           and sin times its amplitude)
         [c° | k^r] = D x,   c = n(c°) ⊙ w_c  (rank),   k^r (rot_dim) rotated the same way: what is cached, ONE page row
         score_h(i, j) = ((U_k,h c_j) · q_i,h° + k_j^r · q_i,h^r) · scale    over i − w < j <= i (``window`` w; None: all)
-        y += W_o · concat_h( sigmoid(w_g,h · x) · U_v,h Σ_j p_h(i, j) c_j )
+        y += W_o · concat_h( sigmoid(w_g,h · x) · U_v,h Σ_j p_h(i, j) c_j ) · out_scale
+
+    (``gate`` "head": one number per head; "element": W_g has a row for every entry of the concatenated heads and the gate
+    is an element-by-element product.)
 
     What is cached is never the expanded keys and values. A page row is r_j = [c_j | k_j^r]; with the per-head map
     E_h = [[U_k,hᵀ, 0], [0, I]] the score is (E_h q_i,h) · r_j, so the query is carried into the rows' space once per
@@ -206,16 +209,22 @@ class RotaryLatentAttention(Mixer):
     Three ways through it, chosen per step (bfloat16; the 32-bit mode takes the last): a step of 256 tokens or more in
     which every sequence starts at its first token expands the step's own rows into keys [U_k,h c | k^r] and values
     U_v,h c (two plain products over the rows) and runs on the tcgen05 prompt kernel, where that takes the sizes; other
-    steps of more than 64 tokens take both maps multiplied out into the products before and behind them; short steps
-    the small per-head products."""
+    steps of more than 64 tokens take both maps multiplied out into the products before and behind them (a gate per
+    element stands between the value map and W_o: only the map in front is multiplied out then); short steps the small
+    per-head products."""
     graph_safe = True
     kernel_modules = ("sandwich", "latent")
     kernel_modules_bf16 = ("attention",)
 
     def __init__(self, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int, v_head_dim: int, kv_rank: int,
                  scale: float, eps: float, position=None, window=None, cache_window=_UNSET, shares_latent: bool = False,
-                 prefix: str = "", names: dict | None = None):
+                 prefix: str = "", names: dict | None = None, gate: str = "head", out_scale: float = 1.0):
         super().__init__(prefix)
+        if gate not in ("head", "element"):
+            raise ValueError(f"{prefix}: a gate per 'head' or per 'element', not {gate!r}")
+        self.gate, self.out_scale = gate, float(out_scale)
+        if self.gate == "head" and self.out_scale != 1.0:
+            raise ValueError(f"{prefix}: an output factor goes with a gate per element")
         self.hidden_size, self.num_heads = int(hidden_size), int(num_heads)
         self.head_dim, self.rot_dim, self.v_head_dim, self.kv_rank = int(head_dim), int(rot_dim), int(v_head_dim), int(kv_rank)
         self.scale, self.eps = float(scale), float(eps)
@@ -229,9 +238,9 @@ class RotaryLatentAttention(Mixer):
         self.names = {k: prefix + v for k, v in n.items()}
         from .registry import build_part
         self.position = build_part("position", position) if position is not None else None
-        if self.rot_dim and (self.position is None or getattr(self.position, "pairing", "half") != "interleaved"
-                             or self.position.rotary_dim != self.rot_dim):
-            raise ValueError(f"{prefix}: the rotated part of {self.rot_dim} dims needs a rotary part of that size with pairing 'interleaved'")
+        if self.rot_dim and (self.position is None or self.position.rotary_dim != self.rot_dim):
+            raise ValueError(f"{prefix}: the rotated part of {self.rot_dim} dims needs a rotary part of that size")
+        self.halves = getattr(self.position, "pairing", "half") == "half"      # dim i pairs with dim i + rot_dim/2
         self.proj = self.o = self.wc_norm = self.q_map = self.v_map = None
 
     def children(self):
@@ -241,7 +250,7 @@ class RotaryLatentAttention(Mixer):
         W, H, d, rd, vd, r = self.hidden_size, self.num_heads, self.head_dim, self.rot_dim, self.v_head_dim, self.kv_rank
         n = self.names
         specs = [WeightSpec(n["q"], (H * (d + rd), W)), WeightSpec(n["uk"], (H * d, r)), WeightSpec(n["uv"], (H * vd, r)),
-                 WeightSpec(n["g"], (H, W)), WeightSpec(n["o"], (W, H * vd))]
+                 WeightSpec(n["g"], (H * vd if self.gate == "element" else H, W)), WeightSpec(n["o"], (W, H * vd))]
         if not self.shares_latent:
             specs += [WeightSpec(n["dkv"], (r + rd, W)), WeightSpec(n["dkv_norm"], (r,), init="ones")]
         return specs
@@ -281,10 +290,11 @@ class RotaryLatentAttention(Mixer):
             folded = torch.cat([torch.bmm(uk.float().view(H, d, r).transpose(1, 2), wq[:, :d]), wq[:, d:]], dim=1)
             stack[0] = folded.reshape(H * R, -1).to(torch.bfloat16)
             self.proj_fold = Linear(torch.cat(stack, dim=0))
-            wo = self.o.weight.float().view(-1, H, vd).permute(1, 0, 2)
-            fold = torch.zeros(H, wo.shape[1], R, dtype=torch.float32, device=wo.device)
-            fold[:, :, :r] = torch.bmm(wo, uv.float().view(H, vd, r))
-            self.o_fold = Linear(fold.permute(1, 0, 2).reshape(-1, H * R).to(torch.bfloat16))
+            if self.gate == "head":
+                wo = self.o.weight.float().view(-1, H, vd).permute(1, 0, 2)
+                fold = torch.zeros(H, wo.shape[1], R, dtype=torch.float32, device=wo.device)
+                fold[:, :, :r] = torch.bmm(wo, uv.float().view(H, vd, r))
+                self.o_fold = Linear(fold.permute(1, 0, 2).reshape(-1, H * R).to(torch.bfloat16))
         # whole prompts expand their own rows into keys [U_k,h c | k^r] and values U_v,h c per head and run on the
         # tcgen05 attention kernel where it takes the sizes: the maps as plain products over the rows (E_hᵀ and [U_v,h | 0])
         self.k_rows = self.v_rows = None
@@ -311,9 +321,9 @@ class RotaryLatentAttention(Mixer):
             proj = self.proj(x, out_dtype=torch.float32)            # norm and rotation read unrounded products
         with phase("latent_norm+rotary+append_ms"):
             q = torch.empty(T, H * (d + rd), dtype=act, device=dev)
-            gates = torch.empty(T, H, dtype=torch.float32, device=dev)
-            K.latent_rot_store(proj, self.wc_norm if writes else None, q, cache.k_pool if writes else None, cache, gates, freq,
-                               H, d, rd, r, amp, self.eps)
+            gates = self._gates(proj)
+            K.latent_rot_store(proj, self.wc_norm if writes else None, q, cache.k_pool if writes else None, cache, self._head_gates(gates), freq,
+                               H, d, rd, r, amp, self.eps, halves=self.halves)
         with phase("query_into_latent_space_ms"):
             qx = torch.empty(T, H * R, dtype=act, device=dev)
             K.headwise_product(q, self.q_map, qx, H, d + rd, R, w_rows_are_k=False)              # E_h q_h
@@ -323,9 +333,25 @@ class RotaryLatentAttention(Mixer):
             ctx = torch.empty(T, H * vd, dtype=act, device=dev)
             K.headwise_product(mix, self.v_map, ctx, H, R, vd, w_rows_are_k=False)               # U_v,h (Σ p c)
         with phase("head_gate_ms"):
-            K.scale_rows_sigmoid(ctx.view(T * H, vd), gates.view(T * H))
+            self._apply_gates(ctx, gates)
         with phase("o_projection+attention_residual_ms"):
             self.o(ctx, out=residual, accumulate=True)
+
+    def _gates(self, proj):
+        """The gates' arguments: a buffer that the storing kernel fills (per head), or the last columns of the projected
+        rows as they are (per element)."""
+        if self.gate == "head":
+            return torch.empty(proj.shape[0], self.num_heads, dtype=torch.float32, device=proj.device)
+        return proj[:, proj.shape[1] - self.num_heads * self.v_head_dim:]
+
+    def _head_gates(self, gates):
+        return gates if self.gate == "head" else None
+
+    def _apply_gates(self, ctx, gates):
+        if self.gate == "head":
+            K.scale_rows_sigmoid(ctx.view(-1, self.v_head_dim), gates.view(-1))
+        else:
+            K.gate_elements(ctx, gates, self.out_scale)
 
     def _attend_rows(self, qx, step, cache):
         """Σ_j p_h(i, j) [c_j | k_j^r] for queries in the rows' space: [T, heads·(rank + rot_dim)]."""
@@ -350,10 +376,10 @@ class RotaryLatentAttention(Mixer):
             proj = self.proj(x, out_dtype=torch.float32)
         with phase("latent_norm+rotary+append_ms"):
             q = torch.empty(T, H * (d + rd), dtype=act, device=dev)
-            gates = torch.empty(T, H, dtype=torch.float32, device=dev)
+            gates = self._gates(proj)
             rows = torch.empty(T, R, dtype=act, device=dev) if writes else None
-            K.latent_rot_store(proj, self.wc_norm if writes else None, q, cache.k_pool if writes else None, cache, gates, freq,
-                               H, d, rd, r, amp, self.eps, rows_out=rows)
+            K.latent_rot_store(proj, self.wc_norm if writes else None, q, cache.k_pool if writes else None, cache, self._head_gates(gates), freq,
+                               H, d, rd, r, amp, self.eps, rows_out=rows, halves=self.halves)
             if writes:
                 step.scratch[rows_key] = rows
         rows = step.scratch[rows_key]
@@ -364,12 +390,12 @@ class RotaryLatentAttention(Mixer):
             tiles = K.query_tiles(step.host["new_counts"], K.flash_tc_query_tile())
             K.flash_prefill_tc_rows(q, k, v, ctx, step, tiles, H, H, d + rd, self.window, self.scale, None, vd=vd)
         with phase("head_gate_ms"):
-            K.scale_rows_sigmoid(ctx.view(T * H, vd), gates.view(T * H))
+            self._apply_gates(ctx, gates)
         with phase("o_projection+attention_residual_ms"):
             self.o(ctx, out=residual, accumulate=True)
 
     def _forward_folded(self, x, step, cache, residual):
-        H, rd, r = self.num_heads, self.rot_dim, self.kv_rank
+        H, rd, r, vd = self.num_heads, self.rot_dim, self.kv_rank, self.v_head_dim
         T, dev, act, R = x.shape[0], x.device, self.rt.act_dtype, self.kv_rank + self.rot_dim
         writes = cache.writes
         if writes and self.shares_latent:
@@ -379,12 +405,21 @@ class RotaryLatentAttention(Mixer):
             proj = self.proj_fold(x, out_dtype=torch.float32)
         with phase("latent_norm+rotary+append_ms"):
             qx = torch.empty(T, H * R, dtype=act, device=dev)
-            gates = torch.empty(T, H, dtype=torch.float32, device=dev)
+            gates = self._gates(proj)
             # the unrotated part of a head's query is already in the rows' space: ``rank`` entries instead of ``dim``
-            K.latent_rot_store(proj, self.wc_norm if writes else None, qx, cache.k_pool if writes else None, cache, gates, freq,
-                               H, r, rd, r, amp, self.eps)
+            K.latent_rot_store(proj, self.wc_norm if writes else None, qx, cache.k_pool if writes else None, cache, self._head_gates(gates), freq,
+                               H, r, rd, r, amp, self.eps, halves=self.halves)
         with phase("latent_attention_ms"):
             mix = self._attend_rows(qx, step, cache)
+        if self.o_fold is None:
+            with phase("value_expansion_ms"):
+                ctx = torch.empty(T, H * vd, dtype=act, device=dev)
+                K.headwise_product(mix, self.v_map, ctx, H, R, vd, w_rows_are_k=False)
+            with phase("head_gate_ms"):
+                self._apply_gates(ctx, gates)
+            with phase("o_projection+attention_residual_ms"):
+                self.o(ctx, out=residual, accumulate=True)
+            return
         with phase("head_gate_ms"):
             K.scale_rows_sigmoid(mix.view(T * H, R), gates.view(T * H))
         with phase("o_projection+attention_residual_ms"):

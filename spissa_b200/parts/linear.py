@@ -71,15 +71,16 @@ class Linear:
 
 
 class GatedLinear:
-    """silu(x·Wgᵀ) ⊙ (x·Wuᵀ) as one product over the stacked weight.
+    """act(x·Wgᵀ) ⊙ (x·Wuᵀ) · mult as one product over the stacked weight (``act``: K.ACT_SILU or K.ACT_GELU).
 
     When the sizes allow, gate and up rows are interleaved in blocks (``block`` gate rows, then
     the ``block`` up rows of the same outputs) so that one tile of the tensor-core kernel holds
-    both halves and applies silu·up in its epilogue.
+    both halves and applies act·up in its epilogue.
     """
 
-    def __init__(self, gate: torch.Tensor, up: torch.Tensor):
+    def __init__(self, gate: torch.Tensor, up: torch.Tensor, act: int = K.ACT_SILU, mult: float = 1.0):
         I = gate.shape[0]
+        self.act, self.mult = act, float(mult)
         self.intermediate = I
         self.block = 128 if I % 128 == 0 else 64 if I % 64 == 0 else 0
         fused = self.block and gate.dtype == torch.bfloat16 and gate.shape[1] % 8 == 0
@@ -96,12 +97,12 @@ class GatedLinear:
     def __call__(self, x: torch.Tensor, act_dtype) -> torch.Tensor:
         out = torch.empty(x.shape[0], self.intermediate, dtype=act_dtype, device=x.device)
         if self.block and x.shape[0] <= GATED_GEMV_TOKENS and K.gemv_supported(x, self.weight):
-            K.gemv(x, self.weight, out, K.TC_SILU_MUL, self.block)
+            K.gemv(x, self.weight, out, K.TC_SILU_MUL, self.block, self.act, self.mult)
         elif self.block and x.shape[0] <= STREAM_TOKENS and K.tc_stream_supported(x, self.weight, K.TC_SILU_MUL, self.block):
-            K.tc_stream(x, self.weight, out, K.TC_SILU_MUL, self.block)
+            K.tc_stream(x, self.weight, out, K.TC_SILU_MUL, self.block, self.act, self.mult)
         elif self.block and K.tc_gemm_supported(x, self.weight):
-            K.tc_gemm(x, self.weight, out, K.TC_SILU_MUL, 2 * self.block)
+            K.tc_gemm(x, self.weight, out, K.TC_SILU_MUL, 2 * self.block, self.act, self.mult)
         else:
             gu = self.plain(x, out_dtype=act_dtype)
-            K.silu_mul(gu, out)
+            K.gated_mul(gu, out, self.act, self.mult)
         return out

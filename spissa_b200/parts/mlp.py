@@ -4,7 +4,8 @@ PolyNorm feed-forward: down( a·N(z) + b·N(z²) + c·N(z³) + e ) with z = x·W
 N(v) = v / sqrt(mean(v²) + eps) over a token's row; (a, b, c, e) is a learned tensor of four numbers (not in the
 reference). The activation runs in 32-bit on the unrounded product.
 
-SwiGLU feed-forward: down( silu(x·Wgᵀ) ⊙ (x·Wuᵀ) ), silu(z) = z / (1 + e^{-z}).
+SwiGLU feed-forward: down( silu(x·Wgᵀ) ⊙ (x·Wuᵀ) ), silu(z) = z / (1 + e^{-z}); GEGLU feed-forward: the same with the tanh
+form of gelu (not in the reference).
 
 GELU feed-forward: down( gelu(x·Wupᵀ) ) with the tanh form gelu(z) = ½ z (1 + tanh(√(2/π) (z + 0.044715 z³))) (not in
 the reference).
@@ -16,13 +17,17 @@ A SwiGLU may carry a gate of one number per token: the rows of silu(·) ⊙ (·)
 sigmoid(x · w_sgᵀ) before the down projection (which is linear, so its output is scaled by the same number).
 
 Routed experts: ``experts`` gated feed-forwards (``activation``: ``clamped_glu`` or ``swiglu``) of which each token uses
-``top``. The scores s are ``score`` of the router's 32-bit logits: ``sigmoid``, or ``softmax`` over all experts; the
-weights are s_k / (Σ s_k + 1e-20) · ``weight_scale``. A shared expert may be gated per token by sigmoid(x · w_sgᵀ)
+``top``; or experts without a gate, down( relu(x·Wupᵀ)² ) (``activation`` ``relu2``). ``identity``: so many of the router's
+outputs, the last ones, name experts without tensors whose output is the input itself. The scores s are ``score`` of the router's 32-bit logits: ``sigmoid``, or ``softmax`` over all experts; the
+weights are s_k / (Σ s_k + 1e-20) · ``weight_scale`` (``normalize`` False: s_k · ``weight_scale``). A shared expert may be gated per token by sigmoid(x · w_sgᵀ)
 (``shared_gate`` names the row w_sg; it rides in the router's product). With the sigmoid score: s = sigmoid(x·Wrᵀ) in 32-bit;
 the choice reads s + correction, the weights read s: the experts form ``groups`` equal groups of neighbours, a group's
 score is the sum of its two largest choice scores, only experts of the ``keep_groups`` best groups can be chosen, the
 ``top`` largest choice scores among them are; weight_k = s_k / (Σ s_k + 1e-20); y += Σ_k weight_k · expert_k(x), plus a
 shared expert that every token uses (not in the reference).
+
+``out_scale`` (gated feed-forwards; routed experts have ``weight_scale``): a factor on the part's output, applied to the
+32-bit activation in front of the (linear) down projection: how a block scales its sublayers into the stream at no cost.
 
 crates/spissa-runtime/src/models/llama/generate.rs:590-637 (gate, up), :642-763 (down);
 crates/spissa-runtime/src/ops.rs:192-194 (silu). Gate and up run as one matrix product
@@ -42,10 +47,13 @@ from ..phases import phase
 @register_part("ffn", "swiglu")
 class SwiGLU(FeedForward):
     graph_safe = True
+    act = K.ACT_SILU
 
-    def __init__(self, hidden_size: int, intermediate_size: int, prefix: str = "", names: dict | None = None):
+    def __init__(self, hidden_size: int, intermediate_size: int, prefix: str = "", names: dict | None = None,
+                 out_scale: float = 1.0):
         super().__init__(prefix)
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
+        self.out_scale = float(out_scale)
         n = dict(gate="gate_proj.weight", up="up_proj.weight", down="down_proj.weight")
         n.update(names or {})
         self.names = {k: prefix + v for k, v in n.items()}
@@ -61,12 +69,12 @@ class SwiGLU(FeedForward):
         g, u = tensors[self.names["gate"]], tensors[self.names["up"]]
         if g.dtype != u.dtype:
             raise ValueError(f"{self.prefix}: gate and up projections must share a storage type")
-        self.gate_up = GatedLinear(g, u)
+        self.gate_up = GatedLinear(g, u, self.act, self.out_scale)
         self.down = Linear(tensors[self.names["down"]])
 
     def fused_fields(self):
         gu = self.gate_up
-        if gu is None or not gu.block or gu.weight.dtype != torch.bfloat16 or self.down.weight.dtype != torch.bfloat16:
+        if self.act != K.ACT_SILU or self.out_scale != 1.0 or gu is None or not gu.block or gu.weight.dtype != torch.bfloat16 or self.down.weight.dtype != torch.bfloat16:
             return None
         return dict(kind="swiglu", gate_up=gu.weight, pair=gu.block, down=self.down.weight,
                     hidden_size=self.hidden_size, intermediate_size=self.intermediate_size)
@@ -81,6 +89,12 @@ class SwiGLU(FeedForward):
                 K.scale_rows_sigmoid(act, row_gate)
         with phase("down_projection+mlp_residual_ms"):
             self.down(act, out=residual, accumulate=True)
+
+
+@register_part("ffn", "geglu")
+class GeGLU(SwiGLU):
+    """The gated feed-forward with the tanh form of gelu on the gate."""
+    act = K.ACT_GELU
 
 
 @register_part("ffn", "polynorm")
@@ -195,12 +209,16 @@ class RoutedExperts(FeedForward):
     def __init__(self, hidden_size: int, intermediate_size: int, experts: int, top: int, limit: float = 0.0,
                  slope: float = 1.702, groups: int = 1, keep_groups: int = 1, shared=None, prefix: str = "",
                  names: dict | None = None, activation: str = "clamped_glu", score: str = "sigmoid",
-                 weight_scale: float = 1.0, correction: bool = True, shared_gate: str | None = None):
+                 weight_scale: float = 1.0, correction: bool = True, shared_gate: str | None = None,
+                 identity: int = 0, normalize: bool = True):
         super().__init__(prefix)
-        if activation not in ("clamped_glu", "swiglu") or score not in ("sigmoid", "softmax"):
+        if activation not in ("clamped_glu", "swiglu", "relu2") or score not in ("sigmoid", "softmax"):
             raise ValueError(f"{prefix}: unknown activation {activation!r} or score {score!r}")
         self.activation, self.score, self.weight_scale = activation, score, float(weight_scale)
         self.has_correction = bool(correction)
+        self.identity, self.normalize = int(identity), bool(normalize)
+        if self.identity < 0 or (self.identity and int(groups or 1) > 1):
+            raise ValueError(f"{prefix}: identity experts stand outside groups")
         self.shared_gate = shared_gate           # name (behind the prefix) of a row [1, hidden]: the shared expert's gate
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
         self.experts, self.top = int(experts), int(top)
@@ -209,7 +227,7 @@ class RoutedExperts(FeedForward):
         self.limit, self.slope = (float(limit), float(slope)) if activation == "clamped_glu" else (0.0, 0.0)
         if self.experts % self.groups:
             raise ValueError(f"{prefix}: {self.experts} experts do not form {self.groups} equal groups")
-        allowed = self.experts if self.groups == 1 else self.keep_groups * (self.experts // self.groups)
+        allowed = self.experts + self.identity if self.groups == 1 else self.keep_groups * (self.experts // self.groups)
         if not (1 <= self.top <= allowed):
             raise ValueError(f"{prefix}: {self.top} experts cannot be chosen among {allowed} allowed")
         n = dict(router="router", correction="correction", expert_prefix="e", gate="gate", up="up", down="down")
@@ -228,15 +246,19 @@ class RoutedExperts(FeedForward):
 
     def weight_specs(self):
         H, I = self.hidden_size, self.intermediate_size
-        specs = [WeightSpec(self.prefix + self.names["router"], (self.experts, H))]
+        outputs = self.experts + self.identity
+        specs = [WeightSpec(self.prefix + self.names["router"], (outputs, H))]
         if self.has_correction:
-            specs.append(WeightSpec(self.prefix + self.names["correction"], (self.experts,)))
+            specs.append(WeightSpec(self.prefix + self.names["correction"], (outputs,)))
         if self.shared_gate:
             specs.append(WeightSpec(self.prefix + self.shared_gate, (1, H)))
         for i in range(self.experts):
-            specs += [WeightSpec(self._expert(i, "gate"), (I, H)), WeightSpec(self._expert(i, "up"), (I, H)),
-                      WeightSpec(self._expert(i, "down"), (H, I))]
+            specs += [WeightSpec(self._expert(i, which), (I, H)) for which in self._up_names()]
+            specs.append(WeightSpec(self._expert(i, "down"), (H, I)))
         return specs
+
+    def _up_names(self):
+        return ("up",) if self.activation == "relu2" else ("gate", "up")
 
     def bind(self, tensors, rt):
         super().bind(tensors, rt)
@@ -249,13 +271,15 @@ class RoutedExperts(FeedForward):
         # kernels take, in blocks (``glu_block`` gate rows, then the up rows of the same outputs), so that one tile of a
         # product holds both halves and applies the activation in its epilogue
         H, I = self.hidden_size, self.intermediate_size
-        gate0 = tensors[self._expert(0, "gate")]
+        gate0 = tensors[self._expert(0, self._up_names()[0])]
         self.glu_block = 0
-        if gate0.dtype == torch.bfloat16 and H % 8 == 0 and I % 64 == 0:
+        if self.activation != "relu2" and gate0.dtype == torch.bfloat16 and H % 8 == 0 and I % 64 == 0:
             self.glu_block = 128 if I % 128 == 0 else 64
         b = self.glu_block
 
         def gate_up(i):
+            if self.activation == "relu2":
+                return tensors[self._expert(i, "up")]
             g, u = tensors[self._expert(i, "gate")], tensors[self._expert(i, "up")]
             if not b:
                 return torch.cat([g, u], dim=0)
@@ -272,9 +296,11 @@ class RoutedExperts(FeedForward):
             wts = torch.empty(T, self.top, dtype=torch.float32, device=x.device)
             gate = torch.empty(T, dtype=torch.float32, device=x.device) if self.shared_gate else None
             K.moe_select(z, self.correction, ids, wts, self.top, self.groups, self.keep_groups,
-                         softmax=self.score == "softmax", weight_scale=self.weight_scale, experts=self.experts, extra=gate)
+                         softmax=self.score == "softmax", weight_scale=self.weight_scale, experts=self.experts + self.identity,
+                         extra=gate, normalize=self.normalize)
         with phase("experts_ms"):
-            K.moe_experts(x, ids, wts, self.w_gate_up, self.w_down, residual, self.top, self.limit, self.slope, self.glu_block)
+            K.moe_experts(x, ids, wts, self.w_gate_up, self.w_down, residual, self.top, self.limit, self.slope, self.glu_block,
+                          act=K.ACT_RELU2 if self.activation == "relu2" else K.ACT_SILU, identities=self.identity > 0)
         if self.shared is not None and self.shared_gate:
             self.shared.forward(x, step, residual, row_gate=gate)
         elif self.shared is not None:

@@ -24,12 +24,14 @@ from .registry import register_part
 class RMSNorm(Norm):
     graph_safe = True
 
-    def __init__(self, size: int, eps: float, prefix: str = "", weight_name: str = "weight", around_zero: bool = False):
+    def __init__(self, size: int, eps: float, prefix: str = "", weight_name: str = "weight", around_zero: bool = False,
+                 weight_scale: float = 1.0):
         super().__init__(prefix)
         self.size = int(size)
         self.eps = float(eps)
         self.weight_name = prefix + weight_name
         self.around_zero = bool(around_zero)   # the stored weight w lies around zero and 1 + w multiplies (not in the reference)
+        self.weight_scale = float(weight_scale)   # a factor on the output (the head behind a final norm is linear: scaled logits)
         self.weight = None
 
     def weight_specs(self):
@@ -40,6 +42,8 @@ class RMSNorm(Norm):
         self.weight = tensors[self.weight_name].contiguous()
         if self.around_zero:
             self.weight = (1.0 + self.weight.float()).contiguous()     # 32-bit: 1 + w rounded to 16 bits would lose w
+        if self.weight_scale != 1.0:
+            self.weight = (self.weight.float() * self.weight_scale).contiguous()
 
     def multiplier(self) -> torch.Tensor:
         """The weight as it multiplies, float32 [size] (for a kernel that applies this norm inside another pass)."""
@@ -55,10 +59,13 @@ class RMSNorm(Norm):
             return None
         return dict(kind="rmsnorm", weight=self.weight, eps=self.eps, size=self.size)
 
-    def forward(self, h: torch.Tensor, rows: torch.Tensor | None = None) -> torch.Tensor:
+    takes_row = True
+
+    def forward(self, h: torch.Tensor, rows: torch.Tensor | None = None, add: torch.Tensor | None = None) -> torch.Tensor:
+        """``add`` (float32 [size]): a row that joins every row of the stream first, in the same pass."""
         n = h.shape[0] if rows is None else rows.shape[0]
         out = torch.empty(n, self.size, dtype=self.rt.act_dtype, device=h.device)
-        K.rmsnorm(h, self.weight, out, self.eps, rows)
+        K.rmsnorm(h, self.weight, out, self.eps, rows, add)
         return out
 
 

@@ -15,6 +15,14 @@ Gated linear attention: linear attention whose state decays per key channel by a
     S_t = diag(α_t) S_{t-1} + k_t v_tᵀ,   o_t = S_tᵀ q_t,   ô_t = o_t / sqrt(mean(o_t²) + eps) ⊙ w  (w [vdim], shared by heads);
     y_t = Wo · ( concat_h(ô_t) ⊙ silu(g_t) ) · out_scale.
 
+RG-LRU block (Griffin's recurrent block): a real-gated linear recurrent unit behind a short causal convolution, times a
+gelu branch, both of size ``width``:
+    y_t = gelu(Wy x_t + by),  u_t = conv(Wx x_t + bx)  (per channel, ``taps`` taps, bias; the inputs before the start are 0);
+    u is cut into ``parts`` equal parts with square gate matrices:  r = sigmoid(Ra u + ρ),  i = sigmoid(Ri u + ι);
+    log a_t = −decay_factor · r ⊙ softplus(λ),  S_t = a_t ⊙ S_{t-1} + sqrt(1 − a_t²) ⊙ i ⊙ u_t  (S₀ = 0);
+    y += Wo (S_t ⊙ y_t) · out_scale.
+The convolution's last inputs are a second state, a ring of ``taps`` rows (row p mod taps holds position p's input).
+
 All states are 32-bit and belong to the sequence's slot; the recurrences run in 32-bit on the unrounded
 projections, which are one matrix product over the stacked weights.
 """
@@ -23,7 +31,7 @@ from __future__ import annotations
 import torch
 
 from ..csrc import lib as K
-from .base import Mixer, StateRequest, WeightSpec
+from .base import CacheBundle, Mixer, StateRequest, WeightSpec
 from .linear import Linear
 from .registry import register_part
 from ..phases import phase
@@ -162,5 +170,62 @@ class GatedLinearAttention(Mixer):
             y = torch.empty(x.shape[0], self.num_heads * self.vdim, dtype=self.rt.act_dtype, device=x.device)
             K.gla(p, cache.state, self.a2, self.a2b, self.norm, y, step, self.num_heads, self.dim, self.vdim, self.rank,
                   self.tau, self.eps, self.out_scale)
+        with phase("o_projection+mixer_residual_ms"):
+            self.o(y, out=residual, accumulate=True)
+
+
+@register_part("mixer", "rglru")
+class RGLRU(Mixer):
+    """``out_scale``: a factor on the mixer's output, applied to the 32-bit product S ⊙ y in front of the output projection."""
+    graph_safe = True
+    kernel_modules = ("rglru",)
+
+    def __init__(self, hidden_size: int, width: int, parts: int, taps: int, decay_factor: float = 8.0, out_scale: float = 1.0,
+                 prefix: str = "", names: dict | None = None):
+        super().__init__(prefix)
+        self.hidden_size, self.width, self.parts, self.taps = int(hidden_size), int(width), int(parts), int(taps)
+        self.decay_factor, self.out_scale = float(decay_factor), float(out_scale)
+        if self.parts < 1 or self.width % self.parts:
+            raise ValueError(f"{prefix}: a width of {self.width} is not {self.parts} equal parts")
+        if self.taps < 1:
+            raise ValueError(f"{prefix}: the convolution needs at least one tap")
+        n = dict(y="y", yb="y.b", x="x", xb="x.b", conv="conv", convb="conv.b", ra="ra", rab="ra.b", ri="ri", rib="ri.b",
+                 lam="lam", o="o")
+        n.update(names or {})
+        self.names = {k: prefix + v for k, v in n.items()}
+        self.proj = self.o = self.w = None
+
+    def weight_specs(self):
+        H, W, P, s, n = self.hidden_size, self.width, self.parts, self.width // self.parts, self.names
+        return [WeightSpec(n["y"], (W, H)), WeightSpec(n["yb"], (W,)), WeightSpec(n["x"], (W, H)), WeightSpec(n["xb"], (W,)),
+                WeightSpec(n["conv"], (W, self.taps)), WeightSpec(n["convb"], (W,)),
+                WeightSpec(n["ra"], (P, s, s)), WeightSpec(n["rab"], (P, s)), WeightSpec(n["ri"], (P, s, s)),
+                WeightSpec(n["rib"], (P, s)), WeightSpec(n["lam"], (W,)), WeightSpec(n["o"], (H, W))]
+
+    def cache_request(self):
+        ring = StateRequest((self.taps, self.width), torch.float32) if self.taps > 1 else None
+        return CacheBundle.of(conv=ring, state=StateRequest((self.width,), torch.float32))
+
+    def bind(self, tensors, rt):
+        super().bind(tensors, rt)
+        n = self.names
+        if tensors[n["y"]].dtype != tensors[n["x"]].dtype:
+            raise ValueError(f"{self.prefix}: the projections of one input must share a storage type")
+        self.proj = Linear(torch.cat([tensors[n["y"]], tensors[n["x"]]], dim=0))
+        self.o = Linear(tensors[n["o"]])
+        small = {k: tensors[n[k]].float().reshape(-1).contiguous() for k in ("yb", "xb", "convb", "rab", "rib")}
+        # ln(1 + e^λ) in 64-bit, rounded once
+        decay = (self.decay_factor * torch.logaddexp(tensors[n["lam"]].double(), torch.zeros((), dtype=torch.float64, device=rt.device)))
+        self.w = dict(small, conv=tensors[n["conv"]].float().contiguous(), decay=decay.float().contiguous(),
+                      ra=tensors[n["ra"]].contiguous(), ri=tensors[n["ri"]].contiguous())
+
+    def forward(self, x, step, cache, residual):
+        with phase("mixer_projection_ms"):
+            p = self.proj(x, out_dtype=torch.float32)              # the recurrence reads unrounded products
+        with phase("rglru_ms"):
+            y = torch.empty(x.shape[0], self.width, dtype=self.rt.act_dtype, device=x.device)
+            ring = cache.get("conv")
+            K.rglru(p, self.w, ring.state if ring is not None else None, cache["state"].state, y, step, self.width, self.taps,
+                    self.parts, self.out_scale)
         with phase("o_projection+mixer_residual_ms"):
             self.o(y, out=residual, accumulate=True)
