@@ -6,6 +6,7 @@
     python bench.py --design gozatar [--design-sizes 1k,2k,4k]      (the Gozatar decoder likewise)
     python bench.py --design kugirax [--design-sizes 1k,2k,4k]      (the Kugirax decoder likewise)
     python bench.py --design fotulix [--design-sizes 1k,2k,4k]      (the Fotulix decoder beside Kugirax and Llama)
+    python bench.py --design luvavik [--design-sizes 1k,2k,4k]      (the Luvavik decoder beside Kugirax, Duzinex and Llama)
 
 Prints ONE JSON line. ``value`` is decoded tokens per second at batch 8 from prompts of
 about 2,048 tokens in a cache of 4,096 tokens per sequence, timed on the device with CUDA
@@ -318,6 +319,48 @@ def kugirax_config_like_fotulix(size: dict, fx: dict, window: int = DESIGN_WINDO
     return dict(architecture="Kugirax", vocab=DESIGN_VOCAB, width=W, norm=dict(eps=1e-6), logit_softcap=30.0, layers=layers)
 
 
+# --design luvavik: six layers, eight runs (layers 1 and 2 run twice): R dense, [L routed, R routed] x 2, R dense, L dense,
+# R routed, with R a recurrent block of the stream's width (parts of 256 channels, four taps) and L an attention through
+# cached rows (rank + 64 rotated dims shared by the heads, no window, a gate per element); dense feed-forwards of ``ff``,
+# routed ones with 32 squared-relu experts of ff/4 and 8 identity experts, 4 per token. Beside it the closest existing
+# designs at equal sizes: a Kugirax decoder of eight layers with its latent attention (rows of the same size, no window)
+# and its routed layers (32 gated experts of ff/4, 4 per token) at the same runs, the Duzinex decoder (for its minGRU,
+# the other recurrence with a state per channel) and Llama.
+LUVAVIK_SIZES = {
+    # (latent: heads, dim, rot_dim, vdim, kv_rank), Kugirax's attention (heads, kv heads, dim) and query rank
+    "1k": dict(lat=(8, 128, 64, 128, 192), att=(8, 2, 128), q_rank=512),
+    "2k": dict(lat=(16, 128, 64, 128, 192), att=(16, 4, 128), q_rank=768),
+    "4k": dict(lat=(32, 128, 64, 128, 448), att=(32, 8, 128), q_rank=1536),
+}
+LUVAVIK_RUNS = (("R", False), ("L", True), ("R", True), ("L", True), ("R", True), ("R", False), ("L", False), ("R", True))
+LUVAVIK_PART, LUVAVIK_TAPS, LUVAVIK_EXPERTS, LUVAVIK_IDENTITY, LUVAVIK_TOP = 256, 4, 32, 8, 4
+
+
+def luvavik_config(size: dict, lv: dict) -> dict:
+    W, ff = size["width"], size["ff"]
+    lh, ld, lrd, lvd, r = lv["lat"]
+    mixers = dict(R=("rglru", dict(width=W, blocks=W // LUVAVIK_PART, conv=LUVAVIK_TAPS)),
+                  L=("latent_attention", dict(heads=lh, dim=ld, rot_dim=lrd, vdim=lvd, kv_rank=r, scale=(ld + lrd) ** -0.5,
+                                              rot=dict(dims=lrd, base=10000.0))))
+    moe = dict(kind="moe", expert=dict(ff=ff // 4),
+               router=dict(experts=LUVAVIK_EXPERTS, identity=LUVAVIK_IDENTITY, top=LUVAVIK_TOP))
+    layers = [dict(type=mixers[m][0], mixer=mixers[m][1], mlp=moe if routed else dict(kind="dense", ff=ff))
+              for m, routed in LUVAVIK_RUNS[:3] + LUVAVIK_RUNS[5:]]
+    return dict(architecture="Luvavik", vocab=DESIGN_VOCAB, width=W, norm=dict(eps=1e-6), residual_mult=0.9, logit_scale=1.25,
+                loop=dict(start=1, stop=3, times=2), layers=layers)
+
+
+def kugirax_config_like_luvavik(size: dict, lv: dict) -> dict:
+    W, ff = size["width"], size["ff"]
+    h, g, d = lv["att"]
+    lh, ld, lrd, lvd, r = lv["lat"]
+    mixers = dict(R=("attention", dict(heads=h, kv_heads=g, dim=d, vdim=d, conv=LUVAVIK_TAPS, scale=d ** -0.5, rot=dict(dims=d, base=10000.0))),
+                  L=("latent_attention", dict(heads=lh, dim=ld, vdim=lvd, q_rank=lv["q_rank"], kv_rank=r + lrd, scale=ld ** -0.5)))
+    moe = dict(kind="moe", expert=dict(ff=ff // 4), router=dict(experts=LUVAVIK_EXPERTS, top=LUVAVIK_TOP, scale=1.5))
+    layers = [dict(type=mixers[m][0], mixer=mixers[m][1], mlp=moe if routed else dict(kind="dense", ff=ff)) for m, routed in LUVAVIK_RUNS]
+    return dict(architecture="Kugirax", vocab=DESIGN_VOCAB, width=W, norm=dict(eps=1e-6), logit_softcap=30.0, layers=layers)
+
+
 def design_compare(args) -> int:
     """Prefill (one 2,048-token prompt) and decode (batch 8 behind such prompts) of the Duzinex decoder and of the
     Llama decoder with the same width, feed-forward size and number of layer runs; per-phase device times of both
@@ -337,13 +380,17 @@ def design_compare(args) -> int:
     for name in names:
         size = DESIGN_SIZES[name]
         dz = (duzinex_config(size) if design == "duzinex" else gozatar_config(size, GOZATAR_SIZES[name]) if design == "gozatar"
-              else kugirax_config(size, KUGIRAX_SIZES[name]) if design == "kugirax" else fotulix_config(size, FOTULIX_SIZES[name]))
+              else kugirax_config(size, KUGIRAX_SIZES[name]) if design == "kugirax"
+              else fotulix_config(size, FOTULIX_SIZES[name]) if design == "fotulix" else luvavik_config(size, LUVAVIK_SIZES[name]))
         runs = len(config_from_dict(dz).to_spec().schedule)
         row = {}
         arms = [(design, dz), ("llama", llama_config_like(size, runs))]
         if design == "fotulix":
             arms.insert(1, ("kugirax", kugirax_config_like_fotulix(size, FOTULIX_SIZES[name])))
             out["beside"] = "kugirax, llama"
+        if design == "luvavik":
+            arms[1:1] = [("kugirax", kugirax_config_like_luvavik(size, LUVAVIK_SIZES[name])), ("duzinex", duzinex_config(size))]
+            out["beside"] = "kugirax, duzinex, llama"
         for label, cfg_dict in arms:
             cfg = config_from_dict(cfg_dict)
             engine = Engine.from_config(cfg, seed=0, dtype=args.dtype, max_tokens=B * (T + 128), max_seqs=B, device="cuda:0")
@@ -418,7 +465,8 @@ def design_compare(args) -> int:
         row["rooflines"] = (design_rooflines(size, row, T, B, peaks, eb) if design == "duzinex"
                             else gozatar_rooflines(size, GOZATAR_SIZES[name], row, T, peaks, eb) if design == "gozatar"
                             else kugirax_rooflines(size, KUGIRAX_SIZES[name], row, T, peaks, eb) if design == "kugirax"
-                            else fotulix_rooflines(size, FOTULIX_SIZES[name], row, T, B, peaks, eb))
+                            else fotulix_rooflines(size, FOTULIX_SIZES[name], row, T, B, peaks, eb) if design == "fotulix"
+                            else luvavik_rooflines(size, LUVAVIK_SIZES[name], row, T, B, peaks, eb))
         out["sizes"][name] = row
     print(json.dumps(out))
     return 0
@@ -623,6 +671,59 @@ def fotulix_rooflines(size, fx, row, T, B, peaks, eb) -> dict:
     return out
 
 
+def luvavik_rooflines(size, lv, row, T, B, peaks, eb) -> dict:
+    """The same for the Luvavik decoder's kernel groups of a prompt step (sums over its eight runs), beside the like groups
+    of the Kugirax decoder at equal sizes, of the Duzinex decoder's minGRU and of Llama."""
+    W, ff = size["width"], size["ff"]
+    lh, ld, lrd, lvd, r = lv["lat"]
+    h, g, d = lv["att"]
+    lz, kz, dz, ll = (row[k]["prefill_phases_ms"] for k in ("luvavik", "kugirax", "duzinex", "llama"))
+    tf, bw = peaks["bf16_tflops"] * 1e12, peaks["hbm_gbs"] * 1e9
+    n_rec = sum(m == "R" for m, _ in LUVAVIK_RUNS)
+    n_lat, n_moe = len(LUVAVIK_RUNS) - n_rec, sum(routed for _, routed in LUVAVIK_RUNS)
+    n_dense = len(LUVAVIK_RUNS) - n_moe
+    causal, R = T * (T + 1) / 2, r + lrd
+    frac = lambda work, peak, ms: round(work / (ms * 1e-3) / peak, 4) if ms else None
+    out = {}
+
+    def put(label, ms, work, peak):
+        out[label] = dict(ms=ms, frac=frac(work, peak, ms))
+    # what a recurrence has to move: its 32-bit projected rows in, its output out; the gate products come on top
+    put("rglru (hbm)", lz.get("rglru_ms"), n_rec * T * W * (2 * 4.0 + eb), bw)
+    put("rglru gate products (tensor)", lz.get("rglru_ms"), n_rec * T * W * LUVAVIK_PART * 2 * 2.0, tf)
+    put("duzinex mingru (hbm)", dz.get("mingru_ms"), 4 * T * W * (3 * 4.0 + eb), bw)
+    lat_ms = (lz.get("latent_attention_ms") or 0) + (lz.get("key_value_expansion_ms") or 0)
+    put("latent attention (tensor)", lat_ms, n_lat * 2.0 * causal * (ld + lrd + lvd) * lh, tf)
+    k_lat = (kz.get("latent_attention_ms") or 0) + (kz.get("key_value_expansion_ms") or 0)
+    put("kugirax latent attention (tensor)", k_lat, n_lat * 2.0 * causal * (ld + lvd) * lh, tf)
+    q_w = lh * (ld + lrd)
+    put("row norm+rotation+store (hbm)", lz.get("latent_norm+rotary+append_ms"), n_lat * T * (q_w + R) * (4.0 + eb), bw)
+    put("kugirax latent norms+append (hbm)", kz.get("latent_norm+append_ms"), n_lat * T * (lv["q_rank"] + R) * (4.0 + eb), bw)
+    put("element gates (hbm)", lz.get("head_gate_ms"), n_lat * T * lh * lvd * (2 * eb + 4.0), bw)
+    share = LUVAVIK_EXPERTS / (LUVAVIK_EXPERTS + LUVAVIK_IDENTITY)         # of a token's choices that have products
+    put("experts, no gate (tensor)", lz.get("experts_ms"), n_moe * T * LUVAVIK_TOP * share * 2 * 2.0 * W * (ff // 4), tf)
+    put("kugirax experts (tensor)", kz.get("experts_ms"), n_moe * T * LUVAVIK_TOP * 3 * 2.0 * W * (ff // 4), tf)
+    for label, phases, runs in (("feed-forward", lz, n_dense), ("kugirax feed-forward", kz, n_dense), ("llama feed-forward", ll, row["llama"]["layer_runs"])):
+        ms = sum(v for k, v in phases.items() if "gate_projection" in k or "down_projection" in k)
+        put(label + " (tensor)", ms, runs * T * 3 * 2.0 * W * ff, tf)
+    put("norms (hbm)", (lz.get("attention_norm_ms") or 0) + (lz.get("mlp_norm_ms") or 0), 2 * len(LUVAVIK_RUNS) * T * W * (4.0 + eb), bw)
+    put("kugirax norm (hbm)", kz.get("input_norm_ms"), len(LUVAVIK_RUNS) * T * W * (4.0 + eb), bw)
+    put("router (hbm)", lz.get("router_ms"), n_moe * T * W * eb, bw)
+    put("kugirax router (hbm)", kz.get("router_ms"), n_moe * T * W * eb, bw)
+    # a decode step: every weight outside the experts once, of the experts what B tokens' choices touch at most, the cached rows
+    touched = lambda of: 1.0 - (1.0 - LUVAVIK_TOP / of) ** B
+    n_exp = lambda mats, of: n_moe * LUVAVIK_EXPERTS * touched(of) * mats * W * (ff // 4) * eb
+    runs_gb = row["luvavik"]["weight_gb"] * 1e9
+    put("luvavik decode step (hbm)", row["luvavik"]["decode_ms_per_step"],
+        runs_gb + n_exp(2, LUVAVIK_EXPERTS + LUVAVIK_IDENTITY) + n_lat * B * T * R * eb, bw)
+    put("kugirax decode step (hbm)", row["kugirax"]["decode_ms_per_step"],
+        row["kugirax"]["weight_gb"] * 1e9 + n_exp(3, LUVAVIK_EXPERTS) + n_lat * B * T * R * eb + n_rec * B * T * 2 * g * d * eb, bw)
+    nh, nkv, hd = size["llama"]
+    put("llama decode step (hbm)", row["llama"]["decode_ms_per_step"],
+        row["llama"]["weight_gb"] * 1e9 + B * T * row["llama"]["layer_runs"] * 2 * nkv * hd * eb, bw)
+    return out
+
+
 def kernel_case(name: str, reps: int) -> int:
     """One kernel of the step alone, at the 1B shape, on rotating buffers larger than L2.
 
@@ -659,12 +760,13 @@ def kernel_case(name: str, reps: int) -> int:
         torch.cuda.synchronize()
         print(json.dumps({"kernel_case": name, "launches": K.launches}))
         return 0
-    if name == "fotulix_step":
-        # the Fotulix decoder at the 2k size of --design: one prompt of 2,048 tokens, then three decode steps, kernel by
-        # kernel (no CUDA graph): the launch list of this run is what profiles/fotulix_step_and_kernels.md summarises
+    if name in ("fotulix_step", "luvavik_step"):
+        # the Fotulix / Luvavik decoder at the 2k size of --design: one prompt of 2,048 tokens, then three decode steps, kernel
+        # by kernel (no CUDA graph): the launch list of this run is what profiles/*_step_and_kernels.md summarises
         from spissa_b200 import Engine
         from spissa_b200.config import config_from_dict
-        cfg = config_from_dict(fotulix_config(DESIGN_SIZES["2k"], FOTULIX_SIZES["2k"]))
+        cfg = config_from_dict(fotulix_config(DESIGN_SIZES["2k"], FOTULIX_SIZES["2k"]) if name == "fotulix_step"
+                               else luvavik_config(DESIGN_SIZES["2k"], LUVAVIK_SIZES["2k"]))
         eng = Engine.from_config(cfg, seed=0, dtype="bfloat16", max_tokens=T + 128, max_seqs=1, use_graphs=False)
         rng = random.Random(0)
         sl = eng.acquire()
@@ -1140,6 +1242,48 @@ def kernel_case(name: str, reps: int) -> int:
             z = torch.randn(T * FH, device=dev)
             run = lambda i: K.scale_rows_sigmoid(xs[i % 12], z)
             bytes_ = T * FH * (Fd * 2 * 2.0 + 4.0)
+    elif name in ("rglru_chunks", "rglru_step", "gate_elements", "relu2_experts", "relu2_experts_b8"):
+        # the Luvavik kernels at the 2k size of --design (width 2,048 in parts of 256, four taps; 32 squared-relu experts of
+        # 2,048 and 8 identity experts, 4 per token; 16 heads of 128 values)
+        Wd, part, taps = 2048, LUVAVIK_PART, LUVAVIK_TAPS
+        B = 8 if name in ("rglru_step", "relu2_experts_b8") else 1
+        n_new = 1 if B > 1 else T
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+        step = SimpleNamespace(seq_start=i32([n_new * b for b in range(B + 1)]), seq_slot=i32(list(range(B))), n_seqs=B,
+                               positions=(torch.arange(n_new, dtype=torch.int32, device=dev) + (T if B > 1 else 0)).repeat(B),
+                               all_single=n_new == 1, max_new=n_new, host=dict(new_counts=[n_new] * B))
+        if name.startswith("rglru"):
+            n_buf = 64 if B > 1 else 6                           # a decode step's gate matrices are 2 MB: rotate them
+            v = lambda: torch.randn(Wd, device=dev)
+            ws = [dict(yb=v(), xb=v(), conv=torch.randn(Wd, taps, device=dev), convb=v(), rab=v(), rib=v(),
+                       decay=torch.rand(Wd, device=dev), ra=rnd(Wd // part, part, part), ri=rnd(Wd // part, part, part))
+                  for _ in range(n_buf)]
+            projs = [torch.randn(B * n_new, 2 * Wd, device=dev) for _ in range(n_buf)]
+            state, ring = torch.zeros(B, Wd, device=dev), torch.zeros(B, taps, Wd, device=dev)
+            out = torch.empty(B * n_new, Wd, dtype=bf, device=dev)
+            run = lambda i: K.rglru(projs[i % n_buf], ws[i % n_buf], ring, state, out, step, Wd, taps, Wd // part, 0.9)
+            bytes_ = B * n_new * Wd * (2 * 4 + 2.0)
+            if B > 1:
+                bytes_ += 2.0 * Wd * part * 2 + B * Wd * 4.0 * (2 + taps)
+        elif name == "gate_elements":
+            C, ld = 16 * 128, 16 * 192 + 256 + 16 * 128
+            xs, zs = [rnd(T, C) for _ in range(6)], [torch.randn(T, ld, device=dev) for _ in range(6)]
+            run = lambda i: K.gate_elements(xs[i % 6], zs[i % 6][:, ld - C:], 0.9)
+            bytes_ = T * C * (2 * 2 + 4.0)
+        else:
+            E, same, top, F = LUVAVIK_EXPERTS, LUVAVIK_IDENTITY, LUVAVIK_TOP, 2048
+            rows = B * n_new
+            n_buf = 4 if B > 1 else 1
+            ups, dns = [rnd(E, F, Wd) for _ in range(n_buf)], [rnd(E, Wd, F) for _ in range(n_buf)]
+            x = rnd(rows, Wd)
+            ids = torch.stack([torch.randperm(E + same, device=dev)[:top] for _ in range(rows)]).int().contiguous()
+            wts = torch.full((rows, top), 1.0 / top, device=dev)
+            y = torch.zeros(rows, Wd, device=dev)
+            run = lambda i: K.moe_experts(x, ids, wts, ups[i % n_buf], dns[i % n_buf], y, top, 0.0, 0.0, act=K.ACT_RELU2, identities=True)
+            if B > 1:
+                bytes_ = len({e for e in ids.flatten().tolist() if e < E}) * 2.0 * F * Wd * 2
+            else:
+                flops = int((ids < E).sum()) * 2 * 2.0 * Wd * F
     elif name in ("sample_b8", "sample_b64", "argmax_b8"):
         # the sampler on rows of 128,256 logits (standard deviation 4 after the temperature): temperature 0.8, top-p 0.95
         B = 64 if name.endswith("b64") else 8
@@ -1202,7 +1346,7 @@ def main() -> int:
     ap.add_argument("--kernel-case", default=None,
                     help="time one kernel alone (gemm_qkv|gemm_o|gemm_gate_up|gemm_down|gemv_qkv|gemv_o|gemv_gate_up|"
                          "gemv_down|gemv_head|diff_flash|diff_decode|retention_chunks|retention_step|mingru_chunks|polynorm|token_shift|gla_chunks|gla_step|moe_experts|moe_experts_b8|streams_norm|conv_qk_store|stream_qkv|stream_o|stream_gate_up|stream_down|stream_fused_qkv|stream_fused_o|stream_fused_gate_up|stream_fused_down|flash_prefill[_128]|flash_prefill_tc[_128]|flash_decode[_b64]|sample_b8|sample_b64|argmax_b8|decode_layers|step_b8|prefill|fused_qkv|fused_o|fused_gate_up|fused_down) instead of the step")
-    ap.add_argument("--design", default=None, choices=["duzinex", "gozatar", "kugirax", "fotulix"],
+    ap.add_argument("--design", default=None, choices=["duzinex", "gozatar", "kugirax", "fotulix", "luvavik"],
                     help="measure this design beside the Llama decoder at equal layer sizes instead of the headline workload")
     ap.add_argument("--design-sizes", default="", dest="design_sizes", help="which of 1k,2k,4k (default: all)")
     ap.add_argument("--reps", type=int, default=20)

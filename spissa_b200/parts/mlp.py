@@ -249,7 +249,9 @@ class RoutedExperts(FeedForward):
         outputs = self.experts + self.identity
         specs = [WeightSpec(self.prefix + self.names["router"], (outputs, H))]
         if self.has_correction:
-            specs.append(WeightSpec(self.prefix + self.names["correction"], (outputs,)))
+            # random weights: softmax scores are near 1 / outputs, a random correction of the usual size would choose alone
+            specs.append(WeightSpec(self.prefix + self.names["correction"], (outputs,),
+                                    init="const:0.0" if self.score == "softmax" else "normal"))
         if self.shared_gate:
             specs.append(WeightSpec(self.prefix + self.shared_gate, (1, H)))
         for i in range(self.experts):
