@@ -412,6 +412,11 @@ STATUS_TEXT = {101: "the TMA loader waited too long for a free pipeline stage",
                115: "attention: the softmax warps waited too long for the scores",
                116: "attention: the softmax warps waited too long for the previous block's output",
                117: "attention: the softmax warps waited too long for the last block's output",
+               141: "rglru: the MMA issuer waited too long for the gate matrices",
+               142: "rglru: the convolution warps waited too long for their buffer",
+               143: "rglru: the MMA issuer waited too long for a free accumulator",
+               144: "rglru: the MMA issuer waited too long for the convolution",
+               145: "rglru: the recurrence warps waited too long for the gates",
                301: "embedding: a token id outside the vocabulary",
                401: "range check: a page index from a page table lies beyond the pools",
                402: "range check: a sequence's row lies beyond the page table",
@@ -1512,10 +1517,15 @@ def rglru(proj, w: dict, ring, state, out, step, width, taps, parts, mult=1.0):
                                           c_float(mult), c_void_p(_stream())))
         return
     global launches
-    launches += 2
-    n_chunks = query_tiles(step.host["new_counts"], int(lib.sp_rglru_chunk_tokens()))
+    launches += 2                                          # chunks, their start states, outputs
+    tensor_cores = out.dtype == torch.bfloat16
+    counts = step.host["new_counts"]
+    n_chunks = query_tiles(counts, int(lib.sp_rglru_chunk_tokens(dt_code(w["ra"]), int(width) // int(parts), int(tensor_cores))))
+    n_blocks = query_tiles(counts, int(lib.sp_rglru_finish_tokens()))
     av = torch.empty(T, width, 2, dtype=torch.float32, device=proj.device)
     cells = torch.empty(n_chunks, width, 2, dtype=torch.float32, device=proj.device)
+    starts = torch.empty(n_chunks, width, dtype=torch.float32, device=proj.device)
     _check("rglru", lib.sp_rglru_chunked(
-        *head, c_void_p(_ptr(av)), c_void_p(_ptr(cells)), n_chunks, c_void_p(_ptr(out)), dt_code(out), T, step.n_seqs, int(width),
-        int(taps), int(parts), c_float(mult), int(out.dtype == torch.bfloat16), c_void_p(_stream())))
+        *head, c_void_p(_ptr(av)), c_void_p(_ptr(cells)), c_void_p(_ptr(starts)), n_chunks, n_blocks, c_void_p(_ptr(out)), dt_code(out), T,
+        step.n_seqs, int(width), int(taps), int(parts), c_float(mult), int(tensor_cores), c_void_p(_ptr(status_word(proj.device))),
+        c_void_p(_stream())))

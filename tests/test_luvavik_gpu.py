@@ -101,7 +101,8 @@ REC_CUTS = {
 }
 
 
-@pytest.mark.parametrize("W,parts,taps", [(64, 4, 4), (96, 1, 3), (50, 5, 1), (130, 2, 2), (256, 2, 4), (120, 5, 6), (320, 4, 5), (33, 1, 4)])
+@pytest.mark.parametrize("W,parts,taps", [(64, 4, 4), (96, 1, 3), (50, 5, 1), (130, 2, 2), (256, 2, 4), (120, 5, 6), (320, 4, 5), (33, 1, 4),
+                                          (256, 1, 4), (768, 3, 2), (384, 3, 4), (128, 1, 1)])
 @pytest.mark.parametrize("kind", ["float32", "bfloat16"])
 def test_recurrent_block_in_every_cut(W, parts, taps, kind):
     """Chunks of 64 tokens in parallel and one token at a time agree with the recurrence written out, from zero and from
