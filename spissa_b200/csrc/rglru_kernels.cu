@@ -194,54 +194,45 @@ __device__ __forceinline__ void rg_block_scan(const RgArgs& a, const RgPlace& pl
 // ---------------------------------------------------------------- u for the tensor-core kernels
 constexpr int RM_TOK = 8;                            // a thread makes u of two neighbouring channels for this many tokens
 
-// The inputs of a convolution of TAPS taps over RM_TOK tokens of channels c and c + 1, and its weights: asked for here, used
-// by RgConv2::make. ``c1_ok`` false: channel c stands in for c + 1; ``wide``: both channels' inputs in one access.
+// The inputs of a convolution of TAPS taps over RM_TOK tokens of channels c and c + 1 (c even, rows on 8-byte boundaries), asked
+// for by ``fetch`` and used by ``make``; rows at the end of the chunk stand in for those behind it.
 template <int TAPS>
 struct RgConv2 {
-    static constexpr int N = RM_TOK + (TAPS > 0 ? TAPS - 1 : 0);
+    static constexpr int BACK = TAPS > 0 ? TAPS - 1 : 0, N = RM_TOK + BACK;
     float2 x[N];
-    bool rows;                                       // every input is a row of the step (without its bias yet)
 
-    __device__ __forceinline__ void fetch(const RgArgs& a, const RgPlace& pl, int t, int t_end, int c, bool c1_ok, bool wide) {
+    __device__ __forceinline__ float2 load(const float* p) const { return __ldg((const float2*)p); }
+    __device__ __forceinline__ void fetch(const RgArgs& a, const RgPlace& pl, int t, int t_end, int c) {
         if constexpr (TAPS > 0) {
-            const int c1 = c1_ok ? c + 1 : c;
-            rows = t - (TAPS - 1) >= pl.first && t + RM_TOK <= t_end;
-            if (rows && wide) {
-                const float* x0 = a.proj + (size_t)(t - (TAPS - 1)) * a.ld + a.W + c;
+            const float* row = a.proj + (size_t)t * a.ld + a.W + c;
+            const int last = t_end - 1 - t;
 #pragma unroll
-                for (int i = 0; i < N; ++i) x[i] = __ldg((const float2*)(x0 + (size_t)i * a.ld));
-            } else if (rows) {
-                const float* x0 = a.proj + (size_t)(t - (TAPS - 1)) * a.ld + a.W;
+            for (int i = 0; i < RM_TOK; ++i) x[BACK + i] = load(row + (size_t)min(i, last) * a.ld);
 #pragma unroll
-                for (int i = 0; i < N; ++i) x[i] = make_float2(__ldg(x0 + (size_t)i * a.ld + c), __ldg(x0 + (size_t)i * a.ld + c1));
-            } else {
-                const float b0 = a.xb[c], b1 = a.xb[c1];
-#pragma unroll
-                for (int i = 0; i < N; ++i) {
-                    const int tt = min(t + i - (TAPS - 1), t_end - 1);
-                    x[i] = make_float2(rg_input(a, pl, tt, c, b0), rg_input(a, pl, tt, c1, b1));
-                }
+            for (int i = 0; i < BACK; ++i) {
+                const int tt = t - BACK + i, p = pl.pos0 + (tt - pl.first);
+                if (tt >= pl.first) x[i] = load(a.proj + (size_t)tt * a.ld + a.W + c);
+                else if (p >= 0) x[i] = load(a.ring + ((size_t)pl.slot * TAPS + p % TAPS) * a.W + c);
+                else x[i] = make_float2(0.0f, 0.0f);
             }
         }
     }
 
     // u of the tokens; tokens at t_end or beyond get 0
-    __device__ __forceinline__ void make(const RgArgs& a, const RgPlace& pl, int t, int t_end, int c, bool c1_ok, float2 (&u)[RM_TOK]) {
-        const int c1 = c1_ok ? c + 1 : c;
+    __device__ __forceinline__ void make(const RgArgs& a, const RgPlace& pl, int t, int t_end, int c, float2 (&u)[RM_TOK]) {
+        const int c1 = c + 1;
         const float2 beta = make_float2(a.convb[c], a.convb[c1]);
         if constexpr (TAPS > 0) {
-            float2 w[TAPS], base = beta;
+            const float2 bias = make_float2(a.xb[c], a.xb[c1]);
+            float2 w[TAPS];
 #pragma unroll
             for (int k = 0; k < TAPS; ++k) w[k] = make_float2(a.conv[(size_t)c * TAPS + k], a.conv[(size_t)c1 * TAPS + k]);
-            if (rows) {
-                // the input's bias enters every tap alike: β + b · Σ κ
-                const float2 bias = make_float2(a.xb[c], a.xb[c1]);
 #pragma unroll
-                for (int k = 0; k < TAPS; ++k) { base.x = fmaf(w[k].x, bias.x, base.x); base.y = fmaf(w[k].y, bias.y, base.y); }
-            }
+            for (int i = 0; i < N; ++i)
+                if (i >= BACK || t - BACK + i >= pl.first) { x[i].x += bias.x; x[i].y += bias.y; }
 #pragma unroll
             for (int i = 0; i < RM_TOK; ++i) {
-                float2 v = base;
+                float2 v = beta;
 #pragma unroll
                 for (int k = 0; k < TAPS; ++k) { v.x = fmaf(w[k].x, x[i + k].x, v.x); v.y = fmaf(w[k].y, x[i + k].y, v.y); }
                 u[i] = v;
@@ -294,7 +285,6 @@ rglru_chunk_mma_kernel(RgArgs a, int col_tiles) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t_end = pl.t0 + pl.n;
     const int nk = (size + RM_BK - 1) / RM_BK;
-    const bool wide = (a.ld & 1) == 0 && (a.W & 1) == 0 && (((uintptr_t)a.proj) & 7) == 0;      // (the part's size is a multiple of 8)
     // the blocks of K in order from the one behind the block's own channels: its own come last, so that their u is still in
     // shared memory when the gates meet it
     auto block_of = [&](int i) { const int kb = own + 1 + i; return kb < nk ? kb : kb - nk; };
@@ -318,14 +308,14 @@ rglru_chunk_mma_kernel(RgArgs a, int col_tiles) {
     RgConv2<TAPS> cv;
     auto fetch_a = [&](int i) {
         const int k = block_of(i) * RM_BK + 2 * lane;
-        if (k < size && t < t_end) cv.fetch(a, pl, t, t_end, part * size + k, k + 1 < size, wide);
+        if (k < size && t < t_end) cv.fetch(a, pl, t, t_end, part * size + k);          // (the part's size is a multiple of 8)
     };
     auto make_a = [&](int i) {
         __nv_bfloat16* Ah = sm + (i & 1) * RM_STAGE;
         __nv_bfloat16* Al = Ah + RM_A;
         const int k = block_of(i) * RM_BK + 2 * lane;
         float2 u[RM_TOK];
-        if (k < size && t < t_end) cv.make(a, pl, t, t_end, part * size + k, k + 1 < size, u);
+        if (k < size && t < t_end) cv.make(a, pl, t, t_end, part * size + k, u);
         else {
 #pragma unroll
             for (int r = 0; r < RM_TOK; ++r) u[r] = make_float2(0.0f, 0.0f);
@@ -389,33 +379,33 @@ rglru_chunk_mma_kernel(RgArgs a, int col_tiles) {
 // ---------------------------------------------------------------- the same on tcgen05, turned round (parts of 128 and 256)
 // The gate matrices' rows are the M of tcgen05.mma and the tokens its N, so that a channel is a lane of tensor memory and the
 // recurrence runs along its columns: no exchange between threads. A CTA keeps 128 channels' rows of both gates (all of K) in
-// shared memory and walks blocks of 64 tokens:
+// shared memory and walks chunks of 32 tokens:
 //   warp 0        one thread fetches the rows once by TMA (128-byte swizzle), ahead of the predecessor's end
-//   warp 1        one thread issues the products of a block: both gates x (high part + low part of u), K-major operands
-//   warps 2-9     the convolution of the next block: u of the part's channels as two bfloat16 numbers, in the swizzled layout
-//   warps 10-17   thread = (channel, 32 tokens): u of its own channel into registers (the buffer is then free), gates from
-//                 tensor memory, the recurrence of a chunk of 32 tokens, (Π a, S) out
-// Two accumulators (of 2 x 64 columns) let the products of a block run under the recurrence of the one before. Every wait is
-// bounded; one that runs out records a code, every role falls through to the common exit, tensor memory is freed.
+//   warp 1        one thread issues the products of a chunk: both gates x (high part + low part of u), K-major operands
+//   warps 2-9     the convolution: u of the part's channels as two bfloat16 numbers, in the swizzled layout, two buffers; a
+//                 warp makes 8 tokens of half the blocks of K, and the next block's inputs are on their way meanwhile
+//   warps 10-17   two groups take the chunks in turn, thread = channel: u of its own channel into registers (the buffer is then
+//                 free), gates from tensor memory, the recurrence, (Π a, S) out
+// Two accumulators (r 32 | i 32 columns each) let the products of a chunk run under the recurrence of the one before. Every
+// wait is bounded; one that runs out records a code, every role falls through to the common exit, tensor memory is freed.
 constexpr int RT_ROWS = 128;                         // channels of a CTA
-constexpr int RT_TOK = 64;                           // tokens of a block
 constexpr int RT_CHUNK = 32;                         // tokens of a chunk
 constexpr int RT_THREADS = 18 * 32;
-constexpr uint32_t RT_COLS = 256;                    // tensor memory: two accumulators of r 64 | i 64 columns
+constexpr uint32_t RT_COLS = 128;                    // tensor memory: two accumulators
 template <int NKB> struct RtSmem {
-    static constexpr int W_BOX = RT_ROWS * 128, U_BOX = RT_TOK * 128;
+    static constexpr int W_BOX = RT_ROWS * 128, U_BOX = RT_CHUNK * 128;
     static constexpr int W_BYTES = 2 * NKB * W_BOX, U_BYTES = 2 * NKB * U_BOX;       // [gate][block of K], [high / low][block of K]
-    static constexpr int TOTAL = W_BYTES + U_BYTES + 1024;
+    static constexpr int TOTAL = W_BYTES + 2 * U_BYTES + 1024;
 };
 
 template <int TAPS, int NKB>
 __global__ void __launch_bounds__(RT_THREADS, 1)
 rglru_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_r, const __grid_constant__ CUtensorMap map_i, const RgArgs a,
-                      int row_tiles, int walkers, int n_tiles, int* status) {
+                      int row_tiles, int walkers, int n_chunks, int* status) {
     using L = RtSmem<NKB>;
-    static_assert(NKB % 2 == 0, "the convolution's two buffers go by the block of K");
+    static_assert(NKB % 2 == 0, "two halves of the convolution's warps share the blocks of K");
     extern __shared__ __align__(16) uint8_t rt_smem[];
-    __shared__ __align__(8) uint64_t bar_w, bar_u_full, bar_u_free, bar_acc[2], bar_acc_free[2];
+    __shared__ __align__(8) uint64_t bar_w, bar_u_full[2], bar_u_free[2], bar_acc[2], bar_acc_free[2];
     __shared__ uint32_t tmem_slot;
     const uint32_t base = (smem_u32(rt_smem) + 1023u) & ~1023u;
     uint8_t* const base_ptr = rt_smem + (base - smem_u32(rt_smem));
@@ -425,11 +415,11 @@ rglru_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_r, const __grid_co
     const int c0 = tile_c * RT_ROWS, part = c0 / a.size, n0 = c0 - part * a.size;     // a part is one or two tiles
     if (threadIdx.x == 0) {
         mbar_init(smem_u32(&bar_w), 1);
-        mbar_init(smem_u32(&bar_u_full), 8);
-        mbar_init(smem_u32(&bar_u_free), 8);
-        for (int b = 0; b < 2; ++b) {
+        for (int b = 0; b < 2; ++b) {                     // arrivals by warp: eight of the convolution, four of a group
+            mbar_init(smem_u32(&bar_u_full[b]), 8);
+            mbar_init(smem_u32(&bar_u_free[b]), 4);
             mbar_init(smem_u32(&bar_acc[b]), 1);
-            mbar_init(smem_u32(&bar_acc_free[b]), 8);
+            mbar_init(smem_u32(&bar_acc_free[b]), 4);
         }
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
@@ -455,100 +445,105 @@ rglru_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_r, const __grid_co
 
     if (warp == 1) {
         if (lane == 0) {
-            constexpr uint32_t idesc = umma_idesc_bf16(RT_ROWS, RT_TOK);
+            constexpr uint32_t idesc = umma_idesc_bf16(RT_ROWS, RT_CHUNK);
             bool ok = mbar_wait(smem_u32(&bar_w), 0, status, 141);
             uint32_t it = 0;
             RgPlace pl;
-            for (int x = walker; x < n_tiles && ok; x += walkers) {
-                if (!rg_place(a, RT_TOK, x, pl)) continue;
-                const uint32_t buf = it & 1u;
-                ok = mbar_wait(smem_u32(&bar_acc_free[buf]), ((it >> 1) & 1u) ^ 1u, status, 143) &&
-                     mbar_wait(smem_u32(&bar_u_full), it & 1u, status, 144);
+            for (int x = walker; x < n_chunks && ok; x += walkers) {
+                if (!rg_place(a, RT_CHUNK, x, pl)) continue;
+                const uint32_t buf = it & 1u, phase = (it >> 1) & 1u;
+                ok = mbar_wait(smem_u32(&bar_acc_free[buf]), phase ^ 1u, status, 143) &&
+                     mbar_wait(smem_u32(&bar_u_full[buf]), phase, status, 144);
                 if (!ok) break;
                 tc_fence_after();
-#pragma unroll
+#pragma unroll 1
                 for (int gate = 0; gate < 2; ++gate) {
-                    const uint32_t d = tmem + buf * 128u + (uint32_t)gate * RT_TOK;
+                    const uint32_t d = tmem + buf * 64u + (uint32_t)gate * RT_CHUNK;
+#pragma unroll 1
+                    for (int i = 0; i < 2 * NKB; ++i) {              // the low parts first: small terms before large ones
+                        const int lo = i < NKB ? 1 : 0, kb = i < NKB ? i : i - NKB;
+                        const uint64_t dw = umma_desc_sw128(w_smem + (gate * NKB + kb) * L::W_BOX);
+                        const uint64_t du = umma_desc_sw128(u_smem + buf * L::U_BYTES + (lo * NKB + kb) * L::U_BOX);
 #pragma unroll
-                    for (int lo = 1; lo >= 0; --lo)                  // the low parts first: small terms before large ones
-#pragma unroll
-                        for (int kb = 0; kb < NKB; ++kb) {
-                            const uint64_t dw = umma_desc_sw128(w_smem + (gate * NKB + kb) * L::W_BOX);
-                            const uint64_t du = umma_desc_sw128(u_smem + (lo * NKB + kb) * L::U_BOX);
-#pragma unroll
-                            for (int k = 0; k < 4; ++k) tc_mma_bf16(d, dw + 2 * k, du + 2 * k, idesc, (lo == 1 && (kb | k) == 0) ? 0u : 1u);
-                        }
+                        for (int k = 0; k < 4; ++k) tc_mma_bf16(d, dw + 2 * k, du + 2 * k, idesc, (i | k) == 0 ? 0u : 1u);
+                    }
                 }
                 tc_commit(smem_u32(&bar_acc[buf]));
                 ++it;
             }
         }
     } else if (warp >= 2 && warp < 10) {
-        const int row0 = (warp - 2) * RM_TOK;                        // eight tokens per warp, two channels of a block of K per lane
-        const bool wide = (a.ld & 1) == 0 && (((uintptr_t)a.proj) & 7) == 0;
-        const int c = part * a.size + 2 * lane;
+        // eight tokens and half the blocks of K per warp, two channels of a block per lane
+        const int row0 = ((warp - 2) & 3) * RM_TOK, kb0 = ((warp - 2) >> 2) * (NKB / 2);
+        const int c = part * a.size + kb0 * 64 + 2 * lane;
         bool ok = true;
         uint32_t it = 0;
         RgPlace pl, ahead;
-        RgConv2<TAPS> cv[2];                                         // a block of K's inputs are asked for while the one before is made
+        RgConv2<TAPS> cur, nxt;                                      // the inputs that come next are asked for while one block is made
         int x = walker;
-        auto find = [&](RgPlace& p) {                                // the next block that exists, from x on
-            for (; x < n_tiles; x += walkers) if (rg_place(a, RT_TOK, x, p)) return true;
+        auto find = [&](RgPlace& p) {                                // the next chunk that exists, from x on
+            for (; x < n_chunks; x += walkers) if (rg_place(a, RT_CHUNK, x, p)) return true;
             return false;
         };
-        bool have = find(pl);
-        if (have && pl.t0 + row0 < pl.t0 + pl.n) cv[0].fetch(a, pl, pl.t0 + row0, pl.t0 + pl.n, c, true, wide);
+        bool have = find(pl), more = false;
+        if (have && row0 < pl.n) cur.fetch(a, pl, pl.t0 + row0, pl.t0 + pl.n, c);
+        int j = 0;
+#pragma unroll 1
         while (have) {
-            x += walkers;
-            const bool more = find(ahead);
-            ok = mbar_wait(smem_u32(&bar_u_free), (it & 1u) ^ 1u, status, 142);
-            ok = __all_sync(0xffffffffu, ok);
-            if (!ok) break;
-            const int t = pl.t0 + row0, t_end = pl.t0 + pl.n;
-#pragma unroll
-            for (int kb = 0; kb < NKB; ++kb) {
-                if (kb + 1 < NKB) {
-                    if (t < t_end) cv[(kb + 1) & 1].fetch(a, pl, t, t_end, c + (kb + 1) * 64, true, wide);
-                } else if (more && row0 < ahead.n) {
-                    cv[0].fetch(a, ahead, ahead.t0 + row0, ahead.t0 + ahead.n, c, true, wide);
-                }
-                float2 u[RM_TOK];
-                if (t < t_end) cv[kb & 1].make(a, pl, t, t_end, c + kb * 64, true, u);
-                else {
-#pragma unroll
-                    for (int r = 0; r < RM_TOK; ++r) u[r] = make_float2(0.0f, 0.0f);
-                }
-                uint8_t* hi_box = base_ptr + L::W_BYTES + kb * L::U_BOX + row0 * 128;      // row0 is a multiple of 8: row & 7 = r
-#pragma unroll
-                for (int r = 0; r < RM_TOK; ++r) {
-                    const uint32_t at = r * 128 + (((lane >> 2) ^ r) << 4) + (lane & 3) * 4;
-                    const __nv_bfloat162 hi = __floats2bfloat162_rn(u[r].x, u[r].y);
-                    const float2 back = __bfloat1622float2(hi);
-                    *(__nv_bfloat162*)(hi_box + at) = hi;
-                    *(__nv_bfloat162*)(hi_box + NKB * L::U_BOX + at) = __floats2bfloat162_rn(u[r].x - back.x, u[r].y - back.y);
-                }
+            const bool last_j = j + 1 == NKB / 2;
+            if (last_j) { x += walkers; more = find(ahead); }
+            const RgPlace& np = last_j ? ahead : pl;
+            const int nj = last_j ? 0 : j + 1;
+            if ((!last_j || more) && row0 < np.n) nxt.fetch(a, np, np.t0 + row0, np.t0 + np.n, c + nj * 64);
+            const uint32_t buf = it & 1u;
+            if (j == 0) {
+                ok = mbar_wait(smem_u32(&bar_u_free[buf]), ((it >> 1) & 1u) ^ 1u, status, 142);
+                ok = __all_sync(0xffffffffu, ok);
+                if (!ok) break;
             }
-            asm volatile("fence.proxy.async.shared::cta;" ::: "memory");      // the products read what these stores wrote
-            __syncwarp();
-            if (lane == 0) mbar_arrive(smem_u32(&bar_u_full));
-            ++it;
-            pl = ahead;
-            have = more;
+            float2 u[RM_TOK];
+            if (row0 < pl.n) cur.make(a, pl, pl.t0 + row0, pl.t0 + pl.n, c + j * 64, u);
+            else {
+#pragma unroll
+                for (int r = 0; r < RM_TOK; ++r) u[r] = make_float2(0.0f, 0.0f);
+            }
+            uint8_t* hi_box = base_ptr + L::W_BYTES + buf * L::U_BYTES + (kb0 + j) * L::U_BOX + row0 * 128;      // row0 is a multiple of 8: row & 7 = r
+#pragma unroll
+            for (int r = 0; r < RM_TOK; ++r) {
+                const uint32_t at = r * 128 + (((lane >> 2) ^ r) << 4) + (lane & 3) * 4;
+                const __nv_bfloat162 hi = __floats2bfloat162_rn(u[r].x, u[r].y);
+                const float2 back = __bfloat1622float2(hi);
+                *(__nv_bfloat162*)(hi_box + at) = hi;
+                *(__nv_bfloat162*)(hi_box + NKB * L::U_BOX + at) = __floats2bfloat162_rn(u[r].x - back.x, u[r].y - back.y);
+            }
+            if (last_j) {
+                asm volatile("fence.proxy.async.shared::cta;" ::: "memory");      // the products read what these stores wrote
+                __syncwarp();
+                if (lane == 0) mbar_arrive(smem_u32(&bar_u_full[buf]));
+                ++it;
+                pl = ahead;
+                have = more;
+            }
+            j = nj;
+            cur = nxt;
         }
     } else if (warp >= 10) {
-        const int q = warp & 3, half = (warp - 10) >> 2;             // lanes 32q … of tensor memory, tokens 32·half …
+        const uint32_t group = (uint32_t)(warp - 10) >> 2;           // takes every second chunk of this CTA
+        const int q = warp & 3;                                      // lanes 32q … of tensor memory
         const int ch = q * 32 + lane, c = c0 + ch;
         const float rb = a.rab[c], ib = a.rib[c], dec = a.decay[c];
         const int k = (n0 + ch) & 63;
-        const uint8_t* own = base_ptr + L::W_BYTES + ((n0 + ch) >> 6) * L::U_BOX + half * 32 * 128 + (k & 7) * 2;
+        const uint8_t* own = base_ptr + L::W_BYTES + group * L::U_BYTES + ((n0 + ch) >> 6) * L::U_BOX + (k & 7) * 2;
         bool ok = true;
         uint32_t it = 0;
         RgPlace pl;
-        for (int x = walker; x < n_tiles && ok; x += walkers) {
-            if (!rg_place(a, RT_TOK, x, pl)) continue;
-            const uint32_t buf = it & 1u;
+        for (int x = walker; x < n_chunks && ok; x += walkers) {
+            if (!rg_place(a, RT_CHUNK, x, pl)) continue;
+            if ((it & 1u) != group) { ++it; continue; }
+            const uint32_t phase = (it >> 1) & 1u;
+            ++it;
             // (the convolution's own barrier too: this warp reads what those warps stored)
-            ok = mbar_wait(smem_u32(&bar_u_full), it & 1u, status, 145) && mbar_wait(smem_u32(&bar_acc[buf]), (it >> 1) & 1u, status, 145);
+            ok = mbar_wait(smem_u32(&bar_u_full[group]), phase, status, 145) && mbar_wait(smem_u32(&bar_acc[group]), phase, status, 145);
             ok = __all_sync(0xffffffffu, ok);
             if (!ok) break;
             tc_fence_after();
@@ -559,23 +554,22 @@ rglru_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_r, const __grid_co
                 up[i] = ((uint32_t)*(const uint16_t*)p << 16) | *(const uint16_t*)(p + NKB * L::U_BOX);
             }
             __syncwarp();
-            if (lane == 0) mbar_arrive(smem_u32(&bar_u_free));
-            const int n = min(RT_CHUNK, pl.n - half * RT_CHUNK);     // tokens of this thread's chunk (none: n <= 0)
-            const int t = pl.t0 + half * RT_CHUNK;
+            if (lane == 0) mbar_arrive(smem_u32(&bar_u_free[group]));
+            const int t = pl.t0, n = pl.n;
             const bool begins = t == pl.first;                       // a sequence's first chunk begins with its state
             float A = begins ? 0.0f : 1.0f, S = begins ? a.state[(size_t)pl.slot * a.W + c] : 0.0f;
             float2* av = a.av + (size_t)t * a.W + c;
-            const uint32_t acc = tmem + ((uint32_t)(q * 32) << 16) + buf * 128u + half * RT_CHUNK;
+            const uint32_t acc = tmem + ((uint32_t)(q * 32) << 16) + group * 64u;
 #pragma unroll
             for (int h = 0; h < 2; ++h) {
                 uint32_t zr[16], zi[16];
                 tc_ld_32x16(acc + h * 16, zr);
-                tc_ld_32x16(acc + RT_TOK + h * 16, zi);
+                tc_ld_32x16(acc + RT_CHUNK + h * 16, zi);
                 tc_ld_wait();
                 if (h == 1) {
                     tc_fence_before();
                     __syncwarp();
-                    if (lane == 0) mbar_arrive(smem_u32(&bar_acc_free[buf]));
+                    if (lane == 0) mbar_arrive(smem_u32(&bar_acc_free[group]));
                 }
                 // the tokens' gates side by side (no branch per token), then the recurrence
 #pragma unroll
@@ -596,12 +590,7 @@ rglru_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_r, const __grid_co
                     }
                 }
             }
-            if (n > 0) {
-                int cell = (pl.t0 - pl.first) / RT_CHUNK + half;
-                for (int b = 0; b < pl.s; ++b) cell += (a.seq_start[b + 1] - a.seq_start[b] + RT_CHUNK - 1) / RT_CHUNK;
-                a.cells[(size_t)cell * a.W + c] = make_float2(A, S);
-            }
-            ++it;
+            a.cells[(size_t)x * a.W + c] = make_float2(A, S);        // chunks are counted as cells are
         }
     }
     __syncwarp();
@@ -974,7 +963,7 @@ int gate_map(CUtensorMap* map, const void* ptr, int rows, int size) {
 }
 
 template <int TAPS, int NKB>
-int launch_tc(const CUtensorMap& mr, const CUtensorMap& mi, const RgArgs& a, int n_tiles, int* status, cudaStream_t stream) {
+int launch_tc(const CUtensorMap& mr, const CUtensorMap& mi, const RgArgs& a, int n_chunks, int* status, cudaStream_t stream) {
     static SpPerDevice ready;
     if (!ready.done()) {
         if (cudaFuncSetAttribute(rglru_chunk_tc_kernel<TAPS, NKB>, cudaFuncAttributeMaxDynamicSharedMemorySize, RtSmem<NKB>::TOTAL) != cudaSuccess)
@@ -983,13 +972,14 @@ int launch_tc(const CUtensorMap& mr, const CUtensorMap& mi, const RgArgs& a, int
     }
     const int row_tiles = a.W / RT_ROWS, sms = sp_sm_count();
     int walkers = sms / row_tiles;
-    walkers = walkers < 1 ? 1 : walkers > n_tiles ? n_tiles : walkers;
+    walkers = walkers < 1 ? 1 : walkers > n_chunks ? n_chunks : walkers;
     SP_CHECK_CALL("rglru_chunk", sp_launch_dependent(rglru_chunk_tc_kernel<TAPS, NKB>, dim3(row_tiles * walkers), dim3(RT_THREADS),
-                                                     (size_t)RtSmem<NKB>::TOTAL, stream, mr, mi, a, row_tiles, walkers, n_tiles, status));
+                                                     (size_t)RtSmem<NKB>::TOTAL, stream, mr, mi, a, row_tiles, walkers, n_chunks, status));
     return 0;
 }
 
 bool takes_tc(int g_dt, int size, int tensor_cores) { return tensor_cores && g_dt == SP_DT_BF16 && (size == 128 || size == 256); }
+bool in_pairs(const RgArgs& a) { return (a.ld & 1) == 0 && (a.W & 1) == 0 && (((uintptr_t)a.proj | (uintptr_t)a.ring) & 7) == 0; }
 
 }  // namespace
 
@@ -1016,15 +1006,13 @@ SP_API int sp_rglru_chunked(const float* proj, int ld, const float* yb, const fl
     const dim3 grid(parts * col_tiles, n_chunks);
     if (tc) {
         a.chunk = RT_CHUNK;
-        if (!aligned) SP_FAIL("rglru: the gate matrices must start on a 16-byte boundary");
+        if (!aligned || !in_pairs(a)) SP_FAIL("rglru: the gate matrices must start on a 16-byte boundary, rows and ring on 8-byte ones");
         CUtensorMap mr, mi;
         if (gate_map(&mr, ra, W, a.size) || gate_map(&mi, ri, W, a.size)) return 1;
-        // blocks of 64 tokens: at most as many as this (a sequence's last block may be half a block)
-        const int n_tiles = (n_chunks + B + 1) / 2;
-        if (a.size == 256 ? (taps == 4 ? launch_tc<4, 4>(mr, mi, a, n_tiles, status, stream) : launch_tc<0, 4>(mr, mi, a, n_tiles, status, stream))
-                          : (taps == 4 ? launch_tc<4, 2>(mr, mi, a, n_tiles, status, stream) : launch_tc<0, 2>(mr, mi, a, n_tiles, status, stream)))
+        if (a.size == 256 ? (taps == 4 ? launch_tc<4, 4>(mr, mi, a, n_chunks, status, stream) : launch_tc<0, 4>(mr, mi, a, n_chunks, status, stream))
+                          : (taps == 4 ? launch_tc<4, 2>(mr, mi, a, n_chunks, status, stream) : launch_tc<0, 2>(mr, mi, a, n_chunks, status, stream)))
             return 1;
-    } else if (tensor_cores && g_dt == SP_DT_BF16 && a.size % 8 == 0 && aligned) {
+    } else if (tensor_cores && g_dt == SP_DT_BF16 && a.size % 8 == 0 && aligned && in_pairs(a)) {
         static SpPerDevice ready;
         if (!ready.done()) {
             if (cudaFuncSetAttribute(rglru_chunk_mma_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, RM_SMEM) != cudaSuccess ||
