@@ -73,6 +73,26 @@ __device__ __forceinline__ bool rg_place(const RgArgs& a, int tokens, int x, RgP
     return false;
 }
 
+// The same for a block that takes pieces x in rising order: the sequence it stands in is remembered.
+struct RgWalk {
+    int s = -1, base = 0, nc = 0, first = 0, cnt = 0, pos0 = 0, slot = -1;
+    __device__ __forceinline__ bool place(const RgArgs& a, int tokens, int x, RgPlace& pl) {
+        while (x >= base + nc) {
+            if (++s >= a.B) { s = a.B - 1; return false; }
+            base += nc;
+            first = a.seq_start[s];
+            cnt = a.seq_start[s + 1] - first;
+            nc = (cnt + tokens - 1) / tokens;
+            pos0 = a.positions[first];
+            slot = a.seq_slot[s];
+        }
+        pl.s = s; pl.first = first; pl.pos0 = pos0; pl.slot = slot;
+        pl.t0 = first + (x - base) * tokens;
+        pl.n = min(tokens, first + cnt - pl.t0);
+        return slot >= 0 && slot < a.n_slots;
+    }
+};
+
 // x + b of channel c at token ``t``: from the step's own rows, from the ring for the tokens before the step's first, or
 // nothing before the sequence's start. There is no branch around the load, so that the loads of many tokens are under way
 // together: the address is always one of the step's rows or of the ring's (a convolution of one tap never looks back).
@@ -128,7 +148,12 @@ __device__ __forceinline__ void rg_gates(float zr, float zi, float u, float deca
 // The same for the tensor-core kernels, whose gates come from operands of sixteen bits: the hardware's approximations (a few
 // units in the last place). a − 1 keeps its relative accuracy near a = 1, where the state's memory lies: the power series
 // of e^x − 1 for x > −0.3 (its next term is below 2⁻²⁷ of the sum there).
-__device__ __forceinline__ float rg_sigmoid_fast(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
+__device__ __forceinline__ float rg_ex2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+__device__ __forceinline__ float rg_sigmoid_fast(float z) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(1.0f + rg_ex2(-1.4426950408889634f * z)));
+    return y;
+}
 __device__ __forceinline__ void rg_gates_fast(float zr, float zi, float u, float decay, float& d, float& v) {
     const float x = -decay * rg_sigmoid_fast(zr);
     float series = fmaf(x, 1.0f / 5040.0f, 1.0f / 720.0f);
@@ -137,10 +162,10 @@ __device__ __forceinline__ void rg_gates_fast(float zr, float zi, float u, float
     series = fmaf(x, series, 1.0f / 6.0f);
     series = fmaf(x, series, 0.5f);
     series = fmaf(x * x, series, x);
-    const float below = x > -0.3f ? series : __expf(x) - 1.0f;
+    const float below = x > -0.3f ? series : rg_ex2(1.4426950408889634f * x) - 1.0f;
     d = 1.0f + below;
     float root;
-    asm("sqrt.approx.f32 %0, %1;" : "=f"(root) : "f"(-below * (2.0f + below)));
+    asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(root) : "f"(-below * (2.0f + below)));
     v = root * rg_sigmoid_fast(zi) * u;
 }
 
@@ -218,15 +243,15 @@ struct RgConv2 {
         }
     }
 
-    // u of the tokens; tokens at t_end or beyond get 0
-    __device__ __forceinline__ void make(const RgArgs& a, const RgPlace& pl, int t, int t_end, int c, float2 (&u)[RM_TOK]) {
+    // u of the tokens; tokens at t_end or beyond get 0. ``weight(k)``: both channels' tap k, then (TAPS) β, then (TAPS + 1) b
+    template <typename W2>
+    __device__ __forceinline__ void make(const RgArgs& a, const RgPlace& pl, int t, int t_end, int c, float2 (&u)[RM_TOK], W2&& weight) {
         const int c1 = c + 1;
-        const float2 beta = make_float2(a.convb[c], a.convb[c1]);
         if constexpr (TAPS > 0) {
-            const float2 bias = make_float2(a.xb[c], a.xb[c1]);
+            const float2 beta = weight(TAPS), bias = weight(TAPS + 1);
             float2 w[TAPS];
 #pragma unroll
-            for (int k = 0; k < TAPS; ++k) w[k] = make_float2(a.conv[(size_t)c * TAPS + k], a.conv[(size_t)c1 * TAPS + k]);
+            for (int k = 0; k < TAPS; ++k) w[k] = weight(k);
 #pragma unroll
             for (int i = 0; i < N; ++i)
                 if (i >= BACK || t - BACK + i >= pl.first) { x[i].x += bias.x; x[i].y += bias.y; }
@@ -238,7 +263,7 @@ struct RgConv2 {
                 u[i] = v;
             }
         } else {
-            const float2 bias = make_float2(a.xb[c], a.xb[c1]);
+            const float2 beta = make_float2(a.convb[c], a.convb[c1]), bias = make_float2(a.xb[c], a.xb[c1]);
 #pragma unroll
             for (int i = 0; i < RM_TOK; ++i) u[i] = beta;
             for (int k = 0; k < a.taps; ++k) {
@@ -257,6 +282,13 @@ struct RgConv2 {
         for (int i = 0; i < RM_TOK; ++i) if (t + i >= t_end) u[i] = make_float2(0.0f, 0.0f);
     }
 };
+
+template <int TAPS>
+__device__ __forceinline__ float2 rg_conv_weight(const RgArgs& a, int c, int k) {
+    if (k == TAPS) return make_float2(a.convb[c], a.convb[c + 1]);
+    if (k == TAPS + 1) return make_float2(a.xb[c], a.xb[c + 1]);
+    return make_float2(a.conv[(size_t)c * TAPS + k], a.conv[(size_t)(c + 1) * TAPS + k]);
+}
 
 // ---------------------------------------------------------------- gate products on mma.sync (parts of any multiple of 8)
 constexpr int RM_BK = 64;
@@ -315,7 +347,7 @@ rglru_chunk_mma_kernel(RgArgs a, int col_tiles) {
         __nv_bfloat16* Al = Ah + RM_A;
         const int k = block_of(i) * RM_BK + 2 * lane;
         float2 u[RM_TOK];
-        if (k < size && t < t_end) cv.make(a, pl, t, t_end, part * size + k, u);
+        if (k < size && t < t_end) cv.make(a, pl, t, t_end, part * size + k, u, [&](int w) { return rg_conv_weight<TAPS>(a, part * size + k, w); });
         else {
 #pragma unroll
             for (int r = 0; r < RM_TOK; ++r) u[r] = make_float2(0.0f, 0.0f);
@@ -381,21 +413,23 @@ rglru_chunk_mma_kernel(RgArgs a, int col_tiles) {
 // recurrence runs along its columns: no exchange between threads. A CTA keeps 128 channels' rows of both gates (all of K) in
 // shared memory and walks chunks of 32 tokens:
 //   warp 0        one thread fetches the rows once by TMA (128-byte swizzle), ahead of the predecessor's end
-//   warp 1        one thread issues the products of a chunk: both gates x (high part + low part of u), K-major operands
+//   warp 1        one thread issues the products of a chunk: for each gate 64 columns, the high parts of u and the low parts,
+//                 whose sums meet in the registers (K-major operands)
 //   warps 2-9     the convolution: u of the part's channels as two bfloat16 numbers, in the swizzled layout, two buffers; a
 //                 warp makes 8 tokens of half the blocks of K, and the next block's inputs are on their way meanwhile
-//   warps 10-17   two groups take the chunks in turn, thread = channel: u of its own channel into registers (the buffer is then
-//                 free), gates from tensor memory, the recurrence, (Π a, S) out
-// Two accumulators (r 32 | i 32 columns each) let the products of a chunk run under the recurrence of the one before. Every
+//   warps 10-17   two groups take the chunks in turn, thread = channel: u of its own channel into tensor memory beside the
+//                 accumulator (the buffer is then free), gates from there, the recurrence, (Π a, S) out
+// Two accumulators (r high | r low | i high | i low, 32 columns each) let the products of a chunk run under the recurrence of the one before. Every
 // wait is bounded; one that runs out records a code, every role falls through to the common exit, tensor memory is freed.
 constexpr int RT_ROWS = 128;                         // channels of a CTA
 constexpr int RT_CHUNK = 32;                         // tokens of a chunk
 constexpr int RT_THREADS = 18 * 32;
-constexpr uint32_t RT_COLS = 128;                    // tensor memory: two accumulators
+constexpr uint32_t RT_COLS = 512, RT_U = 256;        // tensor memory: two accumulators of 128 columns, from RT_U on 32 columns of u per group
 template <int NKB> struct RtSmem {
-    static constexpr int W_BOX = RT_ROWS * 128, U_BOX = RT_CHUNK * 128;
-    static constexpr int W_BYTES = 2 * NKB * W_BOX, U_BYTES = 2 * NKB * U_BOX;       // [gate][block of K], [high / low][block of K]
-    static constexpr int TOTAL = W_BYTES + 2 * U_BYTES + 1024;
+    static constexpr int W_BOX = RT_ROWS * 128, U_BOX = 2 * RT_CHUNK * 128, LOW = RT_CHUNK * 128;
+    static constexpr int W_BYTES = 2 * NKB * W_BOX, U_BYTES = NKB * U_BOX;           // [gate][block of K], [block of K][high | low rows]
+    static constexpr int TAPS_AT = W_BYTES + 2 * U_BYTES;                            // [taps | β | b][the part's channels] float32
+    static constexpr int total(int taps) { return TAPS_AT + (taps + 2) * NKB * 64 * 4 + 1024; }
 };
 
 template <int TAPS, int NKB>
@@ -440,34 +474,40 @@ rglru_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_r, const __grid_co
             tma_load_2d(w_smem + (NKB + kb) * L::W_BOX, &map_i, kb * 64, c0, smem_u32(&bar_w));
         }
     }
+    // the convolution's weights of the part's channels (nobody's output either)
+    float* const taps_smem = (float*)(base_ptr + L::TAPS_AT);
+    for (int e = threadIdx.x; e < (TAPS + 2) * NKB * 64; e += RT_THREADS) {
+        const int kk = e / (NKB * 64), cc = part * a.size + e % (NKB * 64);
+        taps_smem[e] = kk < TAPS ? a.conv[(size_t)cc * TAPS + kk] : kk == TAPS ? a.convb[cc] : a.xb[cc];
+    }
+    __syncthreads();
     sp_allow_dependents();
     sp_wait_for_predecessor();
 
     if (warp == 1) {
         if (lane == 0) {
-            constexpr uint32_t idesc = umma_idesc_bf16(RT_ROWS, RT_CHUNK);
+            constexpr uint32_t idesc = umma_idesc_bf16(RT_ROWS, 2 * RT_CHUNK);
             bool ok = mbar_wait(smem_u32(&bar_w), 0, status, 141);
             uint32_t it = 0;
             RgPlace pl;
+            RgWalk walk;
             for (int x = walker; x < n_chunks && ok; x += walkers) {
-                if (!rg_place(a, RT_CHUNK, x, pl)) continue;
+                if (!walk.place(a, RT_CHUNK, x, pl)) continue;
                 const uint32_t buf = it & 1u, phase = (it >> 1) & 1u;
                 ok = mbar_wait(smem_u32(&bar_acc_free[buf]), phase ^ 1u, status, 143) &&
                      mbar_wait(smem_u32(&bar_u_full[buf]), phase, status, 144);
                 if (!ok) break;
                 tc_fence_after();
-#pragma unroll 1
-                for (int gate = 0; gate < 2; ++gate) {
-                    const uint32_t d = tmem + buf * 64u + (uint32_t)gate * RT_CHUNK;
-#pragma unroll 1
-                    for (int i = 0; i < 2 * NKB; ++i) {              // the low parts first: small terms before large ones
-                        const int lo = i < NKB ? 1 : 0, kb = i < NKB ? i : i - NKB;
-                        const uint64_t dw = umma_desc_sw128(w_smem + (gate * NKB + kb) * L::W_BOX);
-                        const uint64_t du = umma_desc_sw128(u_smem + buf * L::U_BYTES + (lo * NKB + kb) * L::U_BOX);
 #pragma unroll
-                        for (int k = 0; k < 4; ++k) tc_mma_bf16(d, dw + 2 * k, du + 2 * k, idesc, (i | k) == 0 ? 0u : 1u);
+                for (int gate = 0; gate < 2; ++gate)
+#pragma unroll
+                    for (int kb = 0; kb < NKB; ++kb) {
+                        const uint64_t dw = umma_desc_sw128(w_smem + (gate * NKB + kb) * L::W_BOX);
+                        const uint64_t du = umma_desc_sw128(u_smem + buf * L::U_BYTES + kb * L::U_BOX);
+#pragma unroll
+                        for (int k = 0; k < 4; ++k)
+                            tc_mma_bf16(tmem + buf * 128u + (uint32_t)gate * 64u, dw + 2 * k, du + 2 * k, idesc, (kb | k) == 0 ? 0u : 1u);
                     }
-                }
                 tc_commit(smem_u32(&bar_acc[buf]));
                 ++it;
             }
@@ -481,8 +521,9 @@ rglru_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_r, const __grid_co
         RgPlace pl, ahead;
         RgConv2<TAPS> cur, nxt;                                      // the inputs that come next are asked for while one block is made
         int x = walker;
+        RgWalk walk;
         auto find = [&](RgPlace& p) {                                // the next chunk that exists, from x on
-            for (; x < n_chunks; x += walkers) if (rg_place(a, RT_CHUNK, x, p)) return true;
+            for (; x < n_chunks; x += walkers) if (walk.place(a, RT_CHUNK, x, p)) return true;
             return false;
         };
         bool have = find(pl), more = false;
@@ -502,7 +543,9 @@ rglru_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_r, const __grid_co
                 if (!ok) break;
             }
             float2 u[RM_TOK];
-            if (row0 < pl.n) cur.make(a, pl, pl.t0 + row0, pl.t0 + pl.n, c + j * 64, u);
+            if (row0 < pl.n) cur.make(a, pl, pl.t0 + row0, pl.t0 + pl.n, c + j * 64, u, [&](int w) {
+                return *(const float2*)(taps_smem + w * NKB * 64 + (kb0 + j) * 64 + 2 * lane);
+            });
             else {
 #pragma unroll
                 for (int r = 0; r < RM_TOK; ++r) u[r] = make_float2(0.0f, 0.0f);
@@ -514,7 +557,7 @@ rglru_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_r, const __grid_co
                 const __nv_bfloat162 hi = __floats2bfloat162_rn(u[r].x, u[r].y);
                 const float2 back = __bfloat1622float2(hi);
                 *(__nv_bfloat162*)(hi_box + at) = hi;
-                *(__nv_bfloat162*)(hi_box + NKB * L::U_BOX + at) = __floats2bfloat162_rn(u[r].x - back.x, u[r].y - back.y);
+                *(__nv_bfloat162*)(hi_box + L::LOW + at) = __floats2bfloat162_rn(u[r].x - back.x, u[r].y - back.y);
             }
             if (last_j) {
                 asm volatile("fence.proxy.async.shared::cta;" ::: "memory");      // the products read what these stores wrote
@@ -537,8 +580,9 @@ rglru_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_r, const __grid_co
         bool ok = true;
         uint32_t it = 0;
         RgPlace pl;
+        RgWalk walk;
         for (int x = walker; x < n_chunks && ok; x += walkers) {
-            if (!rg_place(a, RT_CHUNK, x, pl)) continue;
+            if (!walk.place(a, RT_CHUNK, x, pl)) continue;
             if ((it & 1u) != group) { ++it; continue; }
             const uint32_t phase = (it >> 1) & 1u;
             ++it;
@@ -547,46 +591,51 @@ rglru_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_r, const __grid_co
             ok = __all_sync(0xffffffffu, ok);
             if (!ok) break;
             tc_fence_after();
-            uint32_t up[RT_CHUNK];                                   // u: high part above, low part below
+            const uint32_t lanes = tmem + ((uint32_t)(q * 32) << 16), own_u = lanes + RT_U + group * RT_CHUNK;
+            {
+                uint32_t up[RT_CHUNK];                               // high part above, low part below
 #pragma unroll
-            for (int i = 0; i < RT_CHUNK; ++i) {
-                const uint8_t* p = own + i * 128 + (((k >> 3) ^ (i & 7)) << 4);
-                up[i] = ((uint32_t)*(const uint16_t*)p << 16) | *(const uint16_t*)(p + NKB * L::U_BOX);
+                for (int i = 0; i < RT_CHUNK; ++i) {
+                    const uint8_t* p = own + i * 128 + (((k >> 3) ^ (i & 7)) << 4);
+                    up[i] = ((uint32_t)*(const uint16_t*)p << 16) | *(const uint16_t*)(p + L::LOW);
+                }
+                tc_st_32x32(own_u, up);
+                __syncwarp();
+                if (lane == 0) mbar_arrive(smem_u32(&bar_u_free[group]));
+                tc_st_wait();
             }
-            __syncwarp();
-            if (lane == 0) mbar_arrive(smem_u32(&bar_u_free[group]));
             const int t = pl.t0, n = pl.n;
             const bool begins = t == pl.first;                       // a sequence's first chunk begins with its state
             float A = begins ? 0.0f : 1.0f, S = begins ? a.state[(size_t)pl.slot * a.W + c] : 0.0f;
             float2* av = a.av + (size_t)t * a.W + c;
-            const uint32_t acc = tmem + ((uint32_t)(q * 32) << 16) + group * 64u;
-#pragma unroll
-            for (int h = 0; h < 2; ++h) {
-                uint32_t zr[16], zi[16];
-                tc_ld_32x16(acc + h * 16, zr);
-                tc_ld_32x16(acc + RT_CHUNK + h * 16, zi);
+            const uint32_t acc = lanes + group * 128u;
+            // eight tokens at a time: their gates side by side (no branch per token), then the recurrence
+#pragma unroll 1
+            for (int h = 0; h < RT_CHUNK / 8; ++h) {
+                uint32_t zr[8], zi[8], lr[8], li[8];
+                tc_ld_32x8(acc + h * 8, zr);
+                tc_ld_32x8(acc + 32 + h * 8, lr);
+                tc_ld_32x8(acc + 64 + h * 8, zi);
+                tc_ld_32x8(acc + 96 + h * 8, li);
+                uint32_t up[8];
+                tc_ld_32x8(own_u + h * 8, up);
                 tc_ld_wait();
-                if (h == 1) {
+                if (h == RT_CHUNK / 8 - 1) {
                     tc_fence_before();
                     __syncwarp();
                     if (lane == 0) mbar_arrive(smem_u32(&bar_acc_free[group]));
                 }
-                // the tokens' gates side by side (no branch per token), then the recurrence
+                float d[8], v[8];
 #pragma unroll
-                for (int i = 0; i < 16; ++i) {
-                    const uint32_t w = up[h * 16 + i];
-                    float d, v;
-                    rg_gates_fast(__uint_as_float(zr[i]) + rb, __uint_as_float(zi[i]) + ib,
-                                  __uint_as_float(w & 0xffff0000u) + __uint_as_float(w << 16), dec, d, v);
-                    zr[i] = __float_as_uint(d);
-                    zi[i] = __float_as_uint(v);
-                }
+                for (int i = 0; i < 8; ++i)
+                    rg_gates_fast(__uint_as_float(zr[i]) + (__uint_as_float(lr[i]) + rb), __uint_as_float(zi[i]) + (__uint_as_float(li[i]) + ib),
+                                  __uint_as_float(up[i] & 0xffff0000u) + __uint_as_float(up[i] << 16), dec, d[i], v[i]);
 #pragma unroll
-                for (int i = 0; i < 16; ++i) {
-                    if (h * 16 + i < n) {
-                        S = fmaf(__uint_as_float(zr[i]), S, __uint_as_float(zi[i]));
-                        A *= __uint_as_float(zr[i]);
-                        av[(size_t)(h * 16 + i) * a.W] = make_float2(A, S);
+                for (int i = 0; i < 8; ++i) {
+                    if (h * 8 + i < n) {
+                        S = fmaf(d[i], S, v[i]);
+                        A *= d[i];
+                        av[(size_t)(h * 8 + i) * a.W] = make_float2(A, S);
                     }
                 }
             }
@@ -966,15 +1015,15 @@ template <int TAPS, int NKB>
 int launch_tc(const CUtensorMap& mr, const CUtensorMap& mi, const RgArgs& a, int n_chunks, int* status, cudaStream_t stream) {
     static SpPerDevice ready;
     if (!ready.done()) {
-        if (cudaFuncSetAttribute(rglru_chunk_tc_kernel<TAPS, NKB>, cudaFuncAttributeMaxDynamicSharedMemorySize, RtSmem<NKB>::TOTAL) != cudaSuccess)
-            SP_FAIL("rglru: cannot reserve %d bytes of shared memory", RtSmem<NKB>::TOTAL);
+        if (cudaFuncSetAttribute(rglru_chunk_tc_kernel<TAPS, NKB>, cudaFuncAttributeMaxDynamicSharedMemorySize, RtSmem<NKB>::total(TAPS)) != cudaSuccess)
+            SP_FAIL("rglru: cannot reserve %d bytes of shared memory", RtSmem<NKB>::total(TAPS));
         ready.mark();
     }
     const int row_tiles = a.W / RT_ROWS, sms = sp_sm_count();
     int walkers = sms / row_tiles;
     walkers = walkers < 1 ? 1 : walkers > n_chunks ? n_chunks : walkers;
     SP_CHECK_CALL("rglru_chunk", sp_launch_dependent(rglru_chunk_tc_kernel<TAPS, NKB>, dim3(row_tiles * walkers), dim3(RT_THREADS),
-                                                     (size_t)RtSmem<NKB>::TOTAL, stream, mr, mi, a, row_tiles, walkers, n_chunks, status));
+                                                     (size_t)RtSmem<NKB>::total(TAPS), stream, mr, mi, a, row_tiles, walkers, n_chunks, status));
     return 0;
 }
 
