@@ -7,6 +7,7 @@
     python bench.py --design kugirax [--design-sizes 1k,2k,4k]      (the Kugirax decoder likewise)
     python bench.py --design fotulix [--design-sizes 1k,2k,4k]      (the Fotulix decoder beside Kugirax and Llama)
     python bench.py --design luvavik [--design-sizes 1k,2k,4k]      (the Luvavik decoder beside Kugirax, Duzinex and Llama)
+    python bench.py --design lazulix [--design-sizes 1k,2k,4k]      (the Lazulix decoder beside Fotulix, Duzinex and Llama)
 
 Prints ONE JSON line. ``value`` is decoded tokens per second at batch 8 from prompts of
 about 2,048 tokens in a cache of 4,096 tokens per sequence, timed on the device with CUDA
@@ -361,6 +362,34 @@ def kugirax_config_like_luvavik(size: dict, lv: dict) -> dict:
     return dict(architecture="Kugirax", vocab=DESIGN_VOCAB, width=W, norm=dict(eps=1e-6), logit_softcap=30.0, layers=layers)
 
 
+# --design lazulix: eight layers, every sublayer between two layer norms, dense clamped feed-forwards of ``ff``: layers 0 and
+# 5 an attention with normed q and k and a gate per element (keys of 128, values of 64), layer 1 the same over layer 0's
+# keys and values, layers 3 and 6 an attention without norm and gate (keys and values of 128), layers 2, 4 and 7 a matrix
+# memory with the heads of the Duzinex decoder's retention. Half of each attention head is rotated, nothing has a window.
+# Beside it the closest existing designs at equal sizes: Fotulix (grouped-query attention between two norms), Duzinex (its
+# retention is the matrix memory without gates and normaliser) and Llama.
+LAZULIX_SIZES = {
+    # (attention: heads, kv heads, dim, vdim), (attention_2: the same)
+    "1k": dict(att=(8, 2, 128, 128), att2=(8, 2, 128, 64)),
+    "2k": dict(att=(16, 4, 128, 128), att2=(16, 4, 128, 64)),
+    "4k": dict(att=(32, 8, 128, 128), att2=(32, 8, 128, 64)),
+}
+LAZULIX_LAYERS = ("attention_2", "shared", "mlstm", "attention", "mlstm", "attention_2", "attention", "mlstm")
+
+
+def lazulix_config(size: dict, lz: dict) -> dict:
+    W, ff = size["width"], size["ff"]
+    rh, rd, rvd = size["ret"]
+
+    def att(h, g, d, vd):
+        return dict(heads=h, kv_heads=g, dim=d, vdim=vd, scale=d ** -0.5,
+                    rot=dict(dims=d // 2, base=500000.0, scaling=dict(factor=4.0, original=4096, fast=32.0, slow=1.0)))
+    mixers = dict(mlstm=("mlstm", dict(heads=rh, dim=rd, vdim=rvd, gate_cap=15.0)), attention=("attention", att(*lz["att"])),
+                  attention_2=("attention_2", att(*lz["att2"])), shared=("attention_2", dict(att(*lz["att2"]), kv_from=0)))
+    layers = [dict(type=mixers[k][0], mixer=mixers[k][1], mlp=dict(kind="dense", ff=ff, limit=7.0)) for k in LAZULIX_LAYERS]
+    return dict(architecture="Lazulix", vocab=DESIGN_VOCAB, width=W, norm=dict(eps=1e-6), embedding=dict(scale=W ** 0.5), layers=layers)
+
+
 def design_compare(args) -> int:
     """Prefill (one 2,048-token prompt) and decode (batch 8 behind such prompts) of the Duzinex decoder and of the
     Llama decoder with the same width, feed-forward size and number of layer runs; per-phase device times of both
@@ -381,7 +410,8 @@ def design_compare(args) -> int:
         size = DESIGN_SIZES[name]
         dz = (duzinex_config(size) if design == "duzinex" else gozatar_config(size, GOZATAR_SIZES[name]) if design == "gozatar"
               else kugirax_config(size, KUGIRAX_SIZES[name]) if design == "kugirax"
-              else fotulix_config(size, FOTULIX_SIZES[name]) if design == "fotulix" else luvavik_config(size, LUVAVIK_SIZES[name]))
+              else fotulix_config(size, FOTULIX_SIZES[name]) if design == "fotulix" else luvavik_config(size, LUVAVIK_SIZES[name]) if design == "luvavik"
+              else lazulix_config(size, LAZULIX_SIZES[name]))
         runs = len(config_from_dict(dz).to_spec().schedule)
         row = {}
         arms = [(design, dz), ("llama", llama_config_like(size, runs))]
@@ -391,6 +421,9 @@ def design_compare(args) -> int:
         if design == "luvavik":
             arms[1:1] = [("kugirax", kugirax_config_like_luvavik(size, LUVAVIK_SIZES[name])), ("duzinex", duzinex_config(size))]
             out["beside"] = "kugirax, duzinex, llama"
+        if design == "lazulix":
+            arms[1:1] = [("fotulix", fotulix_config(size, FOTULIX_SIZES[name])), ("duzinex", duzinex_config(size))]
+            out["beside"] = "fotulix, duzinex, llama"
         for label, cfg_dict in arms:
             cfg = config_from_dict(cfg_dict)
             engine = Engine.from_config(cfg, seed=0, dtype=args.dtype, max_tokens=B * (T + 128), max_seqs=B, device="cuda:0")
@@ -466,7 +499,8 @@ def design_compare(args) -> int:
                             else gozatar_rooflines(size, GOZATAR_SIZES[name], row, T, peaks, eb) if design == "gozatar"
                             else kugirax_rooflines(size, KUGIRAX_SIZES[name], row, T, peaks, eb) if design == "kugirax"
                             else fotulix_rooflines(size, FOTULIX_SIZES[name], row, T, B, peaks, eb) if design == "fotulix"
-                            else luvavik_rooflines(size, LUVAVIK_SIZES[name], row, T, B, peaks, eb))
+                            else luvavik_rooflines(size, LUVAVIK_SIZES[name], row, T, B, peaks, eb) if design == "luvavik"
+                            else lazulix_rooflines(size, LAZULIX_SIZES[name], row, T, B, peaks, eb))
         out["sizes"][name] = row
     print(json.dumps(out))
     return 0
@@ -724,6 +758,65 @@ def luvavik_rooflines(size, lv, row, T, B, peaks, eb) -> dict:
     return out
 
 
+def lazulix_rooflines(size, lz, row, T, B, peaks, eb) -> dict:
+    """The same for the Lazulix decoder's kernel groups of a prompt step and of a decode step (sums over its eight layers),
+    beside the like groups of Fotulix, of the Duzinex decoder's retention and of Llama."""
+    W, ff = size["width"], size["ff"]
+    rh, rd, rvd = size["ret"]
+    (h, g, d, vd), (h2, g2, d2, vd2) = lz["att"], lz["att2"]
+    fx = FOTULIX_SIZES[{1024: "1k", 2048: "2k", 4096: "4k"}[W]]["att"]
+    lp, fp, dp, ll = (row[k]["prefill_phases_ms"] for k in ("lazulix", "fotulix", "duzinex", "llama"))
+    ld, dd = row["lazulix"]["decode_phases_ms"], row["duzinex"]["decode_phases_ms"]
+    tf, bw = peaks["bf16_tflops"] * 1e12, peaks["hbm_gbs"] * 1e9
+    kinds = LAZULIX_LAYERS
+    L, n_m, n_a, n_2, n_s = len(kinds), kinds.count("mlstm"), kinds.count("attention"), kinds.count("attention_2"), kinds.count("shared")
+    causal = T * (T + 1) / 2
+    frac = lambda work, peak, ms: round(work / (ms * 1e-3) / peak, 4) if ms else None
+    out = {}
+
+    def put(label, ms, work, peak):
+        out[label] = dict(ms=ms, frac=frac(work, peak, ms))
+    # what a matrix memory has to move: its 32-bit projected rows in, its output out; per token and head d·vd MACs into the
+    # state and d·vd MACs out of it (the least any form does); a decode step reads and writes every state
+    rows = lambda extra: T * (2 * rh * rd + 2 * rh * rvd + extra) * 4.0 + T * rh * rvd * eb
+    put("mlstm (hbm)", lp.get("mlstm_ms"), n_m * rows(2 * rh), bw)
+    put("mlstm (tensor)", lp.get("mlstm_ms"), n_m * T * rh * 4.0 * rd * rvd, tf)
+    put("duzinex retention (hbm)", dp.get("retention_ms"), 2 * rows(0), bw)
+    put("duzinex retention (tensor)", dp.get("retention_ms"), 2 * T * rh * 4.0 * rd * rvd, tf)
+    put("mlstm decode (hbm)", ld.get("mlstm_ms"), n_m * B * rh * rd * rvd * 8.0, bw)
+    put("duzinex retention decode (hbm)", dd.get("retention_ms"), 2 * B * rh * rd * rvd * 8.0, bw)
+    put("attention (tensor)", lp.get("attention_ms"), 2.0 * causal * (n_a * h * (d + vd) + (n_2 + n_s) * h2 * (d2 + vd2)), tf)
+    put("fotulix attention with a sink (tensor)", fp.get("attention_ms"), len(FOTULIX_SINK) * 4.0 * causal * fx[2] * fx[0], tf)
+    nh, nkv, hd = size["llama"]
+    runs = row["llama"]["layer_runs"]
+    put("llama attention (tensor)", ll.get("attention_ms"), runs * 4.0 * causal * hd * nh, tf)
+    kv1, kv2 = g * (d + vd), g2 * (d2 + vd2)
+    put("attention decode (hbm)", ld.get("attention_ms"), B * T * (n_a * kv1 + (n_2 + n_s) * kv2) * eb, bw)
+    put("llama attention decode (hbm)", row["llama"]["decode_phases_ms"].get("attention_ms"), B * T * runs * 2 * nkv * hd * eb, bw)
+    C1, C2 = h * d + kv1, h2 * d2 + kv2
+    put("bias+norm+rotation+store (hbm)", lp.get("rotary+kv_append_ms"), T * (n_a * C1 + n_2 * C2 + n_s * h2 * d2) * (4.0 + eb), bw)
+    fC = (fx[0] + 2 * fx[1]) * fx[2]
+    n_fx = FOTULIX_LAYERS - len(FOTULIX_LATENT)
+    put("fotulix bias+factor+rotation+store (hbm)", fp.get("rotary+kv_append_ms"), n_fx * T * ((fC + fx[0]) * 4.0 + fC * eb + fx[0] * 4.0), bw)
+    put("element gates (hbm)", lp.get("element_gate_ms"), (n_2 + n_s) * T * h2 * vd2 * (2 * eb + 4.0), bw)
+    put("fotulix head gates (hbm)", fp.get("head_gate_ms"), n_fx * T * fx[0] * fx[2] * 2 * eb, bw)
+    post = lambda p: (p.get("attention_out_norm+mlp_norm_ms") or 0) + (p.get("out_norm_ms") or 0)
+    put("layer norms into the stream (hbm)", post(lp), T * W * (L * 2 * 4 * 4.0 + (2 * L - 1) * eb), bw)
+    put("fotulix rms norms into the stream (hbm)", post(fp) + (fp.get("side_out_norm_ms") or 0),
+        T * W * (FOTULIX_LAYERS * (3 * 4 * 4.0 + 2 * eb) + (FOTULIX_LAYERS - 1) * eb), bw)
+    for label, phases, n in (("feed-forward", lp, L), ("fotulix feed-forward", fp, FOTULIX_LAYERS), ("llama feed-forward", ll, runs)):
+        ms = sum(v for k, v in phases.items() if "gate_projection" in k or "down_projection" in k)
+        put(label + " (tensor)", ms, n * T * 3 * 2.0 * W * ff, tf)
+    # a decode step: every weight once, the cached keys and values of every run, the states in and out
+    lat = sum(FOTULIX_SIZES[{1024: "1k", 2048: "2k", 4096: "4k"}[W]]["lat"][i] for i in (2, 4))
+    put("lazulix decode step (hbm)", row["lazulix"]["decode_ms_per_step"], row["lazulix"]["weight_gb"] * 1e9
+        + B * T * (n_a * kv1 + (n_2 + n_s) * kv2) * eb + n_m * B * rh * rd * rvd * 8.0, bw)
+    put("fotulix decode step (hbm)", row["fotulix"]["decode_ms_per_step"], row["fotulix"]["weight_gb"] * 1e9
+        + B * T * n_fx * 2 * fx[1] * fx[2] * eb + B * len(FOTULIX_LATENT) * min(T, DESIGN_WINDOW) * lat * eb, bw)
+    put("llama decode step (hbm)", row["llama"]["decode_ms_per_step"], row["llama"]["weight_gb"] * 1e9 + B * T * runs * 2 * nkv * hd * eb, bw)
+    return out
+
+
 def kernel_case(name: str, reps: int) -> int:
     """One kernel of the step alone, at the 1B shape, on rotating buffers larger than L2.
 
@@ -760,13 +853,14 @@ def kernel_case(name: str, reps: int) -> int:
         torch.cuda.synchronize()
         print(json.dumps({"kernel_case": name, "launches": K.launches}))
         return 0
-    if name in ("fotulix_step", "luvavik_step"):
-        # the Fotulix / Luvavik decoder at the 2k size of --design: one prompt of 2,048 tokens, then three decode steps, kernel
+    if name in ("fotulix_step", "luvavik_step", "lazulix_step"):
+        # the Fotulix / Luvavik / Lazulix decoder at the 2k size of --design: one prompt of 2,048 tokens, then three decode steps, kernel
         # by kernel (no CUDA graph): the launch list of this run is what profiles/*_step_and_kernels.md summarises
         from spissa_b200 import Engine
         from spissa_b200.config import config_from_dict
         cfg = config_from_dict(fotulix_config(DESIGN_SIZES["2k"], FOTULIX_SIZES["2k"]) if name == "fotulix_step"
-                               else luvavik_config(DESIGN_SIZES["2k"], LUVAVIK_SIZES["2k"]))
+                               else luvavik_config(DESIGN_SIZES["2k"], LUVAVIK_SIZES["2k"]) if name == "luvavik_step"
+                               else lazulix_config(DESIGN_SIZES["2k"], LAZULIX_SIZES["2k"]))
         eng = Engine.from_config(cfg, seed=0, dtype="bfloat16", max_tokens=T + 128, max_seqs=1, use_graphs=False)
         rng = random.Random(0)
         sl = eng.acquire()
@@ -1284,6 +1378,62 @@ def kernel_case(name: str, reps: int) -> int:
                 bytes_ = len({e for e in ids.flatten().tolist() if e < E}) * 2.0 * F * Wd * 2
             else:
                 flops = int((ids < E).sum()) * 2 * 2.0 * Wd * F
+    elif name in ("mlstm_chunks", "mlstm_step", "attention_kv", "attention_kv_decode_b8", "qkv_norm_rot_store", "stream_layernorm_add"):
+        # the Lazulix kernels at the 2k size of --design (8 memories of 128 x 256; 16 heads on 4 kv heads, keys of 128 with
+        # half of them rotated, values of 64; width 2,048)
+        Wd, MH, Md, Mv = 2048, 8, 128, 256
+        FH, FG, Fd, Fv = 16, 4, 128, 64
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+        B = 8 if name in ("mlstm_step", "attention_kv_decode_b8") else 1
+        n_new = 1 if B > 1 else T
+        ar = torch.arange(B, dtype=torch.int32, device=dev)
+        pos = (torch.arange(n_new, dtype=torch.int32, device=dev) + (T - n_new)).repeat(B)
+        step = SimpleNamespace(seq_start=i32([n_new * b for b in range(B + 1)]), seq_slot=ar, token_seq=ar.repeat_interleave(n_new),
+                               n_seqs=B, positions=pos, all_single=n_new == 1, max_new=n_new, max_len=T, seq_len=i32([T] * B),
+                               host=dict(new_counts=[n_new] * B))
+        rows = B * n_new
+        if name.startswith("mlstm"):
+            n_buf = 20 if B > 1 else 6                           # a decode step's states are 8 MB: rotate them
+            ld = 2 * MH * (Md + Mv + 1)
+            projs = [torch.randn(rows, ld, device=dev) for _ in range(n_buf)]
+            states = [torch.zeros(B, MH, Md, Mv, device=dev) for _ in range(n_buf)]
+            nms = [torch.zeros(B, MH, Md + 1, device=dev) for _ in range(n_buf)]
+            w = dict(ib=torch.zeros(MH, device=dev), fb=torch.full((MH,), 3.0, device=dev), norm=torch.ones(MH * Mv, device=dev))
+            out = torch.empty(rows, MH * Mv, dtype=bf, device=dev)
+            run = lambda i: K.mlstm(projs[i % n_buf], w, states[i % n_buf], nms[i % n_buf], out, step, MH, Md, Mv, 15.0, 1e-6)
+            bytes_ = rows * (ld * 4.0 + MH * Mv * 2.0) + (B * MH * Md * Mv * 8.0 if B > 1 else 0.0)
+        elif name == "stream_layernorm_add":
+            xs = [torch.randn(T, Wd, device=dev) for _ in range(6)]
+            ys = [torch.randn(T, Wd, device=dev) for _ in range(6)]
+            w1, w2 = torch.randn(Wd, device=dev), torch.randn(Wd, device=dev)
+            out = torch.empty(T, Wd, dtype=bf, device=dev)
+            run = lambda i: K.stream_norm_add(xs[i % 6], ys[i % 6], w1, 1.0, 1e-6, w_next=w2, out=out, centered=True)
+            bytes_ = T * Wd * (4 * 4.0 + 2.0)
+        else:
+            pages = B * (T // 64)
+            table = torch.arange(pages, dtype=torch.int32, device=dev).view(B, T // 64)
+            meta = SimpleNamespace(page_table=table, page_size=64, seq_slot=ar, positions=pos, token_seq=step.token_seq)
+            n_buf = 16 if B > 1 else 4
+            kps, vps = [rnd(pages, FG, 64, Fd) for _ in range(n_buf)], [rnd(pages, FG, 64, Fv) for _ in range(n_buf)]
+            if name == "qkv_norm_rot_store":
+                C = (FH + FG) * Fd + FG * Fv
+                projs = [torch.randn(T, C + FH * Fv, device=dev) for _ in range(6)]
+                bias, qw, kw = rnd(C), rnd(Fd), rnd(Fd)
+                freq = (10000.0 ** (-torch.arange(0, Fd // 2, 2, device=dev).float() / (Fd // 2))).contiguous()
+                q = torch.empty(T, FH * Fd, dtype=bf, device=dev)
+                run = lambda i: K.qkv_norm_rot_store(projs[i % 6], bias, q, kps[i % n_buf], vps[i % n_buf], meta, freq, FH, FG, Fd, Fv,
+                                                     Fd // 2, q_weight=qw, k_weight=kw, eps=1e-6, rot_mult=1.1)
+                bytes_ = T * C * (4.0 + 2.0)
+            else:
+                from spissa_b200.parts.attention import attend_paged
+                qs = [rnd(rows, FH * Fd) for _ in range(4)]
+                cnt = torch.zeros(4096, dtype=torch.int32, device=dev)
+                views = [SimpleNamespace(k_pool=k, v_pool=v, **vars(meta)) for k, v in zip(kps, vps)]
+                run = lambda i: attend_paged(qs[i % 4], step, views[i % n_buf], FH, FG, Fd, None, Fd ** -0.5, counters=cnt, vd=Fv)
+                if B > 1:
+                    bytes_ = B * T * FG * (Fd + Fv) * 2.0
+                else:
+                    flops = 2.0 * T * (T + 1) / 2 * (Fd + Fv) * FH
     elif name in ("sample_b8", "sample_b64", "argmax_b8"):
         # the sampler on rows of 128,256 logits (standard deviation 4 after the temperature): temperature 0.8, top-p 0.95
         B = 64 if name.endswith("b64") else 8
@@ -1346,7 +1496,7 @@ def main() -> int:
     ap.add_argument("--kernel-case", default=None,
                     help="time one kernel alone (gemm_qkv|gemm_o|gemm_gate_up|gemm_down|gemv_qkv|gemv_o|gemv_gate_up|"
                          "gemv_down|gemv_head|diff_flash|diff_decode|retention_chunks|retention_step|mingru_chunks|polynorm|token_shift|gla_chunks|gla_step|moe_experts|moe_experts_b8|streams_norm|conv_qk_store|stream_qkv|stream_o|stream_gate_up|stream_down|stream_fused_qkv|stream_fused_o|stream_fused_gate_up|stream_fused_down|flash_prefill[_128]|flash_prefill_tc[_128]|flash_decode[_b64]|sample_b8|sample_b64|argmax_b8|decode_layers|step_b8|prefill|fused_qkv|fused_o|fused_gate_up|fused_down) instead of the step")
-    ap.add_argument("--design", default=None, choices=["duzinex", "gozatar", "kugirax", "fotulix", "luvavik"],
+    ap.add_argument("--design", default=None, choices=["duzinex", "gozatar", "kugirax", "fotulix", "luvavik", "lazulix"],
                     help="measure this design beside the Llama decoder at equal layer sizes instead of the headline workload")
     ap.add_argument("--design-sizes", default="", dest="design_sizes", help="which of 1k,2k,4k (default: all)")
     ap.add_argument("--reps", type=int, default=20)

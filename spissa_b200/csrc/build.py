@@ -21,7 +21,7 @@ import time
 from pathlib import Path
 
 CSRC = Path(__file__).resolve().parent
-HEADERS = ["common.cuh", "async_copy.cuh", "tcgen05.cuh", "flash_common.cuh", "attention_noalloc.h"]
+HEADERS = ["common.cuh", "async_copy.cuh", "tcgen05.cuh", "flash_common.cuh", "flash_paged.cuh", "attention_noalloc.h"]
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
     "-O3", "-std=c++17", "-lineinfo", "--shared",
@@ -48,6 +48,7 @@ MODULES = {
     "sampling": "sampling_kernels.cu",
     "tc_gemm": "tc_gemm.cu",
     "attention": "attention_kernels.cu",
+    "attention_kv": "attention_kv_kernels.cu",
     "gemv": "gemv_kernels.cu",
     "flash_tc": "flash_tc.cu",
     "decode_layers": "decode_layers.cu",
@@ -59,6 +60,7 @@ MODULES = {
     "latent": "latent_kernels.cu",
     "sandwich": "sandwich_kernels.cu",
     "rglru": "rglru_kernels.cu",
+    "mlstm": "mlstm_kernels.cu",
 }
 
 

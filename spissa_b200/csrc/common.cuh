@@ -49,16 +49,28 @@ __device__ __forceinline__ void sp_st_dt(void* p, int dt, size_t i, float v) {
 }
 
 // ---------------------------------------------------------------- activations of gated units
-// What a product's epilogue applies: silu(gate)·up, gelu(gate)·up, or (plain rows) the square of relu.
-enum { SP_ACT_SILU = 0, SP_ACT_GELU = 1, SP_ACT_RELU2 = 2 };
+// What a product's epilogue applies: silu(gate)·up, gelu(gate)·up, the clamped unit g·sigmoid(slope·g)·(u + 1) with
+// g = min(gate, limit) and u = clamp(up, ±limit), or (plain rows) the square of relu; times ``mult``.
+enum { SP_ACT_SILU = 0, SP_ACT_GELU = 1, SP_ACT_RELU2 = 2, SP_ACT_CLAMPED = 3 };
+struct SpGate {
+    int kind = SP_ACT_SILU;
+    float mult = 1.0f, limit = 0.0f, slope = 0.0f;
+};
+static inline bool sp_gate_built(const SpGate& g) { return g.kind == SP_ACT_SILU || g.kind == SP_ACT_GELU || (g.kind == SP_ACT_CLAMPED && g.limit > 0.0f); }
 
 // The tanh form of gelu, ½ z (1 + tanh(a)) with a = √(2/π)(z + 0.044715 z³), written with the logistic function:
 // ½ (1 + tanh(a)) = 1 / (1 + e^{−2a}).
 __device__ __forceinline__ float sp_gelu_tanh(float z) {
     return z / (1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
 }
-__device__ __forceinline__ float sp_gated(float gate, float up, int act) {
-    return (act == SP_ACT_GELU ? sp_gelu_tanh(gate) : gate / (1.0f + expf(-gate))) * up;
+__device__ __forceinline__ float sp_gated(float gate, float up, const SpGate& ga) {
+    float slope = 1.0f;
+    if (ga.kind == SP_ACT_CLAMPED) {
+        gate = fminf(gate, ga.limit);
+        up = fminf(fmaxf(up, -ga.limit), ga.limit) + 1.0f;
+        slope = ga.slope;
+    }
+    return (ga.kind == SP_ACT_GELU ? sp_gelu_tanh(gate) : gate / (1.0f + expf(-slope * gate))) * up * ga.mult;
 }
 __device__ __forceinline__ float sp_relu2(float z) {
     const float r = fmaxf(z, 0.0f);

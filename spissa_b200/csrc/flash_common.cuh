@@ -47,14 +47,16 @@ struct Tile {
 };
 
 // Copy rows [0, n_rows) x HD of a bfloat16 matrix with row stride ``ld`` (elements) into a padded
-// shared tile; rows from n_rows to 64 are zeroed. All ``nthreads`` threads take part.
+// shared tile; rows from n_rows to 64 are zeroed. All ``nthreads`` threads take part. ``cols``: entries that a row has
+// (a multiple of 8; the tile's columns beyond them are left as they are).
 template <int HD>
 __device__ __forceinline__ void load_tile_async(uint32_t dst, const __nv_bfloat16* src, size_t ld, int n_rows,
-                                                int tid, int nthreads) {
+                                                int tid, int nthreads, int cols = HD) {
     using T = Tile<HD>;
     for (int c = tid; c < KT * T::CHUNKS; c += nthreads) {
         const int r = c / T::CHUNKS, k = c % T::CHUNKS;
         const uint32_t d = dst + r * T::ROW + k * 16;
+        if (k * 8 >= cols) continue;
         if (r < n_rows) cp_async16(d, src + (size_t)r * ld + k * 8);
         else asm volatile("st.shared.v4.b32 [%0], {%1,%1,%1,%1};" ::"r"(d), "r"(0u) : "memory");
     }
@@ -63,13 +65,14 @@ __device__ __forceinline__ void load_tile_async(uint32_t dst, const __nv_bfloat1
 // One warp, 16 query rows (fragments ``qf``), keys [key0, key0 + 8*NT) of the tile in shared memory.
 // Row ``g`` of the fragment sees keys lo[0]..hi[0], row g+8 keys lo[1]..hi[1] (absolute positions);
 // with MASKED false the caller vouches that every key of the tile is visible to every row.
-// m holds the running maximum of the raw scores times scale_log2 (the log2 domain).
-template <int HD, int NT, bool MASKED>
+// m holds the running maximum of the raw scores times scale_log2 (the log2 domain). VD: the size of a value row.
+template <int HD, int NT, bool MASKED, int VD = HD>
 __device__ __forceinline__ void flash_step(const uint32_t (&qf)[HD / 16][4], uint32_t k_tile, uint32_t v_tile,
                                            int key0, int tile_pos0, const int (&lo)[2], const int (&hi)[2],
-                                           float scale_log2, float (&o)[HD / 8][4], float (&m)[2], float (&l)[2],
+                                           float scale_log2, float (&o)[VD / 8][4], float (&m)[2], float (&l)[2],
                                            int lane, const float* __restrict__ bias_row = nullptr, int bias_cap = 0) {
     using T = Tile<HD>;
+    using TV = Tile<VD>;
     float s[NT][4];
 #pragma unroll
     for (int i = 0; i < NT; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
@@ -156,7 +159,7 @@ __device__ __forceinline__ void flash_step(const uint32_t (&qf)[HD / 16][4], uin
     l[0] = l[0] * corr[0] + sum[0];                   // per-lane partial; lanes are summed at the end
     l[1] = l[1] * corr[1] + sum[1];
 #pragma unroll
-    for (int i = 0; i < HD / 8; ++i) {
+    for (int i = 0; i < VD / 8; ++i) {
         o[i][0] *= corr[0]; o[i][1] *= corr[0];
         o[i][2] *= corr[1]; o[i][3] *= corr[1];
     }
@@ -169,11 +172,11 @@ __device__ __forceinline__ void flash_step(const uint32_t (&qf)[HD / 16][4], uin
         a[2] = pack_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1]);
         a[3] = pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3]);
 #pragma unroll
-        for (int dp = 0; dp < HD / 16; ++dp) {
+        for (int dp = 0; dp < VD / 16; ++dp) {
             const int key = key0 + kk * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
             const int d = dp * 16 + ((lane >> 4) << 3);
             uint32_t b0, b1, b2, b3;
-            ldmatrix_x4_trans(v_tile + key * T::ROW + d * 2, b0, b1, b2, b3);
+            ldmatrix_x4_trans(v_tile + key * TV::ROW + d * 2, b0, b1, b2, b3);
             mma_bf16(o[2 * dp], a, b0, b1);
             mma_bf16(o[2 * dp + 1], a, b2, b3);
         }
@@ -196,13 +199,14 @@ __device__ __forceinline__ uint32_t movmatrix_trans(uint32_t a) {   // the 8x8 m
 // the 8 lanes that share t. It moves only when a score exceeds it by more than 8 (then the lanes agree on the
 // new maximum and rescale o and l); otherwise P = 2^(s - m) ≤ 256 and no lane talks to another. The result
 // o / l does not depend on the reference. ``l`` is per lane (its own keys); the caller adds the lanes.
-template <int HD, int NH, bool MASKED>
+template <int HD, int NH, bool MASKED, int VD = HD>
 __device__ __forceinline__ void decode_step_t(const uint32_t (&qb)[HD / 16][NH][2], uint32_t k_tile, uint32_t v_tile,
                                               int key0, int tile_pos0, int lo, int hi, float scale_log2,
-                                              float (&o)[HD / 16][NH][4], float (&m)[NH][2], float (&l)[NH][2],
+                                              float (&o)[VD / 16][NH][4], float (&m)[NH][2], float (&l)[NH][2],
                                               int lane, const float* __restrict__ bias_group = nullptr, int bias_cap = 0,
                                               int group_heads = 0) {
     using T = Tile<HD>;
+    using TV = Tile<VD>;
     const int g = lane >> 2;
     float s[NH][4], s2[NH][4];                        // two chains of products: an mma need not wait for the one before
 #pragma unroll
@@ -253,7 +257,7 @@ __device__ __forceinline__ void decode_step_t(const uint32_t (&qb)[HD / 16][NH][
                 m[i][c] = mnew;
                 l[i][c] *= corr;
 #pragma unroll
-                for (int dt = 0; dt < HD / 16; ++dt) { o[dt][i][c] *= corr; o[dt][i][c + 2] *= corr; }
+                for (int dt = 0; dt < VD / 16; ++dt) { o[dt][i][c] *= corr; o[dt][i][c + 2] *= corr; }
             }
         }
     }
@@ -269,9 +273,9 @@ __device__ __forceinline__ void decode_step_t(const uint32_t (&qb)[HD / 16][NH][
         pb[i][1] = movmatrix_trans(pack_bf16(p2, p3));            // keys key0 + 8 .. +15
     }
 #pragma unroll
-    for (int dt = 0; dt < HD / 16; ++dt) {
+    for (int dt = 0; dt < VD / 16; ++dt) {
         uint32_t a[4];
-        ldmatrix_x4_trans(v_tile + (key0 + (lane & 7) + ((lane >> 4) << 3)) * T::ROW + (dt * 16 + (((lane >> 3) & 1) << 3)) * 2,
+        ldmatrix_x4_trans(v_tile + (key0 + (lane & 7) + ((lane >> 4) << 3)) * TV::ROW + (dt * 16 + (((lane >> 3) & 1) << 3)) * 2,
                           a[0], a[1], a[2], a[3]);
 #pragma unroll
         for (int i = 0; i < NH; ++i) mma_bf16(o[dt][i], a, pb[i][0], pb[i][1]);

@@ -67,7 +67,9 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
                         const int* __restrict__ seq_row, const int* __restrict__ page_table, int max_pages,
                         int n_seqs, int nh, int nkv, float scale_log2, int* status, SpRange rg,
                         const float* __restrict__ sink, int window, int rows_mode,
-                        const float* __restrict__ dist_bias, int dist_cap) {
+                        const float* __restrict__ dist_bias, int dist_cap, int d, int vd) {
+    // d, vd: the sizes of a head's key and value rows, at most HD and HDV. Where they are smaller the key and value maps end
+    // at them and the copies fill the boxes up with zeros (the query boxes then hold some of the next head: times zero).
     static_assert((HD == 64 || HD == 128 || HD == 192) && (HDV == 64 || HDV == 128),
                   "scores 2 x 64 columns and the output HDV columns of 256 in tensor memory");
     using L = Smem<HD, HDV>;
@@ -143,7 +145,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         if (lane == 0 && live) {
             mbar_expect_tx(smem_u32(&bar_q), L::Q_BYTES);
 #pragma unroll
-            for (int c = 0; c < L::BOXES; ++c) tma_load_2d(q_smem + c * L::Q_BOX, &map_q, h * HD + c * 64, t0, smem_u32(&bar_q));
+            for (int c = 0; c < L::BOXES; ++c) tma_load_2d(q_smem + c * L::Q_BOX, &map_q, h * d + c * 64, t0, smem_u32(&bar_q));
             for (int j = 0; j < n_blocks; ++j) {
                 const int s = j % KV_STAGES;
                 const uint32_t phase = (uint32_t)(j / KV_STAGES) & 1u;
@@ -312,7 +314,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         if (ok && !(status && *(volatile int*)status != 0)) {
             // a sink: one more term in the denominator, with no key and no value (m and the sink's score in log2 units)
             const float inv = 1.0f / (sink ? l + exp2f(sink[h] * LOG2E - m) : l);
-            __nv_bfloat16* dst = out + (size_t)(t0 + row) * nh * HDV + (size_t)h * HDV;
+            __nv_bfloat16* dst = out + (size_t)(t0 + row) * nh * vd + (size_t)h * vd;
 #pragma unroll 1
             for (int c0 = 0; c0 < HDV; c0 += 32) {
                 uint32_t r[32];
@@ -321,6 +323,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
                 if (row < n_rows) {
 #pragma unroll
                     for (int i = 0; i < 32; i += 8) {
+                        if (c0 + i >= vd) break;
                         uint4 w;
                         __nv_bfloat162 a0 = __floats2bfloat162_rn(__uint_as_float(r[i]) * inv, __uint_as_float(r[i + 1]) * inv);
                         __nv_bfloat162 a1 = __floats2bfloat162_rn(__uint_as_float(r[i + 2]) * inv, __uint_as_float(r[i + 3]) * inv);
@@ -378,9 +381,12 @@ int make_map(CUtensorMap* map, const void* ptr, long long rows, int cols, long l
 // Query rows per CTA: the host counts tiles (the grid) with it.
 SP_API int sp_flash_tc_query_tile() { return QT; }
 
+SP_API int sp_flash_tc_kv_supported(int d, int vd, int nh, int nkv, int page_size) {
+    return d > 32 && d <= 192 && d % 8 == 0 && vd >= 8 && vd <= 128 && vd % 8 == 0 && nkv > 0 && nh % nkv == 0 && page_size == PAGE;
+}
 SP_API int sp_flash_tc_supported(int hd, int nh, int nkv, int page_size, int window) {
     (void)window;                                                // any window, or none
-    return (hd == 64 || hd == 128) && nkv > 0 && nh % nkv == 0 && page_size == PAGE;
+    return sp_flash_tc_kv_supported(hd, hd, nh, nkv, page_size);
 }
 
 namespace {
@@ -389,7 +395,7 @@ template <int HD, int HDV = HD>
 int launch_flash_tc(dim3 grid, cudaStream_t stream, const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, void* out,
                     const int* seq_start, const int* positions, const int* seq_row, const int* page_table, int max_pages,
                     int n_seqs, int nh, int nkv, float scale, int* status, const float* sink, int window, int rows_mode,
-                    const float* dist_bias = nullptr, int dist_cap = 0) {
+                    const float* dist_bias = nullptr, int dist_cap = 0, int d = HD, int vd = HDV) {
     static SpPerDevice configured;
     if (!configured.done()) {
         cudaError_t e = cudaFuncSetAttribute(flash_prefill_tc_kernel<HD, HDV>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<HD, HDV>::TOTAL);
@@ -398,39 +404,49 @@ int launch_flash_tc(dim3 grid, cudaStream_t stream, const CUtensorMap& mq, const
     }
     SP_CHECK_CALL("flash_prefill_tc", sp_launch_dependent(flash_prefill_tc_kernel<HD, HDV>, grid, dim3(192), (size_t)Smem<HD, HDV>::TOTAL, stream,
         mq, mk, mv, (__nv_bfloat16*)out, seq_start, positions, seq_row, page_table, max_pages, n_seqs, nh, nkv,
-        scale * LOG2E, status, sp_range_host, sink, window, rows_mode, dist_bias, dist_cap));
+        scale * LOG2E, status, sp_range_host, sink, window, rows_mode, dist_bias, dist_cap, d, vd));
     SP_CHECK_LAUNCH("flash_prefill_tc");
     return 0;
 }
 
 }  // namespace
 
-// q, out: [T, nh*hd] bfloat16; pools: [n_pages, nkv, 64, hd] bfloat16; n_q_tiles = sum over sequences of
-// ceil(new tokens / 128). ``window`` w > 0: a query at position i sees the keys i - w < j <= i.
+// q: [T, nh*d], out: [T, nh*vd] bfloat16; pools: [n_pages, nkv, 64, d] and [n_pages, nkv, 64, vd] bfloat16; n_q_tiles = sum
+// over sequences of ceil(new tokens / 128). ``window`` w > 0: a query at position i sees the keys i - w < j <= i.
 // ``sink`` (float32 per query head, or null): a score that joins every row's denominator once, with no key and no value
 // ``dist_bias`` (float32 [nh][dist_cap + 1], or null): a score added by the distance between query and key
+SP_API int sp_flash_prefill_tc_kv(const void* q, void* out, const void* kpool, const void* vpool, long long n_pages,
+                                  int T, const int* seq_start, const int* positions, const int* seq_row,
+                                  const int* page_table, int max_pages, int page_size, int n_seqs, int n_q_tiles, int nh,
+                                  int nkv, int d, int vd, int window, float scale, int* status, const float* sink,
+                                  const float* dist_bias, int dist_cap, cudaStream_t stream) {
+    if (n_q_tiles <= 0) return 0;
+    if (dist_bias && dist_cap < 0) SP_FAIL("flash_tc: a distance-bias table needs at least one entry per head");
+    if (!sp_flash_tc_kv_supported(d, vd, nh, nkv, page_size))
+        SP_FAIL("flash_tc: built for keys of 40 to 192 and values of 8 to 128, multiples of 8, and pages of 64 (got %d and %d, page %d)", d, vd, page_size);
+    if (((uintptr_t)q & 15) || ((uintptr_t)kpool & 15) || ((uintptr_t)vpool & 15) || ((uintptr_t)out & 15))
+        SP_FAIL("flash_tc: operands must start on a 16-byte boundary");
+    CUtensorMap mq, mk, mv;
+    if (make_map(&mq, q, T, nh * d, (long long)nh * d, QT)) return 1;
+    if (make_map(&mk, kpool, n_pages * nkv * PAGE, d, d, PAGE)) return 1;
+    if (make_map(&mv, vpool, n_pages * nkv * PAGE, vd, vd, PAGE)) return 1;
+    if (n_q_tiles > 65535) SP_FAIL("flash_tc: %d query tiles are beyond this kernel's grid", n_q_tiles);
+    dim3 grid(nh, n_q_tiles);
+    const int w = window > 0 ? window : 0;
+#define SP_KV_ARGS grid, stream, mq, mk, mv, out, seq_start, positions, seq_row, page_table, max_pages, n_seqs, nh, nkv, scale, status, sink, w, 0, dist_bias, dist_cap, d, vd
+    if (d > 128) return launch_flash_tc<192, 128>(SP_KV_ARGS);
+    if (d > 64) return vd > 64 ? launch_flash_tc<128, 128>(SP_KV_ARGS) : launch_flash_tc<128, 64>(SP_KV_ARGS);
+    return vd > 64 ? launch_flash_tc<64, 128>(SP_KV_ARGS) : launch_flash_tc<64, 64>(SP_KV_ARGS);
+#undef SP_KV_ARGS
+}
+
 SP_API int sp_flash_prefill_tc_bias(const void* q, void* out, const void* kpool, const void* vpool, long long n_pages,
                                     int T, const int* seq_start, const int* positions, const int* seq_row,
                                     const int* page_table, int max_pages, int page_size, int n_seqs, int n_q_tiles, int nh,
                                     int nkv, int hd, int window, float scale, int* status, const float* sink,
                                     const float* dist_bias, int dist_cap, cudaStream_t stream) {
-    if (n_q_tiles <= 0) return 0;
-    if (dist_bias && dist_cap < 0) SP_FAIL("flash_tc: a distance-bias table needs at least one entry per head");
-    if (!sp_flash_tc_supported(hd, nh, nkv, page_size, window))
-        SP_FAIL("flash_tc: built for head sizes 64 and 128 and pages of 64 (got head %d, page %d)", hd, page_size);
-    if (((uintptr_t)q & 15) || ((uintptr_t)kpool & 15) || ((uintptr_t)vpool & 15) || ((uintptr_t)out & 15))
-        SP_FAIL("flash_tc: operands must start on a 16-byte boundary");
-    CUtensorMap mq, mk, mv;
-    if (make_map(&mq, q, T, nh * hd, (long long)nh * hd, QT)) return 1;
-    if (make_map(&mk, kpool, n_pages * nkv * PAGE, hd, hd, PAGE)) return 1;
-    if (make_map(&mv, vpool, n_pages * nkv * PAGE, hd, hd, PAGE)) return 1;
-    if (n_q_tiles > 65535) SP_FAIL("flash_tc: %d query tiles are beyond this kernel's grid", n_q_tiles);
-    dim3 grid(nh, n_q_tiles);
-    const int w = window > 0 ? window : 0;
-    return hd == 64 ? launch_flash_tc<64>(grid, stream, mq, mk, mv, out, seq_start, positions, seq_row, page_table, max_pages,
-                                          n_seqs, nh, nkv, scale, status, sink, w, 0, dist_bias, dist_cap)
-                    : launch_flash_tc<128>(grid, stream, mq, mk, mv, out, seq_start, positions, seq_row, page_table, max_pages,
-                                           n_seqs, nh, nkv, scale, status, sink, w, 0, dist_bias, dist_cap);
+    return sp_flash_prefill_tc_kv(q, out, kpool, vpool, n_pages, T, seq_start, positions, seq_row, page_table, max_pages, page_size,
+                                  n_seqs, n_q_tiles, nh, nkv, hd, hd, window, scale, status, sink, dist_bias, dist_cap, stream);
 }
 
 SP_API int sp_flash_prefill_tc_sink(const void* q, void* out, const void* kpool, const void* vpool, long long n_pages,

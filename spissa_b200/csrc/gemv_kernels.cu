@@ -94,7 +94,7 @@ template <int MT, int RT, int UNROLL>
 __global__ void __launch_bounds__(MAX_KS * 32)
 gemv_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ W, void* __restrict__ out,
             int out_dt, int M, int N, int K, int ldx, int ldw, int ldo, int mode, int pair, int ks, int cs,
-            RopeOut rope, int act, float mult) {
+            RopeOut rope, SpGate ga) {
     __shared__ __align__(16) float red[MAX_KS][MT][RT][32][4];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, t = lane & 3;
@@ -221,7 +221,7 @@ gemv_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict
                     const int col = tile * 8 * HALF + r * 8 + 2 * t + (e & 1);
                     if (col < N / 2) {
                         const float gate = acc[i][r][e], up = acc[i][HALF + r < RT ? HALF + r : r][e];
-                        sp_st_dt(out, out_dt, (size_t)m * ldo + col, sp_gated(gate, up, act) * mult);
+                        sp_st_dt(out, out_dt, (size_t)m * ldo + col, sp_gated(gate, up, ga));
                     }
                 }
             } else if (mode == MODE_ROPE_KV) {
@@ -280,7 +280,7 @@ gemv_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict
 template <int RT, int U>
 __global__ void __launch_bounds__(128)
 gemv_stream_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ W, void* __restrict__ out,
-                   int out_dt, int M, int N, int K, int ldx, int ldw, int ldo, int mode, int pair, int tiles, int act, float mult) {
+                   int out_dt, int M, int N, int K, int ldx, int ldw, int ldo, int mode, int pair, int tiles, SpGate ga) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, t = lane & 3;
     const int tile = blockIdx.x * 4 + warp;
@@ -378,7 +378,7 @@ gemv_stream_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __r
                 const int col = tile * 8 * HALF + r * 8 + 2 * t + (e & 1);
                 if (col < N / 2) {
                     const float gate = acc[r][e], up = acc[HALF + r < RT ? HALF + r : r][e];
-                    sp_st_dt(out, out_dt, (size_t)m * ldo + col, sp_gated(gate, up, act) * mult);
+                    sp_st_dt(out, out_dt, (size_t)m * ldo + col, sp_gated(gate, up, ga));
                 }
             }
         } else {
@@ -430,7 +430,7 @@ SP_API int sp_gemv_supported(const void* x, const void* W, int M, int K, int ldx
 namespace {
 
 int launch_gemv(const void* x, const void* W, void* out, int out_dt, int M, int N, int K, int ldx, int ldw, int ldo,
-                int mode, int pair, const RopeOut& rope, cudaStream_t stream, int act = SP_ACT_SILU, float mult = 1.0f) {
+                int mode, int pair, const RopeOut& rope, cudaStream_t stream, SpGate ga = SpGate{}) {
     const __nv_bfloat16* xp = (const __nv_bfloat16*)x;
     const __nv_bfloat16* wp = (const __nv_bfloat16*)W;
     const int stream_tiles = mode == MODE_SILU_MUL ? (N / 2 + 7) / 8 : (N + 7) / 8;
@@ -438,10 +438,10 @@ int launch_gemv(const void* x, const void* W, void* out, int out_dt, int M, int 
         // enough rows (the output head) to give every warp rows of its own and still fill every SM sixteen warps deep
         if (mode == MODE_SILU_MUL)
             sp_launch_dependent(gemv_stream_kernel<2, 4>, dim3((stream_tiles + 3) / 4), dim3(128), 0, stream, xp, wp, out, out_dt, M,
-                                N, K, ldx, ldw, ldo, mode, pair, stream_tiles, act, mult);
+                                N, K, ldx, ldw, ldo, mode, pair, stream_tiles, ga);
         else
             sp_launch_dependent(gemv_stream_kernel<1, 8>, dim3((stream_tiles + 3) / 4), dim3(128), 0, stream, xp, wp, out, out_dt, M,
-                                N, K, ldx, ldw, ldo, mode, pair, stream_tiles, act, mult);
+                                N, K, ldx, ldw, ldo, mode, pair, stream_tiles, ga);
         SP_CHECK_LAUNCH("gemv_stream");
         return 0;
     }
@@ -449,7 +449,7 @@ int launch_gemv(const void* x, const void* W, void* out, int out_dt, int M, int 
     const dim3 grid(p.tiles * p.cs), block(p.ks * 32);
 #define GV_LAUNCH(MT, RT, UN)                                                                              \
     SP_CHECK_CALL("gemv", sp_launch_cluster(gemv_kernel<MT, RT, UN>, grid, block, 0, stream, p.cs, xp, wp, out, out_dt,  \
-                                            M, N, K, ldx, ldw, ldo, mode, pair, p.ks, p.cs, rope, act, mult))
+                                            M, N, K, ldx, ldw, ldo, mode, pair, p.ks, p.cs, rope, ga))
     if (p.rt == 4) GV_LAUNCH(2, 4, 2);
     else if (p.rt == 2 && M <= 16) GV_LAUNCH(1, 2, 4);
     else if (p.rt == 2) GV_LAUNCH(4, 2, 2);
@@ -479,13 +479,14 @@ SP_API int sp_gemv(const void* x, const void* W, void* out, int out_dt, int M, i
     return launch_gemv(x, W, out, out_dt, M, N, K, ldx, ldw, ldo, mode, pair, RopeOut{}, stream);
 }
 
-// mode 2 with another activation of the gate (SP_ACT_*) and a factor on the outputs
+// mode 2 with another activation of the gate (SP_ACT_*; limit and slope of the clamped one) and a factor on the outputs
 SP_API int sp_gemv_gated(const void* x, const void* W, void* out, int out_dt, int M, int N, int K, int ldx, int ldw,
-                         int ldo, int pair, int act, float mult, cudaStream_t stream) {
+                         int ldo, int pair, int act, float mult, float limit, float slope, cudaStream_t stream) {
     if (N <= 0) return 0;
-    if (act != SP_ACT_SILU && act != SP_ACT_GELU) SP_FAIL("gemv: activation code %d is not built for gated rows", act);
+    const SpGate ga{act, mult, limit, slope};
+    if (!sp_gate_built(ga)) SP_FAIL("gemv: activation code %d is not built for gated rows", act);
     if (check_gemv(x, W, M, N, K, ldx, ldw, out_dt, MODE_SILU_MUL, pair)) return 1;
-    return launch_gemv(x, W, out, out_dt, M, N, K, ldx, ldw, ldo, MODE_SILU_MUL, pair, RopeOut{}, stream, act, mult);
+    return launch_gemv(x, W, out, out_dt, M, N, K, ldx, ldw, ldo, MODE_SILU_MUL, pair, RopeOut{}, stream, ga);
 }
 
 // QKV for decoding in one kernel: W = [Wq; Wk; Wv], rotate-half on q and k in the epilogue, q to ``q_out``
@@ -517,7 +518,7 @@ SP_API int sp_gemv_argmax(const void* x, const void* W, void* cand, int M, int N
     const int tiles = sp_gemv_argmax_candidates(N);
     if (ld_cand < tiles) SP_FAIL("gemv (argmax): the candidate table has %d columns, %d are needed", ld_cand, tiles);
     sp_launch_dependent(gemv_stream_kernel<1, 8>, dim3((tiles + 3) / 4), dim3(128), 0, stream, (const __nv_bfloat16*)x,
-                        (const __nv_bfloat16*)W, cand, (int)SP_DT_F32, M, N, K, ldx, ldw, ld_cand, (int)MODE_ARGMAX, 0, tiles, (int)SP_ACT_SILU, 1.0f);
+                        (const __nv_bfloat16*)W, cand, (int)SP_DT_F32, M, N, K, ldx, ldw, ld_cand, (int)MODE_ARGMAX, 0, tiles, SpGate{});
     SP_CHECK_LAUNCH("gemv_argmax");
     return 0;
 }

@@ -799,7 +799,7 @@ __global__ void gated_mul_kernel(const T* __restrict__ gu, T* __restrict__ out, 
         const int c = (int)(e % I);
         const float g = sp_ld(gu, r * 2 * I + c);
         const float u = sp_ld(gu, r * 2 * I + I + c);
-        sp_st(out, e, sp_gated(g, u, act) * mult);
+        sp_st(out, e, sp_gated(g, u, SpGate{act, mult, 0.0f, 0.0f}));
     }
 }
 

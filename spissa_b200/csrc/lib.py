@@ -44,6 +44,8 @@ def load(module: str) -> ctypes.CDLL:
         getattr(lib, f"sp_{module}_last_error").restype = ctypes.c_char_p
         if module == "seqmix":
             lib.sp_retention_chunked_scratch_floats.restype = c_longlong
+        if module == "mlstm":
+            lib.sp_mlstm_scratch_floats.restype = c_longlong
         if module == "hybrid":
             lib.sp_gla_chunked_scratch_floats.restype = c_longlong
         _LIBS[module] = lib
@@ -244,7 +246,7 @@ def gate_elements(x, z, mult: float = 1.0):
                                            z.stride(0), c_float(mult), c_void_p(_stream())))
 
 
-ACT_SILU, ACT_GELU, ACT_RELU2 = 0, 1, 2       # the kernels' activation codes (common.cuh)
+ACT_SILU, ACT_GELU, ACT_RELU2, ACT_CLAMPED = 0, 1, 2, 3       # the kernels' activation codes (common.cuh)
 
 
 def gated_mul(gu, out, act=ACT_SILU, mult: float = 1.0):
@@ -417,6 +419,10 @@ STATUS_TEXT = {101: "the TMA loader waited too long for a free pipeline stage",
                143: "rglru: the MMA issuer waited too long for a free accumulator",
                144: "rglru: the MMA issuer waited too long for the convolution",
                145: "rglru: the recurrence warps waited too long for the gates",
+               151: "mlstm: the chunks' sums waited too long for their products",
+               152: "mlstm: a stage of the outputs' operands did not become free in time",
+               153: "mlstm: the products with the start states took too long",
+               154: "mlstm: the products with the values took too long",
                301: "embedding: a token id outside the vocabulary",
                401: "range check: a page index from a page table lies beyond the pools",
                402: "range check: a sequence's row lies beyond the page table",
@@ -456,12 +462,14 @@ def tc_gemm_supported(a: torch.Tensor, w: torch.Tensor) -> bool:
 TC_STORE, TC_ACCUMULATE, TC_SILU_MUL = 0, 1, 2
 
 
-def tc_gemm(a, w, out, mode=TC_STORE, bn=128, act=ACT_SILU, mult: float = 1.0):
+def tc_gemm(a, w, out, mode=TC_STORE, bn=128, act=ACT_SILU, mult: float = 1.0, limit: float = 0.0,
+            slope: float = 0.0):
     """out = a · wᵀ on the tcgen05 tensor cores (bfloat16 operands, float32 accumulation).
 
     ``mode`` TC_STORE writes ``out`` (bfloat16 or float32), TC_ACCUMULATE adds into a float32 ``out``,
     TC_SILU_MUL takes a weight whose rows interleave gate and up in blocks of ``bn``/2 and writes
-    silu(gate)·up into ``out`` [M, N/2] (``act`` ACT_GELU: gelu(gate)·up; times ``mult``).
+    silu(gate)·up into ``out`` [M, N/2] (``act`` ACT_GELU: gelu(gate)·up; ACT_CLAMPED: g·sigmoid(slope·g)·(u + 1) with
+    g = min(gate, limit), u = clamp(up, ±limit); times ``mult``).
     """
     lib = load("tc_gemm")
     M, K = a.shape
@@ -474,7 +482,7 @@ def tc_gemm(a, w, out, mode=TC_STORE, bn=128, act=ACT_SILU, mult: float = 1.0):
     if mode == TC_SILU_MUL and (act != ACT_SILU or mult != 1.0):
         _check("tc_gemm", lib.sp_tc_gemm_gated(
             c_void_p(_ptr(a)), c_void_p(_ptr(w)), c_void_p(_ptr(out)), dt_code(out), M, N, K, a.stride(0), w.stride(0),
-            out.stride(0), int(bn), int(act), c_float(mult), c_void_p(_ptr(status_word(a.device))), c_void_p(_stream())))
+            out.stride(0), int(bn), int(act), c_float(mult), c_float(limit), c_float(slope), c_void_p(_ptr(status_word(a.device))), c_void_p(_stream())))
         return
     _check("tc_gemm", lib.sp_tc_gemm(
         c_void_p(_ptr(a)), c_void_p(_ptr(w)), c_void_p(_ptr(out)), dt_code(out), M, N, K,
@@ -609,6 +617,13 @@ def flash_supported(q: torch.Tensor, k_pool: torch.Tensor, nh: int, nkv: int, hd
     return bool(load("attention").sp_flash_supported(int(hd), int(nh), int(nkv), int(page_size)))
 
 
+def flash_kv_supported(q: torch.Tensor, k_pool: torch.Tensor, nh: int, nkv: int, d: int, vd: int, page_size: int) -> bool:
+    """The same for key rows of ``d`` and value rows of ``vd`` entries (``flash_prefill`` and ``flash_decode`` with ``vd``)."""
+    if q.dtype != torch.bfloat16 or k_pool.dtype != torch.bfloat16 or d % 8 or vd % 8 or max(d, vd) > 128:
+        return False                              # (asked before the library: a model of other sizes never builds it)
+    return bool(load("attention_kv").sp_flash_kv_supported(int(d), int(vd), int(nh), int(nkv), int(page_size)))
+
+
 def flash_query_tile() -> int:
     """Query rows per CTA of ``flash_prefill``: a step has sum over sequences of ceil(new tokens / this) tiles."""
     return int(load("attention").sp_flash_query_tile())
@@ -630,23 +645,26 @@ def _sink_ptr(sink, nh):
 
 
 def flash_prefill(q, k_pool, v_pool, out, meta, seq_start, n_seqs, n_q_tiles, nh, nkv, hd, window, scale, sink=None,
-                  dist_bias=None):
-    """Causal attention of a step's tokens (any number per sequence) over the paged cache. ``sink`` (float32 [nh]):
+                  dist_bias=None, vd=None):
+    """Causal attention of a step's tokens (any number per sequence) over the paged cache. ``vd``: the size of a value row
+    where it differs from a key row's (``out`` is then [T, nh·vd]). ``sink`` (float32 [nh]):
     per head a score that joins the softmax's denominator once and has no value. ``dist_bias`` (float32 [nh, entries]): a
     score added by the distance between query and key, beyond the scale.
 
     ``seq_start`` [B+1] int32 on the device; ``n_q_tiles`` = sum over sequences of ceil(new tokens /
     ``flash_query_tile()``).
     """
-    lib = load("attention")
+    module = "attention" if vd is None else "attention_kv"
+    lib = load(module)
     _need_contig(q, out)
     pt = meta.page_table
-    _declare_bounds("attention", lib, _pool_pages(meta, k_pool), _table_rows(meta, pt), q.device)
+    _declare_bounds(module, lib, _pool_pages(meta, k_pool), _table_rows(meta, pt), q.device)
     bias_ptr, bias_cap = _dist_bias_args(dist_bias, nh)
-    _check("attention", lib.sp_flash_prefill_bias(
+    entry, sizes = (lib.sp_flash_prefill_bias, (hd,)) if vd is None else (lib.sp_flash_prefill_kv, (hd, int(vd)))
+    _check(module, entry(
         c_void_p(_ptr(q)), c_void_p(_ptr(out)), c_void_p(_ptr(k_pool)), c_void_p(_ptr(v_pool)),
         c_void_p(_ptr(seq_start)), c_void_p(_ptr(meta.positions)), c_void_p(_ptr(meta.seq_slot)),
-        c_void_p(_ptr(pt)), pt.shape[1], meta.page_size, int(n_seqs), int(n_q_tiles), nh, nkv, hd,
+        c_void_p(_ptr(pt)), pt.shape[1], meta.page_size, int(n_seqs), int(n_q_tiles), nh, nkv, *sizes,
         int(window or 0), c_float(scale), _sink_ptr(sink, nh), bias_ptr, bias_cap, c_void_p(_stream())))
 
 
@@ -673,26 +691,28 @@ def flash_decode_scratch_floats(n_seqs: int, nh: int, hd: int, n_chunks: int) ->
 
 
 def flash_decode(q, k_pool, v_pool, out, meta, seq_len, nh, nkv, hd, window, scale, chunk_tiles, n_chunks, scratch,
-                 counters=None, sink=None, dist_bias=None):
+                 counters=None, sink=None, dist_bias=None, vd=None):
     """One query token per sequence: keys split into chunks over CTAs, partial results combined in order.
 
-    ``seq_len`` [B] int32: each sequence's length including the query token. ``scratch``: float32,
+    ``vd``: the size of a value row where it differs from a key row's. ``seq_len`` [B] int32: each sequence's length including the query token. ``scratch``: float32,
     at least ``flash_decode_scratch_floats`` elements. ``counters``: int32, n_seqs·nkv zeros that the kernel
     hands back as zeros; with them the last CTA of each (sequence, kv head) combines, else a second kernel.
     """
     global launches
-    lib = load("attention")
+    module = "attention" if vd is None else "attention_kv"
+    lib = load(module)
     _need_contig(q, out)
     pt = meta.page_table
     n_seqs = q.shape[0]
     if counters is not None and (counters.dtype != torch.int32 or counters.numel() < n_seqs * nkv):
         raise KernelError("flash_decode: counters must be int32 with a word per (sequence, kv head)")
-    _declare_bounds("attention", lib, _pool_pages(meta, k_pool), _table_rows(meta, pt), q.device)
+    _declare_bounds(module, lib, _pool_pages(meta, k_pool), _table_rows(meta, pt), q.device)
     bias_ptr, bias_cap = _dist_bias_args(dist_bias, nh)
-    _check("attention", lib.sp_flash_decode_bias(
+    entry, sizes = (lib.sp_flash_decode_bias, (hd,)) if vd is None else (lib.sp_flash_decode_kv, (hd, int(vd)))
+    _check(module, entry(
         c_void_p(_ptr(q)), c_void_p(_ptr(out)), dt_code(out), c_void_p(_ptr(k_pool)), c_void_p(_ptr(v_pool)),
         c_void_p(_ptr(seq_len)), c_void_p(_ptr(meta.seq_slot)), c_void_p(_ptr(pt)), pt.shape[1], meta.page_size,
-        n_seqs, nh, nkv, hd, int(window or 0), c_float(scale), int(chunk_tiles), int(n_chunks),
+        n_seqs, nh, nkv, *sizes, int(window or 0), c_float(scale), int(chunk_tiles), int(n_chunks),
         c_void_p(_ptr(scratch)), c_longlong(scratch.numel()), c_void_p(_ptr(counters)), _sink_ptr(sink, nh),
         bias_ptr, bias_cap, c_void_p(_stream())))
     if counters is None:
@@ -713,7 +733,8 @@ def gemv_supported(x: torch.Tensor, w: torch.Tensor) -> bool:
             and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
-def gemv(x, w, out, mode=TC_STORE, pair=0, act=ACT_SILU, mult: float = 1.0):
+def gemv(x, w, out, mode=TC_STORE, pair=0, act=ACT_SILU, mult: float = 1.0, limit: float = 0.0,
+         slope: float = 0.0):
     """out = x · wᵀ for up to 64 tokens, streaming ``w`` once. Modes as ``tc_gemm``; for TC_SILU_MUL
     ``pair`` is the number of gate rows before the matching up rows in the interleaved weight."""
     lib = load("gemv")
@@ -725,7 +746,8 @@ def gemv(x, w, out, mode=TC_STORE, pair=0, act=ACT_SILU, mult: float = 1.0):
     if mode == TC_SILU_MUL and (act != ACT_SILU or mult != 1.0):
         _check("gemv", lib.sp_gemv_gated(
             c_void_p(_ptr(x)), c_void_p(_ptr(w)), c_void_p(_ptr(out)), dt_code(out), M, N, K, x.stride(0), w.stride(0),
-            out.stride(0), int(pair), int(act), c_float(mult), c_void_p(_stream())))
+            out.stride(0), int(pair), int(act), c_float(mult), c_float(limit), c_float(slope),
+            c_void_p(_stream())))
         return
     _check("gemv", lib.sp_gemv(
         c_void_p(_ptr(x)), c_void_p(_ptr(w)), c_void_p(_ptr(out)), dt_code(out), M, N, K,
@@ -752,29 +774,32 @@ def gemv_qkv_rope(x, w, q_out, k_pool, v_pool, meta, inv_freq, nh, nkv, hd):
 
 
 # ------------------------------------------------------------------ prefill attention on tcgen05
-def flash_tc_supported(q: torch.Tensor, k_pool: torch.Tensor, nh: int, nkv: int, hd: int, page_size: int, window) -> bool:
-    """Whether the tcgen05 prefill attention takes this shape (head 64 or 128, pages of 64, bfloat16; any window)."""
-    return (q.dtype == torch.bfloat16 and k_pool.dtype == torch.bfloat16 and k_pool.is_contiguous()
-            and bool(load("flash_tc").sp_flash_tc_supported(int(hd), int(nh), int(nkv), int(page_size), int(window or 0))))
+def flash_tc_supported(q: torch.Tensor, k_pool: torch.Tensor, nh: int, nkv: int, hd: int, page_size: int, window,
+                       vd: int | None = None) -> bool:
+    """Whether the tcgen05 prefill attention takes this shape (key rows of 40 to 192 and value rows of 8 to 128 entries,
+    multiples of 8, pages of 64, bfloat16; any window). ``vd``: the size of a value row where it differs from a key row's."""
+    return (q.dtype == torch.bfloat16 and k_pool.dtype == torch.bfloat16 and k_pool.is_contiguous() and hd % 8 == 0
+            and (vd or hd) % 8 == 0 and bool(load("flash_tc").sp_flash_tc_kv_supported(int(hd), int(vd or hd), int(nh), int(nkv), int(page_size))))
 
 
 def flash_prefill_tc(q, k_pool, v_pool, out, meta, seq_start, n_seqs, n_q_tiles, nh, nkv, hd, window, scale, sink=None,
-                     dist_bias=None):
+                     dist_bias=None, vd=None):
     """Causal attention of a step's tokens over the paged cache on the tcgen05 tensor cores. ``dist_bias`` (float32
     [nh, entries]): a score added by the distance between query and key, beyond the scale.
 
     ``n_q_tiles`` = sum over sequences of ceil(new tokens / ``flash_tc_query_tile()``). S, P and O live in tensor memory.
+    ``vd``: the size of a value row where it differs from a key row's (``out`` is then [T, nh·vd]).
     """
     lib = load("flash_tc")
     _need_contig(q, out, k_pool, v_pool)
     pt = meta.page_table
     _declare_bounds("flash_tc", lib, _pool_pages(meta, k_pool), _table_rows(meta, pt), q.device)
     bias_ptr, bias_cap = _dist_bias_args(dist_bias, nh)
-    _check("flash_tc", lib.sp_flash_prefill_tc_bias(
+    _check("flash_tc", lib.sp_flash_prefill_tc_kv(
         c_void_p(_ptr(q)), c_void_p(_ptr(out)), c_void_p(_ptr(k_pool)), c_void_p(_ptr(v_pool)),
         c_longlong(k_pool.shape[0]), q.shape[0], c_void_p(_ptr(seq_start)), c_void_p(_ptr(meta.positions)),
         c_void_p(_ptr(meta.seq_slot)), c_void_p(_ptr(pt)), pt.shape[1], meta.page_size, int(n_seqs), int(n_q_tiles),
-        nh, nkv, hd, int(window or 0), c_float(scale), c_void_p(_ptr(status_word(q.device))), _sink_ptr(sink, nh),
+        nh, nkv, hd, int(vd or hd), int(window or 0), c_float(scale), c_void_p(_ptr(status_word(q.device))), _sink_ptr(sink, nh),
         bias_ptr, bias_cap, c_void_p(_stream())))
 
 
@@ -923,7 +948,8 @@ def tc_stream_supported(x: torch.Tensor, w: torch.Tensor, mode=TC_STORE, pair: i
         int(mode), int(pair)) == 0
 
 
-def tc_stream(x, w, out, mode=TC_STORE, pair=0, act=ACT_SILU, mult: float = 1.0):
+def tc_stream(x, w, out, mode=TC_STORE, pair=0, act=ACT_SILU, mult: float = 1.0, limit: float = 0.0,
+              slope: float = 0.0):
     """out = x · wᵀ for up to 128 tokens on the tensor cores with the rows of ``w`` as the instruction's M: every SM
     streams its share of ``w``; K is cut over the CTAs of a cluster, whose pieces are added in a fixed order. Modes as ``tc_gemm``; for
     TC_SILU_MUL ``pair`` is the number of gate rows before the matching up rows in the interleaved weight."""
@@ -936,7 +962,7 @@ def tc_stream(x, w, out, mode=TC_STORE, pair=0, act=ACT_SILU, mult: float = 1.0)
     if mode == TC_SILU_MUL and (act != ACT_SILU or mult != 1.0):
         _check("tc_stream", lib.sp_tc_stream_gated(
             c_void_p(_ptr(x)), c_void_p(_ptr(w)), c_void_p(_ptr(out)), dt_code(out), M, N, K, x.stride(0), w.stride(0),
-            out.stride(0), int(pair), int(act), c_float(mult), c_void_p(_ptr(status_word(x.device))), c_void_p(_stream())))
+            out.stride(0), int(pair), int(act), c_float(mult), c_float(limit), c_float(slope), c_void_p(_ptr(status_word(x.device))), c_void_p(_stream())))
         return
     _check("tc_stream", lib.sp_tc_stream(
         c_void_p(_ptr(x)), c_void_p(_ptr(w)), c_void_p(_ptr(out)), dt_code(out), M, N, K, x.stride(0), w.stride(0),
@@ -1426,10 +1452,10 @@ def pair_embed(table, pairs, step, state, out, buckets, mul_prev, mul_cur, scale
         c_void_p(_ptr(status)), c_void_p(_stream())))
 
 
-def stream_norm_add(x, y, w_post, mult, eps, w_next=None, out=None, raw=False):
+def stream_norm_add(x, y, w_post, mult, eps, w_next=None, out=None, raw=False, centered=False):
     """x ← x + mult · y / sqrt(mean(y²) + eps) ⊙ w_post, row by row, and y ← 0 (x, y float32 [T, W]; the weights
     float32 as they multiply). ``out`` [T, W] then receives the next reader's input: the RMS norm of the new x with
-    ``w_next``, or with ``raw`` the new x itself."""
+    ``w_next``, or with ``raw`` the new x itself. ``centered``: both norms are layer norms (the mean taken off first)."""
     lib = load("sandwich")
     if x.dtype != torch.float32 or y.dtype != torch.float32 or w_post.dtype != torch.float32 or x.shape != y.shape:
         raise KernelError("stream_norm_add works on two float32 buffers of one shape and float32 weights")
@@ -1439,7 +1465,30 @@ def stream_norm_add(x, y, w_post, mult, eps, w_next=None, out=None, raw=False):
         raise KernelError("stream_norm_add: the next norm needs a float32 weight")
     _check("sandwich", lib.sp_stream_norm_add(
         c_void_p(_ptr(x)), c_void_p(_ptr(y)), c_void_p(_ptr(w_post)), c_void_p(_ptr(w_next)), c_void_p(_ptr(out)),
-        dt_code(out) if out is not None else 0, mode, x.shape[0], x.shape[1], c_float(mult), c_float(eps), c_void_p(_stream())))
+        dt_code(out) if out is not None else 0, mode, x.shape[0], x.shape[1], c_float(mult), c_float(eps), int(bool(centered)),
+        c_void_p(_stream())))
+
+
+def qkv_norm_rot_store(proj, bias, q_out, k_pool, v_pool, meta, freq, nh, nkv, d, vd, rd, q_weight=None, k_weight=None,
+                       eps=0.0, rot_mult=1.0, halves=True):
+    """``proj`` rows (float32) = [q: nh·d | k: nkv·d | v: nkv·vd | ...] (``nkv`` 0: queries only, nothing is cached): add
+    ``bias`` (over q, k, v), take the RMS norm of every q and k head with its weight [d] (None: no norm), rotate pairs
+    over the first ``rd`` dims (``halves``: dim i with dim i + rd/2, else neighbours) by position · freq[i], cos and sin
+    times ``rot_mult``; q to ``q_out``, k and v into their page rows."""
+    lib = load("sandwich")
+    if proj.dtype != torch.float32:
+        raise KernelError("qkv_norm_rot_store reads 32-bit projections")
+    _need_contig(proj, bias, q_out, freq, q_weight, k_weight)
+    pt = meta.page_table
+    _declare_bounds("sandwich", lib, _pool_pages(meta, k_pool), _table_rows(meta, pt), proj.device)
+    ws = [w for w in (q_weight, k_weight) if w is not None]
+    _check("sandwich", lib.sp_qkv_norm_rot_store(
+        c_void_p(_ptr(proj)), proj.shape[1], c_void_p(_ptr(bias)), dt_code(bias) if bias is not None else 0,
+        c_void_p(_ptr(q_weight)), c_void_p(_ptr(k_weight)), _w_dt(*ws) if ws else 0, c_void_p(_ptr(q_out)), dt_code(q_out),
+        c_void_p(_ptr(k_pool)), c_void_p(_ptr(v_pool)), dt_code(k_pool), c_void_p(_ptr(freq)), c_void_p(_ptr(meta.token_seq)),
+        c_void_p(_ptr(meta.positions)), c_void_p(_ptr(meta.seq_slot)), c_void_p(_ptr(pt)), pt.shape[1], meta.page_size,
+        proj.shape[0], int(nh), int(nkv), int(d), int(vd), int(rd), int(bool(halves)), c_float(rot_mult), c_float(eps),
+        c_void_p(_stream())))
 
 
 def gated_qkv_store(proj, bias, q_out, k_pool, v_pool, meta, gates, freq, nh, nkv, d, vd, rd, write_kv=True, rot_mult=1.0,
@@ -1528,4 +1577,36 @@ def rglru(proj, w: dict, ring, state, out, step, width, taps, parts, mult=1.0):
     _check("rglru", lib.sp_rglru_chunked(
         *head, c_void_p(_ptr(av)), c_void_p(_ptr(cells)), c_void_p(_ptr(starts)), n_chunks, n_blocks, c_void_p(_ptr(out)), dt_code(out), T,
         step.n_seqs, int(width), int(taps), int(parts), c_float(mult), int(tensor_cores), c_void_p(_ptr(status_word(proj.device))),
+        c_void_p(_stream())))
+
+
+# ------------------------------------------------------------------ mlstm: a matrix memory with exponential input gates
+def mlstm(proj, w: dict, state, nm, out, step, H, d, vd, cap, eps):
+    """``proj`` rows [q: H·d | k: H·d | v: H·vd | g: H·vd | i: H | f: H] (float32, gates without biases); ``w``: ``ib``, ``fb``
+    [H] and ``norm`` [H·vd] of one storage type; ``state`` float32 [slots, H, d, vd], ``nm`` float32 [slots, H, d + 1] (the
+    normaliser and the running maximum); ``out`` [T, H·vd] = unit rms of the heads' outputs ⊙ norm ⊙ sigmoid(g)."""
+    lib = load("mlstm")
+    if proj.dtype != torch.float32 or state.dtype != torch.float32 or nm.dtype != torch.float32:
+        raise KernelError("mlstm runs on 32-bit projections and states")
+    if state.shape[1:] != (H, d, vd) or nm.shape != (state.shape[0], H, d + 1):
+        raise KernelError(f"mlstm: states {tuple(state.shape)} and {tuple(nm.shape)} do not fit {H} heads of {d} x {vd}")
+    _need_contig(proj, state, nm, out, w["ib"], w["fb"], w["norm"])
+    T = proj.shape[0]
+    scratch, n_chunks, mode = None, 0, 1
+    w_dt = _w_dt(w["ib"], w["fb"], w["norm"])
+    if not step.all_single:
+        global launches
+        # a prompt of some length on the tensor cores (gates, the chunks' sums, their start states, outputs with their norms
+        # and gates), short portions and the 32-bit mode in FFMA products (the norms and gates in a kernel of their own)
+        tc = step.max_new >= CHUNKED_FROM and bool(lib.sp_mlstm_tc_supported(
+            c_void_p(_ptr(proj)), proj.shape[1], c_void_p(_ptr(w["norm"])), w_dt, c_void_p(_ptr(out)), dt_code(out), int(d), int(vd)))
+        mode = 2 if tc else 0
+        launches += 3 if tc and vd <= 256 else 4
+        n_chunks = query_tiles(step.host["new_counts"], int(lib.sp_mlstm_chunk_tokens(int(tc))))
+        scratch = torch.empty(int(lib.sp_mlstm_scratch_floats(n_chunks, T, H, d, vd)), dtype=torch.float32, device=proj.device)
+    _check("mlstm", lib.sp_mlstm(
+        c_void_p(_ptr(proj)), proj.shape[1], c_void_p(_ptr(w["ib"])), c_void_p(_ptr(w["fb"])), c_void_p(_ptr(w["norm"])),
+        w_dt, c_void_p(_ptr(state)), c_void_p(_ptr(nm)), state.shape[0], c_void_p(_ptr(out)),
+        dt_code(out), c_void_p(_ptr(step.seq_start)), c_void_p(_ptr(step.seq_slot)), step.n_seqs, T, n_chunks, int(H), int(d),
+        int(vd), c_float(cap), c_float(eps), c_void_p(_ptr(scratch)), mode, c_void_p(_ptr(status_word(proj.device))),
         c_void_p(_stream())))

@@ -4,10 +4,13 @@
 //                       table's row n. The token before a step's first one is a word of per-slot state.
 //   stream_norm_add     x ← x + r · y / sqrt(mean(y²) + eps) ⊙ w for a sublayer's output y (which is left zeroed for
 //                       the next sublayer to add into); in the same pass the next reader's input: the norm of the new
-//                       x with another weight, or the new x as it is, in the activation type
+//                       x with another weight, or the new x as it is, in the activation type; ``centered``: both norms
+//                       are layer norms (mean taken off, a weight, no bias)
 //   gated_qkv_store     a projected row [q | k | v | one gate per head]: biases, a query factor that grows with the
 //                       logarithm of the position, rotation of neighbouring pairs over the first dims of every head,
 //                       q out, k and v into their page rows, the gates out as 32-bit numbers
+//   qkv_norm_rot_store  a projected row [q | k | v]: biases, an RMS norm with a weight of every q and k head, rotation of
+//                       pairs half the rotated dims apart (or neighbouring ones), q out, k and v into their page rows
 //   latent_rot_store    a projected row [q (per head: plain | rotated part) | low-rank row | shared key part | gates]:
 //                       RMS norm of the low-rank row, rotation of the shared key part and of the queries' rotated
 //                       parts (neighbouring dims or dims half the part apart form a pair), [normed row | rotated key
@@ -155,13 +158,126 @@ __global__ void __launch_bounds__(256) stream_norm_add_kernel(NormAddArgs a) {
     }
 }
 
+// The same with layer norms: (v − mean) / sqrt(mean((v − mean)²) + eps) ⊙ w for the output and for the next reader. Rows of
+// up to NV · 1,024 numbers stay in registers between the passes (NV 0: any width, re-read).
+template <int NV>
+__global__ void __launch_bounds__(256) stream_layernorm_add_kernel(NormAddArgs a) {
+    __shared__ float red[32];
+    sp_allow_dependents();
+    sp_wait_for_predecessor();
+    const int t = blockIdx.x;
+    if (t >= a.T) return;
+    float* xr = a.x + (size_t)t * a.W;
+    float* yr = a.y + (size_t)t * a.W;
+    const float invW = 1.0f / (float)a.W;
+    if (NV > 0) {
+        constexpr int N = NV > 0 ? NV : 1;
+        float4 v[N], x[N];
+        float sum = 0.0f;
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            const int c = (i * 256 + threadIdx.x) * 4;
+            v[i] = x[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (c < a.W) {
+                v[i] = *(const float4*)(yr + c);
+                x[i] = *(const float4*)(xr + c);
+                *(float4*)(yr + c) = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            }
+            sum += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+        }
+        const float mean = sp_block_sum(sum, red) * invW;
+        float ss = 0.0f;
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            if ((i * 256 + threadIdx.x) * 4 >= a.W) continue;
+            v[i].x -= mean; v[i].y -= mean; v[i].z -= mean; v[i].w -= mean;
+            ss = fmaf(v[i].x, v[i].x, ss); ss = fmaf(v[i].y, v[i].y, ss); ss = fmaf(v[i].z, v[i].z, ss); ss = fmaf(v[i].w, v[i].w, ss);
+        }
+        const float f = a.mult / sqrtf(sp_block_sum(ss, red) * invW + a.eps);
+        sum = 0.0f;
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            const int c = (i * 256 + threadIdx.x) * 4;
+            if (c >= a.W) continue;
+            const float4 w = *(const float4*)(a.w_post + c);
+            x[i].x = fmaf(v[i].x * f, w.x, x[i].x); x[i].y = fmaf(v[i].y * f, w.y, x[i].y);
+            x[i].z = fmaf(v[i].z * f, w.z, x[i].z); x[i].w = fmaf(v[i].w * f, w.w, x[i].w);
+            *(float4*)(xr + c) = x[i];
+            sum += (x[i].x + x[i].y) + (x[i].z + x[i].w);
+        }
+        if (a.next_mode == 0) return;
+        float m2 = 0.0f, g = 1.0f;
+        if (a.next_mode == 1) {
+            m2 = sp_block_sum(sum, red) * invW;
+            ss = 0.0f;
+#pragma unroll
+            for (int i = 0; i < N; ++i) {
+                if ((i * 256 + threadIdx.x) * 4 >= a.W) continue;
+                const float p = x[i].x - m2, q = x[i].y - m2, r = x[i].z - m2, u = x[i].w - m2;
+                ss = fmaf(p, p, ss); ss = fmaf(q, q, ss); ss = fmaf(r, r, ss); ss = fmaf(u, u, ss);
+            }
+            g = 1.0f / sqrtf(sp_block_sum(ss, red) * invW + a.eps);
+        }
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            const int c = (i * 256 + threadIdx.x) * 4;
+            if (c >= a.W) continue;
+            float4 o = x[i];
+            if (a.next_mode == 1) {
+                const float4 w = *(const float4*)(a.w_next + c);
+                o.x = (o.x - m2) * (g * w.x); o.y = (o.y - m2) * (g * w.y); o.z = (o.z - m2) * (g * w.z); o.w = (o.w - m2) * (g * w.w);
+            }
+            if (a.out_dt == SP_DT_F32) {
+                *(float4*)((float*)a.out + (size_t)t * a.W + c) = o;
+            } else {
+                __nv_bfloat162 p0 = __floats2bfloat162_rn(o.x, o.y), p1 = __floats2bfloat162_rn(o.z, o.w);
+                uint2 pk;
+                pk.x = *(uint32_t*)&p0; pk.y = *(uint32_t*)&p1;
+                *(uint2*)((__nv_bfloat16*)a.out + (size_t)t * a.W + c) = pk;
+            }
+        }
+        return;
+    }
+    float sum = 0.0f, ss = 0.0f;
+    for (int c = threadIdx.x; c < a.W; c += blockDim.x) sum += yr[c];
+    const float mean = sp_block_sum(sum, red) * invW;
+    for (int c = threadIdx.x; c < a.W; c += blockDim.x) { const float v = yr[c] - mean; ss = fmaf(v, v, ss); }
+    const float f = a.mult / sqrtf(sp_block_sum(ss, red) * invW + a.eps);
+    sum = 0.0f;
+    for (int c = threadIdx.x; c < a.W; c += blockDim.x) {
+        const float x = fmaf((yr[c] - mean) * f, a.w_post[c], xr[c]);
+        xr[c] = x;
+        yr[c] = 0.0f;
+        sum += x;
+    }
+    if (a.next_mode == 0) return;
+    float m2 = 0.0f, g = 1.0f;
+    if (a.next_mode == 1) {
+        m2 = sp_block_sum(sum, red) * invW;
+        ss = 0.0f;
+        for (int c = threadIdx.x; c < a.W; c += blockDim.x) { const float v = xr[c] - m2; ss = fmaf(v, v, ss); }
+        g = 1.0f / sqrtf(sp_block_sum(ss, red) * invW + a.eps);
+    }
+    for (int c = threadIdx.x; c < a.W; c += blockDim.x)
+        sp_st_dt(a.out, a.out_dt, (size_t)t * a.W + c, a.next_mode == 1 ? (xr[c] - m2) * (g * a.w_next[c]) : xr[c]);
+}
+
 SP_API int sp_stream_norm_add(float* x, float* y, const float* w_post, const float* w_next, void* out, int out_dt,
-                              int next_mode, int T, int W, float mult, float eps, cudaStream_t stream) {
+                              int next_mode, int T, int W, float mult, float eps, int centered, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (next_mode < 0 || next_mode > 2 || (next_mode && !out) || (next_mode == 1 && !w_next))
         SP_FAIL("stream_norm_add: mode %d needs an output (and a weight for the norm)", next_mode);
     NormAddArgs a{x, y, w_post, w_next, out, out_dt, next_mode, T, W, mult, eps};
     const bool vec = (W % 4) == 0 && ((((uintptr_t)x | (uintptr_t)y | (uintptr_t)w_post | (uintptr_t)w_next | (uintptr_t)out) & 15) == 0);
+    if (centered) {
+        const dim3 g(T), b(256);
+        if (vec && W <= 1024) SP_CHECK_CALL("stream_norm_add", sp_launch_dependent(stream_layernorm_add_kernel<1>, g, b, 0, stream, a));
+        else if (vec && W <= 2048) SP_CHECK_CALL("stream_norm_add", sp_launch_dependent(stream_layernorm_add_kernel<2>, g, b, 0, stream, a));
+        else if (vec && W <= 4096) SP_CHECK_CALL("stream_norm_add", sp_launch_dependent(stream_layernorm_add_kernel<4>, g, b, 0, stream, a));
+        else if (vec && W <= 8192) SP_CHECK_CALL("stream_norm_add", sp_launch_dependent(stream_layernorm_add_kernel<8>, g, b, 0, stream, a));
+        else SP_CHECK_CALL("stream_norm_add", sp_launch_dependent(stream_layernorm_add_kernel<0>, g, b, 0, stream, a));
+        return 0;
+    }
     if (vec) SP_CHECK_CALL("stream_norm_add", sp_launch_dependent(stream_norm_add_kernel<4>, dim3(T), dim3(256), 0, stream, a));
     else SP_CHECK_CALL("stream_norm_add", sp_launch_dependent(stream_norm_add_kernel<1>, dim3(T), dim3(256), 0, stream, a));
     return 0;
@@ -292,6 +408,147 @@ SP_API int sp_gated_qkv_store(const float* proj, int ld, const void* bias, int b
     else if (q_dt == SP_DT_BF16 && c_dt == SP_DT_F32) GQ_LAUNCH(__nv_bfloat16, float);
     else SP_FAIL("gated_qkv_store: unsupported dtype codes %d/%d", q_dt, c_dt);
 #undef GQ_LAUNCH
+    return 0;
+}
+
+// ============================================================== [q | k | v]: bias, norm per head, rotation, store
+struct NormRotArgs {
+    const float* proj; int ld;           // [T][ld] = [q: nh·d | k: nkv·d | v: nkv·vd | ...]; nkv 0: queries only
+    const void* bias; int b_dt;          // over q, k, v; or null
+    const void* qw; const void* kw; int w_dt;   // [d] weights of the heads' RMS norms, or null: no norm
+    void* q_out; int q_dt;               // [T][nh·d]
+    void* kpool; void* vpool; int c_dt;  // [pages][nkv][page_size][d], [pages][nkv][page_size][vd]
+    const float* freq;                   // [rd/2] or null
+    RowPlace pl;
+    int T, nh, nkv, d, vd, rd, halves;   // halves: dim i pairs with dim i + rd/2, else dim 2i with dim 2i + 1
+    float rot_mult, eps;
+};
+
+__device__ __forceinline__ float4 ld4_dt(const void* p, int dt, size_t i) {
+    if (dt == SP_DT_F32) return *(const float4*)((const float*)p + i);
+    const uint2 u = *(const uint2*)((const __nv_bfloat16*)p + i);
+    const float2 a = __bfloat1622float2(*(const __nv_bfloat162*)&u.x), b = __bfloat1622float2(*(const __nv_bfloat162*)&u.y);
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void st4(float* p, size_t i, float4 v) { *(float4*)(p + i) = v; }
+__device__ __forceinline__ void st4(__nv_bfloat16* p, size_t i, float4 v) {
+    __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    uint2 u;
+    u.x = *(uint32_t*)&a; u.y = *(uint32_t*)&b;
+    *(uint2*)(p + i) = u;
+}
+
+// One block per token, a warp per head in turn; a head's values wait in shared memory so that a lane reaches both dims of
+// a pair. VEC: d, vd, rd/2 and all strides are multiples of four and pairs lie half apart: four neighbouring dims at a time.
+constexpr int NR_WARPS = 8;
+template <typename TO, typename TC, bool VEC>
+__global__ void __launch_bounds__(NR_WARPS * 32) qkv_norm_rot_store_kernel(NormRotArgs a) {
+    extern __shared__ __align__(16) float cs[];          // [2][rd/2], then [warps][d]
+    sp_allow_dependents();
+    sp_wait_for_predecessor();
+    const int t = blockIdx.x;
+    if (t >= a.T) return;
+    const int pos = a.pl.positions[t];
+    const int half = a.rd >> 1, d = a.d, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    pair_angles(cs, a.freq, half, pos, a.rot_mult);
+    float* hv = cs + ((2 * half + 3) & ~3) + warp * ((d + 3) & ~3);
+    __syncthreads();
+    int page = 0;
+    const bool place_ok = a.nkv > 0 && page_of(a.pl, t, pos, page);
+    const int off = pos % a.pl.page_size;
+    const float* src = a.proj + (size_t)t * a.ld;
+    TO* q_out = (TO*)a.q_out + (size_t)t * a.nh * d;
+    for (int h = warp; h < a.nh + a.nkv; h += NR_WARPS) {
+        const bool is_q = h < a.nh;
+        const void* w = is_q ? a.qw : a.kw;
+        float ss = 0.0f;
+        if (VEC) {
+            for (int i = lane * 4; i < d; i += 128) {
+                float4 v = *(const float4*)(src + h * d + i);
+                if (a.bias) { const float4 b = ld4_dt(a.bias, a.b_dt, (size_t)h * d + i); v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w; }
+                ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
+                *(float4*)(hv + i) = v;
+            }
+        } else {
+            for (int i = lane; i < d; i += 32) {
+                const float v = src[h * d + i] + (a.bias ? sp_ld_dt(a.bias, a.b_dt, (size_t)h * d + i) : 0.0f);
+                ss = fmaf(v, v, ss);
+                hv[i] = v;
+            }
+        }
+        if (w) {
+            const float inv = 1.0f / sqrtf(sp_warp_sum(ss) / (float)d + a.eps);
+            __syncwarp();
+            for (int i = lane; i < d; i += 32) hv[i] = hv[i] * inv * sp_ld_dt(w, a.w_dt, i);
+        }
+        __syncwarp();
+        const size_t base = is_q ? (size_t)h * d : (((size_t)page * a.nkv + (h - a.nh)) * a.pl.page_size + off) * d;
+        if (VEC) {
+            for (int i = lane * 4; i < d; i += 128) {
+                float4 v = *(const float4*)(hv + i);
+                if (i < a.rd) {
+                    const bool lo = i < half;
+                    const int p = lo ? i : i - half;
+                    const float4 o = *(const float4*)(hv + (lo ? i + half : p)), c = *(const float4*)(cs + p);
+                    float4 s4 = *(const float4*)(cs + half + p);
+                    if (lo) { s4.x = -s4.x; s4.y = -s4.y; s4.z = -s4.z; s4.w = -s4.w; }
+                    v.x = v.x * c.x + o.x * s4.x; v.y = v.y * c.y + o.y * s4.y; v.z = v.z * c.z + o.z * s4.z; v.w = v.w * c.w + o.w * s4.w;
+                }
+                if (is_q) st4(q_out, base + i, v);
+                else if (place_ok) st4((TC*)a.kpool, base + i, v);
+            }
+        } else {
+            for (int i = lane; i < d; i += 32) {
+                float v = hv[i];
+                if (i < a.rd) {
+                    const bool lo = a.halves ? i < half : (i & 1) == 0;
+                    const int p = a.halves ? (lo ? i : i - half) : i >> 1;
+                    const int other = a.halves ? (lo ? i + half : p) : i ^ 1;
+                    v = lo ? v * cs[p] - hv[other] * cs[half + p] : v * cs[p] + hv[other] * cs[half + p];
+                }
+                if (is_q) sp_st(q_out, base + i, v);
+                else if (place_ok) sp_st((TC*)a.kpool, base + i, v);
+            }
+        }
+        __syncwarp();
+    }
+    if (!place_ok) return;
+    const int v0 = (a.nh + a.nkv) * d;
+    for (int e = threadIdx.x * (VEC ? 4 : 1); e < a.nkv * a.vd; e += blockDim.x * (VEC ? 4 : 1)) {
+        const int g = e / a.vd, r = e - g * a.vd;
+        const size_t to = (((size_t)page * a.nkv + g) * a.pl.page_size + off) * a.vd + r;
+        if (VEC) {
+            float4 v = *(const float4*)(src + v0 + e);
+            if (a.bias) { const float4 b = ld4_dt(a.bias, a.b_dt, (size_t)v0 + e); v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w; }
+            st4((TC*)a.vpool, to, v);
+        } else {
+            sp_st((TC*)a.vpool, to, src[v0 + e] + (a.bias ? sp_ld_dt(a.bias, a.b_dt, (size_t)v0 + e) : 0.0f));
+        }
+    }
+}
+
+SP_API int sp_qkv_norm_rot_store(const float* proj, int ld, const void* bias, int b_dt, const void* qw, const void* kw, int w_dt,
+                                 void* q_out, int q_dt, void* kpool, void* vpool, int c_dt, const float* freq,
+                                 const int* token_seq, const int* positions, const int* seq_row, const int* page_table,
+                                 int max_pages, int page_size, int T, int nh, int nkv, int d, int vd, int rd, int halves,
+                                 float rot_mult, float eps, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (d <= 0 || vd <= 0 || rd < 0 || rd > d || (rd & 1)) SP_FAIL("qkv_norm_rot_store: the rotated dims %d must be even and at most %d", rd, d);
+    if (rd > 0 && !freq) SP_FAIL("qkv_norm_rot_store: a frequency table is needed");
+    if (ld < (nh + nkv) * d + nkv * vd) SP_FAIL("qkv_norm_rot_store: rows of %d numbers are too short", ld);
+    NormRotArgs a{proj, ld, bias, b_dt, qw, kw, w_dt, q_out, q_dt, kpool, vpool, c_dt, freq,
+                  RowPlace{token_seq, positions, seq_row, page_table, max_pages, page_size, sp_range_host},
+                  T, nh, nkv, d, vd, rd, halves, rot_mult, eps};
+    const bool vec = (halves || rd == 0) && d % 4 == 0 && vd % 4 == 0 && rd % 8 == 0 && ld % 4 == 0 &&
+                     ((((uintptr_t)proj | (uintptr_t)bias | (uintptr_t)q_out | (uintptr_t)kpool | (uintptr_t)vpool) & 15) == 0);
+    const size_t smem = (size_t)(((rd + 3) & ~3) + NR_WARPS * ((d + 3) & ~3)) * sizeof(float);
+    if (smem > 48 * 1024) SP_FAIL("qkv_norm_rot_store: heads of %d are beyond this kernel's range", d);
+#define NR_LAUNCH(TO, TC) do { if (vec) SP_CHECK_CALL("qkv_norm_rot_store", sp_launch_dependent(qkv_norm_rot_store_kernel<TO, TC, true>, dim3(T), dim3(NR_WARPS * 32), smem, stream, a)); \
+    else SP_CHECK_CALL("qkv_norm_rot_store", sp_launch_dependent(qkv_norm_rot_store_kernel<TO, TC, false>, dim3(T), dim3(NR_WARPS * 32), smem, stream, a)); } while (0)
+    if (q_dt == SP_DT_F32 && c_dt == SP_DT_F32) NR_LAUNCH(float, float);
+    else if (q_dt == SP_DT_BF16 && c_dt == SP_DT_BF16) NR_LAUNCH(__nv_bfloat16, __nv_bfloat16);
+    else SP_FAIL("qkv_norm_rot_store: queries and cache share a storage type (codes %d/%d)", q_dt, c_dt);
+#undef NR_LAUNCH
     return 0;
 }
 

@@ -174,13 +174,11 @@ template <int BN, int STAGES, int CG = 1>
 __global__ void __launch_bounds__(192, 1)
 tc_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                void* __restrict__ C, int c_dt, int M, int N, int K, int ldc, int mode, int* status,
-               const __grid_constant__ EpiArgs ep, const SpRange rg, const int* __restrict__ group, float glu_limit,
-               float glu_slope, int act, float mult) {
+               const __grid_constant__ EpiArgs ep, const SpRange rg, const int* __restrict__ group, SpGate ga) {
     // ``group`` (single CTAs only): a grouped product. The rows of A lie sorted by group in tiles of 128 rows; entry
     // t of the table is the row of W at which the weights of row tile t's group begin (W stacks the groups' matrices,
-    // N rows each), or -1 for a row tile that is not in use, which all three roles pass over alike. ``glu_slope``
-    // non-zero: the gated epilogue is g·sigmoid(slope·g)·(u + 1) with g = min(gate, limit), u = clamp(up, ±limit).
-    // ``act`` (SP_ACT_*): the gate's activation otherwise, with ``mult`` on the outputs; SP_ACT_RELU2 squares the relu of
+    // N rows each), or -1 for a row tile that is not in use, which all three roles pass over alike. ``ga``:
+    // the activation of gated tiles with its constants (see SpGate); SP_ACT_RELU2 squares the relu of
     // a plain store.
     using L = SmemLayout<BN, STAGES, CG>;
     extern __shared__ uint8_t smem_raw[];
@@ -521,20 +519,13 @@ tc_gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                     tc_ld_wait();
 #pragma unroll
                     for (int j = 0; j < 32; ++j) {
-                        float g = __uint_as_float(r[j]) * rstd;
-                        if (glu_slope != 0.0f) {
-                            g = fminf(g, glu_limit);
-                            const float up = fminf(fmaxf(__uint_as_float(u[j]) * rstd, -glu_limit), glu_limit);
-                            v[j] = (g / (1.0f + expf(-glu_slope * g))) * (up + 1.0f);
-                        } else {
-                            v[j] = sp_gated(g, __uint_as_float(u[j]) * rstd, act) * mult;
-                        }
+                        v[j] = sp_gated(__uint_as_float(r[j]) * rstd, __uint_as_float(u[j]) * rstd, ga);
                     }
                 } else {
                     tc_ld_wait();
 #pragma unroll
                     for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]) * rstd;
-                    if (act == SP_ACT_RELU2) {
+                    if (ga.kind == SP_ACT_RELU2) {
 #pragma unroll
                         for (int j = 0; j < 32; ++j) v[j] = sp_relu2(v[j]);
                     }
@@ -593,7 +584,7 @@ __device__ __forceinline__ uint32_t part_addr(uint32_t part, int col, int row) {
 template <int BN, int STAGES>
 __global__ void __launch_bounds__(192, 1)
 tc_gemm_splitk_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
-                      void* __restrict__ C, int c_dt, int M, int N, int K, int ldc, int mode, int splits, int* status, int act, float mult) {
+                      void* __restrict__ C, int c_dt, int M, int N, int K, int ldc, int mode, int splits, int* status, SpGate ga) {
     using L = SmemLayout<BN, STAGES>;
     static_assert(STAGES * L::STAGE_BYTES >= BM * BN * 4, "the partial tile must fit over the pipeline stages");
     extern __shared__ uint8_t smem_raw[];
@@ -720,7 +711,7 @@ tc_gemm_splitk_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_co
                     }
                 }
 #pragma unroll
-                for (int j = 0; j < 32; ++j) v[j] = sp_gated(v[j], b[j], act) * mult;
+                for (int j = 0; j < 32; ++j) v[j] = sp_gated(v[j], b[j], ga);
                 if (grow < M) store_row32(C, c_dt, (size_t)grow * ldc + n0 / 2 + c0, n0 / 2 + c0, N / 2, v, false);
             } else if (grow < M) {
                 store_row32(C, c_dt, (size_t)grow * ldc + n0 + c0, n0 + c0, N, v, mode == MODE_ACCUMULATE);
@@ -799,7 +790,7 @@ int make_map(CUtensorMap* map, const void* ptr, int rows, int K, int ld, int box
 
 template <int BN, int STAGES>
 int launch(const CUtensorMap& ma, const CUtensorMap& mw, void* C, int c_dt, int M, int N, int K, int ldc, int mode,
-           int* status, cudaStream_t stream, const EpiArgs& ep, int act, float mult) {
+           int* status, cudaStream_t stream, const EpiArgs& ep, SpGate ga) {
     using L = SmemLayout<BN, STAGES>;
     static SpPerDevice configured;
     if (!configured.done()) {
@@ -813,7 +804,7 @@ int launch(const CUtensorMap& ma, const CUtensorMap& mw, void* C, int c_dt, int 
     const int grid = (int)(tiles < sm_count ? tiles : sm_count);
     SP_CHECK_CALL("tc_gemm", sp_launch_dependent(tc_gemm_kernel<BN, STAGES>, dim3(grid), dim3(192), (size_t)L::TOTAL, stream, ma, mw,
                                                  C, c_dt, M, N, K, ldc, mode, status, ep, sp_range_host, (const int*)nullptr,
-                                                 0.0f, 0.0f, act, mult));
+                                                 ga));
     return 0;
 }
 
@@ -834,16 +825,17 @@ int launch_grouped(const CUtensorMap& ma, const CUtensorMap& mw, void* C, int c_
     const int grid = (int)(tiles < sm_count ? tiles : sm_count);
     EpiArgs ep;
     memset(&ep, 0, sizeof(ep));
+    const SpGate ga{slope != 0.0f ? (int)SP_ACT_CLAMPED : act, 1.0f, limit, slope};
     SP_CHECK_CALL("tc_gemm (grouped)", sp_launch_dependent(tc_gemm_kernel<BN, STAGES>, dim3(grid), dim3(192), (size_t)L::TOTAL, stream,
                                                            ma, mw, C, c_dt, M, N, K, ldc, mode, status, ep, sp_range_host, group,
-                                                           limit, slope, act, 1.0f));
+                                                           ga));
     return 0;
 }
 
 // The same tiles by pairs of CTAs (tcgen05 cta_group::2): tiles of 256 rows, one pair per two SMs.
 template <int BN, int STAGES>
 int launch_pair(const CUtensorMap& ma, const CUtensorMap& mw_half, void* C, int c_dt, int M, int N, int K, int ldc, int mode,
-                int* status, cudaStream_t stream, const EpiArgs& ep, int act, float mult) {
+                int* status, cudaStream_t stream, const EpiArgs& ep, SpGate ga) {
     using L = SmemLayout<BN, STAGES, 2>;
     static_assert(L::TOTAL <= 232448, "a CTA's shared memory");
     static SpPerDevice configured;
@@ -858,13 +850,13 @@ int launch_pair(const CUtensorMap& ma, const CUtensorMap& mw_half, void* C, int 
     const int pairs = (int)(tiles < sm_count / 2 ? tiles : sm_count / 2);
     SP_CHECK_CALL("tc_gemm", sp_launch_cluster(tc_gemm_kernel<BN, STAGES, 2>, dim3(2 * pairs), dim3(192), (size_t)L::TOTAL, stream,
                                                -2, ma, mw_half, C, c_dt, M, N, K, ldc, mode, status, ep, sp_range_host,
-                                               (const int*)nullptr, 0.0f, 0.0f, act, mult));
+                                               (const int*)nullptr, ga));
     return 0;
 }
 
 template <int BN, int STAGES>
 int launch_splitk(const CUtensorMap& ma, const CUtensorMap& mw, void* C, int c_dt, int M, int N, int K, int ldc,
-                  int mode, int splits, int* status, cudaStream_t stream, int act, float mult) {
+                  int mode, int splits, int* status, cudaStream_t stream, SpGate ga) {
     using L = SmemLayout<BN, STAGES>;
     static SpPerDevice configured;
     if (!configured.done()) {
@@ -875,7 +867,7 @@ int launch_splitk(const CUtensorMap& ma, const CUtensorMap& mw, void* C, int c_d
     const int n_tiles = ((N + BN - 1) / BN) * ((M + BM - 1) / BM);
     SP_CHECK_CALL("tc_gemm_splitk", sp_launch_cluster(tc_gemm_splitk_kernel<BN, STAGES>, dim3(n_tiles * splits), dim3(192),
                                                      (size_t)L::TOTAL, stream, splits, ma, mw, C, c_dt, M, N, K, ldc,
-                                                     mode, splits, status, act, mult));
+                                                     mode, splits, status, ga));
     return 0;
 }
 
@@ -912,8 +904,7 @@ SP_API int sp_tc_gemm_supported(const void* A, const void* W, int K, int lda, in
 SP_API int sp_tc_gemm_n_tiles(int N, int bn) { return bn > 0 ? (N + bn - 1) / bn : 0; }
 
 static int tc_gemm_any(const void* A, const void* W, void* C, int c_dt, int M, int N, int K, int lda, int ldw, int ldc,
-                       int mode, int bn, const EpiArgs* epp, int* status, cudaStream_t stream, int act = SP_ACT_SILU,
-                       float mult = 1.0f);
+                       int mode, int bn, const EpiArgs* epp, int* status, cudaStream_t stream, SpGate ga = SpGate{});
 
 // CTAs that would share a tile along K in sp_tc_gemm for these sizes (1: none): the host asks before it chooses
 // between a fused epilogue (never split) and the plain one followed by a small kernel.
@@ -936,11 +927,13 @@ SP_API int sp_tc_gemm(const void* A, const void* W, void* C, int c_dt, int M, in
     return tc_gemm_any(A, W, C, c_dt, M, N, K, lda, ldw, ldc, mode, bn, nullptr, status, stream);
 }
 
-// mode 2 with another activation of the gate (SP_ACT_*) and a factor on the outputs
+// mode 2 with another activation of the gate (SP_ACT_*; limit and slope of the clamped one) and a factor on the outputs
 SP_API int sp_tc_gemm_gated(const void* A, const void* W, void* C, int c_dt, int M, int N, int K, int lda, int ldw, int ldc,
-                            int bn, int act, float mult, int* status, cudaStream_t stream) {
-    if (act != SP_ACT_SILU && act != SP_ACT_GELU) SP_FAIL("tc_gemm: activation code %d is not built for gated rows", act);
-    return tc_gemm_any(A, W, C, c_dt, M, N, K, lda, ldw, ldc, MODE_SILU_MUL, bn, nullptr, status, stream, act, mult);
+                            int bn, int act, float mult, float limit, float slope, int* status,
+                            cudaStream_t stream) {
+    const SpGate ga{act, mult, limit, slope};
+    if (!sp_gate_built(ga)) SP_FAIL("tc_gemm: activation code %d is not built for gated rows", act);
+    return tc_gemm_any(A, W, C, c_dt, M, N, K, lda, ldw, ldc, MODE_SILU_MUL, bn, nullptr, status, stream, ga);
 }
 
 // A grouped product on 128-row tiles of A (M a multiple of 128): row tile t multiplies with the N rows of W that begin
@@ -967,7 +960,7 @@ SP_API int sp_tc_gemm_grouped(const void* A, const void* W, void* C, int c_dt, i
 }
 
 static int tc_gemm_any(const void* A, const void* W, void* C, int c_dt, int M, int N, int K, int lda, int ldw, int ldc,
-                       int mode, int bn, const EpiArgs* epp, int* status, cudaStream_t stream, int act, float mult) {
+                       int mode, int bn, const EpiArgs* epp, int* status, cudaStream_t stream, SpGate ga) {
     EpiArgs ep;
     memset(&ep, 0, sizeof(ep));
     if (epp) ep = *epp;
@@ -995,17 +988,17 @@ static int tc_gemm_any(const void* A, const void* W, void* C, int c_dt, int M, i
     // a prompt's worth of rows: pairs of CTAs on tiles of 256 rows, each fetching half of the W tile
     if (pairs_from > 0 && M >= pairs_from) {
         if (make_map(&mw, W, N, K, ldw, bn / 2)) return 1;
-        if (bn == 128) return launch_pair<128, 8>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep, act, mult);
-        if (bn == 192) return launch_pair<192, 7>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep, act, mult);
-        return launch_pair<256, 6>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep, act, mult);
+        if (bn == 128) return launch_pair<128, 8>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep, ga);
+        if (bn == 192) return launch_pair<192, 7>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep, ga);
+        return launch_pair<256, 6>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep, ga);
     }
     if (make_map(&mw, W, N, K, ldw, bn)) return 1;
     const int splits = fused ? 1 : pick_splits(M, N, K, bn);
     if (splits > 1) {
-        if (bn == 128) return launch_splitk<128, 6>(ma, mw, C, c_dt, M, N, K, ldc, mode, splits, status, stream, act, mult);
-        return launch_splitk<256, 4>(ma, mw, C, c_dt, M, N, K, ldc, mode, splits, status, stream, act, mult);
+        if (bn == 128) return launch_splitk<128, 6>(ma, mw, C, c_dt, M, N, K, ldc, mode, splits, status, stream, ga);
+        return launch_splitk<256, 4>(ma, mw, C, c_dt, M, N, K, ldc, mode, splits, status, stream, ga);
     }
-    if (bn == 128) return launch<128, 6>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep, act, mult);
-    if (bn == 192) return launch<192, 5>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep, act, mult);
-    return launch<256, 4>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep, act, mult);
+    if (bn == 128) return launch<128, 6>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep, ga);
+    if (bn == 192) return launch<192, 5>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep, ga);
+    return launch<256, 4>(ma, mw, C, c_dt, M, N, K, ldc, mode, status, stream, ep, ga);
 }

@@ -90,8 +90,7 @@ struct Args {
     int c_dt, M, N, K, ldc, mode, pair, pieces;
     EpiArgs ep;
     SpRange rg;
-    int act;                // gated tiles: the gate's activation (SP_ACT_*) and a factor on the outputs
-    float mult;
+    SpGate ga;              // gated tiles: the gate's activation, its constants and a factor on the outputs
 };
 
 template <int NT, bool GATED>
@@ -234,7 +233,7 @@ tc_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
                 const float rs = rstd_s[j];
                 if (GATED) {
                     const float gg = g[t] * rs, uu = u[t] * rs;
-                    sp_st_dt(a.C, a.c_dt, o, sp_gated(gg, uu, a.act) * a.mult);
+                    sp_st_dt(a.C, a.c_dt, o, sp_gated(gg, uu, a.ga));
                 } else if (a.mode == MODE_ACCUMULATE) {
                     const float hn = pre.oldc[t] + g[t];
                     ((float*)a.C)[o] = hn;
@@ -537,7 +536,7 @@ SP_API int sp_tc_stream_supported(const void* A, const void* W, int M, int N, in
 
 static int tc_stream_any(const void* A, const void* W, void* C, int c_dt, int M, int N, int K, int lda, int ldw, int ldc,
                          int mode, int pair, const EpiArgs* epp, int* status, cudaStream_t stream,
-                         int act = SP_ACT_SILU, float mult = 1.0f);
+                         SpGate ga = SpGate{});
 
 // mode 0: C = A·Wᵀ (bfloat16 or float32); 1: C (float32) += A·Wᵀ; 2: W interleaves ``pair`` gate rows and ``pair``
 // up rows, C [M, N/2] = silu(gate)·up; 3: the greedy head's candidates.
@@ -547,11 +546,13 @@ SP_API int sp_tc_stream(const void* A, const void* W, void* C, int c_dt, int M, 
     return tc_stream_any(A, W, C, c_dt, M, N, K, lda, ldw, ldc, mode, pair, nullptr, status, stream);
 }
 
-// mode 2 with another activation of the gate (SP_ACT_*) and a factor on the outputs
+// mode 2 with another activation of the gate (SP_ACT_*; limit and slope of the clamped one) and a factor on the outputs
 SP_API int sp_tc_stream_gated(const void* A, const void* W, void* C, int c_dt, int M, int N, int K, int lda, int ldw, int ldc,
-                              int pair, int act, float mult, int* status, cudaStream_t stream) {
-    if (act != SP_ACT_SILU && act != SP_ACT_GELU) SP_FAIL("tc_stream: activation code %d is not built for gated rows", act);
-    return tc_stream_any(A, W, C, c_dt, M, N, K, lda, ldw, ldc, MODE_SILU_MUL, pair, nullptr, status, stream, act, mult);
+                              int pair, int act, float mult, float limit, float slope, int* status,
+                            cudaStream_t stream) {
+    const SpGate ga{act, mult, limit, slope};
+    if (!sp_gate_built(ga)) SP_FAIL("tc_stream: activation code %d is not built for gated rows", act);
+    return tc_stream_any(A, W, C, c_dt, M, N, K, lda, ldw, ldc, MODE_SILU_MUL, pair, nullptr, status, stream, ga);
 }
 
 // Floats per token that the accumulating epilogue writes into ssq_out when it prepares the next norm.
@@ -568,7 +569,7 @@ SP_API int sp_tc_stream_fused(const void* A, const void* W, void* C, int c_dt, i
 }
 
 static int tc_stream_any(const void* A, const void* W, void* C, int c_dt, int M, int N, int K, int lda, int ldw, int ldc,
-                         int mode, int pair, const EpiArgs* epp, int* status, cudaStream_t stream, int act, float mult) {
+                         int mode, int pair, const EpiArgs* epp, int* status, cudaStream_t stream, SpGate ga) {
     if (N <= 0) return 0;
     if (mode < 0 || mode > 4) SP_FAIL("tc_stream: unknown mode %d", mode);
     if (mode == MODE_ACCUMULATE && c_dt != SP_DT_F32) SP_FAIL("tc_stream: accumulation needs a float32 C");
@@ -590,7 +591,7 @@ static int tc_stream_any(const void* A, const void* W, void* C, int c_dt, int M,
     Args args;
     args.ep = ep;
     args.rg = sp_range_host;
-    args.act = act; args.mult = mult;
+    args.ga = ga;
     args.C = C; args.status = status;
     args.c_dt = c_dt; args.M = M; args.N = N; args.K = K; args.ldc = ldc; args.mode = mode; args.pair = pair;
     // the greedy head keeps candidates per tile: one CTA computes a tile over all of K

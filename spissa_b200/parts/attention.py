@@ -143,35 +143,51 @@ class GQAAttention(Mixer):
                             self.sink, self.counters)
 
 
-def attend_paged(q, step, cache, nh, nkv, hd, window, scale, sink=None, counters=None, dist_bias=None):
+def attention_modules(hd: int, vd: int) -> tuple:
+    """The kernel libraries that ``attend_paged`` needs for bfloat16 key rows of ``hd`` and value rows of ``vd`` entries."""
+    if hd == vd and hd % 16 == 0 and hd <= 128:
+        return ("attention",)
+    if hd % 8 or vd % 8 or max(hd, vd) > 128:
+        return ()
+    return ("attention_kv", "flash_tc") if hd > 32 else ("attention_kv",)
+
+
+def attend_paged(q, step, cache, nh, nkv, hd, window, scale, sink=None, counters=None, dist_bias=None, vd=None):
     """Softmax attention of the step's queries ``q`` [T, nh·hd] over the paged keys and values of ``cache`` (a
-    ``KVLayerView``; key and value rows of one size): the tensor-core kernels where they take the sizes, else the
-    generic one. ``sink``: float32 [nh] or None. ``dist_bias``: float32 [nh, distances] or None, a score added by the
-    distance between query and key. ``counters``: the arrival counters of the split-key decode kernel."""
+    ``KVLayerView``): the tensor-core kernels where they take the sizes, else the generic one. ``vd``: the size of a value
+    row where it differs from a key row's. ``sink``: float32 [nh] or None. ``dist_bias``: float32 [nh, distances] or None,
+    a score added by the distance between query and key. ``counters``: the arrival counters of the split-key decode
+    kernel."""
     T = q.shape[0]
-    ctx = torch.empty_like(q)
-    if K.flash_supported(q, cache.k_pool, nh, nkv, hd, cache.page_size):
-        if step.all_single:
-            # the split is made for the length's bucket, not the length: a step run directly and the same step
-            # replayed from a graph (captured for the bucket) then add up in the same order, bit for bit
-            chunk_tiles, n_chunks = K.flash_decode_plan(T, nkv, length_bucket(step.max_len, cache.page_size),
-                                                        cache.page_size)
-            need = K.flash_decode_scratch_floats(T, nh, hd, n_chunks)
-            scratch = torch.empty(need, dtype=torch.float32, device=q.device)
-            K.flash_decode(q, cache.k_pool, cache.v_pool, ctx, cache, step.seq_len, nh, nkv, hd, window,
-                           scale, chunk_tiles, n_chunks, scratch,
-                           counters if counters is not None and T * nkv <= counters.numel() else None, sink=sink,
-                           dist_bias=dist_bias)
-        elif T >= 256 and K.flash_tc_supported(q, cache.k_pool, nh, nkv, hd, cache.page_size, window):
-            # long prompts: 128-token tiles on the tcgen05 tensor cores (S, P and O in tensor memory)
-            tiles = K.query_tiles(step.host["new_counts"], K.flash_tc_query_tile())
-            K.flash_prefill_tc(q, cache.k_pool, cache.v_pool, ctx, cache, step.seq_start, step.n_seqs, tiles,
-                               nh, nkv, hd, window, scale, sink=sink, dist_bias=dist_bias)
-        else:
-            tiles = K.query_tiles(step.host["new_counts"], K.flash_query_tile())
-            K.flash_prefill(q, cache.k_pool, cache.v_pool, ctx, cache, step.seq_start, step.n_seqs,
-                            tiles, nh, nkv, hd, window, scale, sink=sink, dist_bias=dist_bias)
+    if vd == hd:
+        vd = None
+    ctx = torch.empty_like(q) if vd is None else torch.empty(T, nh * vd, dtype=q.dtype, device=q.device)
+    if vd is None and K.flash_supported(q, cache.k_pool, nh, nkv, hd, cache.page_size):
+        flash = {}
+    elif q.dtype == torch.bfloat16 and K.flash_kv_supported(q, cache.k_pool, nh, nkv, hd, vd or hd, cache.page_size):
+        flash = dict(vd=vd or hd)              # sizes of their own, or one that the kernels for one size are not built for
     else:
-        K.attention_generic(q, cache.k_pool, cache.v_pool, ctx, cache, nh, nkv, hd, window, scale, sink=sink,
+        K.attention_generic(q, cache.k_pool, cache.v_pool, ctx, cache, nh, nkv, hd, window, scale, vd=vd, sink=sink,
                             dist_bias=dist_bias)
+        return ctx
+    if step.all_single:
+        # the split is made for the length's bucket, not the length: a step run directly and the same step
+        # replayed from a graph (captured for the bucket) then add up in the same order, bit for bit
+        chunk_tiles, n_chunks = K.flash_decode_plan(T, nkv, length_bucket(step.max_len, cache.page_size),
+                                                    cache.page_size)
+        need = K.flash_decode_scratch_floats(T, nh, vd or hd, n_chunks)
+        scratch = torch.empty(need, dtype=torch.float32, device=q.device)
+        K.flash_decode(q, cache.k_pool, cache.v_pool, ctx, cache, step.seq_len, nh, nkv, hd, window,
+                       scale, chunk_tiles, n_chunks, scratch,
+                       counters if counters is not None and T * nkv <= counters.numel() else None, sink=sink,
+                       dist_bias=dist_bias, **flash)
+    elif T >= 256 and K.flash_tc_supported(q, cache.k_pool, nh, nkv, hd, cache.page_size, window, vd=vd):
+        # long prompts: 128-token tiles on the tcgen05 tensor cores (S, P and O in tensor memory)
+        tiles = K.query_tiles(step.host["new_counts"], K.flash_tc_query_tile())
+        K.flash_prefill_tc(q, cache.k_pool, cache.v_pool, ctx, cache, step.seq_start, step.n_seqs, tiles,
+                           nh, nkv, hd, window, scale, sink=sink, dist_bias=dist_bias, vd=vd)
+    else:
+        tiles = K.query_tiles(step.host["new_counts"], K.flash_query_tile())
+        K.flash_prefill(q, cache.k_pool, cache.v_pool, ctx, cache, step.seq_start, step.n_seqs,
+                        tiles, nh, nkv, hd, window, scale, sink=sink, dist_bias=dist_bias, **flash)
     return ctx

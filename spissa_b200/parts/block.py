@@ -221,7 +221,7 @@ class SandwichBlock(Block):
 
     with r = ``residual_mult``. The feed-forward and the ``side`` sublayer (a feed-forward part that reads the stream
     itself, not a norm of it) may be absent. ``norms`` has the places ``mixer``, ``mixer_out``, ``ffn``, ``ffn_out``
-    and ``side_out``; all are RMS norms (they hand their multiplying weight to the kernel that applies them). The
+    and ``side_out``; all are RMS norms or all layer norms (they hand their multiplying weight to the kernel that applies them). The
     sublayers keep their interface: they ADD into a 32-bit row buffer that is zero when they get it; one kernel takes
     the buffer's norm into the stream, leaves it zeroed and writes the next sublayer's input in the same pass."""
     graph_safe = True
@@ -237,9 +237,10 @@ class SandwichBlock(Block):
         self.ffn_norm = build_part("norm", norms["ffn"]) if ffn is not None else None
         self.ffn_out = build_part("norm", norms["ffn_out"]) if ffn is not None else None
         self.side_out = build_part("norm", norms["side_out"]) if side is not None else None
-        for n in (self.mixer_norm, self.mixer_out, self.ffn_norm, self.ffn_out, self.side_out):
-            if n is not None and not hasattr(n, "multiplier"):
-                raise ValueError(f"{prefix}: the norms of this arrangement are RMS norms")
+        norms = [n for n in (self.mixer_norm, self.mixer_out, self.ffn_norm, self.ffn_out, self.side_out) if n is not None]
+        if any(not hasattr(n, "multiplier") for n in norms) or len({n.centered for n in norms}) != 1:
+            raise ValueError(f"{prefix}: the norms of this arrangement are all RMS norms or all layer norms")
+        self.centered = norms[0].centered
         self.next_norm, self.takes_normed = None, False      # see ``feeds``
 
     def children(self):
@@ -252,7 +253,7 @@ class SandwichBlock(Block):
     def feeds(self, nxt) -> bool:
         """Told once, when the model is put together, that ``nxt`` always runs right behind this block on the same
         stream: this block's last pass over the stream then writes ``nxt``'s first norm as well. True if taken."""
-        if (isinstance(nxt, SandwichBlock) and nxt.hidden_size == self.hidden_size
+        if (isinstance(nxt, SandwichBlock) and nxt.hidden_size == self.hidden_size and nxt.centered == self.centered
                 and nxt.mixer_norm.eps == (self.side_out or self.ffn_out or self.mixer_out).eps):
             self.next_norm, nxt.takes_normed = nxt.mixer_norm, True
             return True
@@ -274,21 +275,23 @@ class SandwichBlock(Block):
         if self.ffn is not None:
             with phase("attention_out_norm+mlp_norm_ms"):
                 x = torch.empty(h.shape[0], W, dtype=self.rt.act_dtype, device=h.device)
-                K.stream_norm_add(h, y, last.multiplier(), r, last.eps, w_next=self.ffn_norm.multiplier(), out=x)
+                K.stream_norm_add(h, y, last.multiplier(), r, last.eps, w_next=self.ffn_norm.multiplier(), out=x,
+                                  centered=self.centered)
             self.ffn.forward(x, step, y)
             last = self.ffn_out
         with phase("out_norm_ms"):
             if self.side is None:
                 xn = torch.empty(h.shape[0], W, dtype=self.rt.act_dtype, device=h.device) if nxt is not None else None
-                K.stream_norm_add(h, y, last.multiplier(), r, last.eps, w_next=ahead, out=xn)
+                K.stream_norm_add(h, y, last.multiplier(), r, last.eps, w_next=ahead, out=xn, centered=self.centered)
                 if nxt is not None:
                     step.scratch[NORMED_STREAM] = xn
                 return
             x = torch.empty(h.shape[0], W, dtype=self.rt.act_dtype, device=h.device)
-            K.stream_norm_add(h, y, last.multiplier(), r, last.eps, out=x, raw=True)     # the side sublayer reads the stream itself
+            K.stream_norm_add(h, y, last.multiplier(), r, last.eps, out=x, raw=True,      # the side sublayer reads the stream itself
+                              centered=self.centered)
         self.side.forward(x, step, y)
         with phase("side_out_norm_ms"):
             xn = torch.empty(h.shape[0], W, dtype=self.rt.act_dtype, device=h.device) if nxt is not None else None
-            K.stream_norm_add(h, y, self.side_out.multiplier(), r, self.side_out.eps, w_next=ahead, out=xn)
+            K.stream_norm_add(h, y, self.side_out.multiplier(), r, self.side_out.eps, w_next=ahead, out=xn, centered=self.centered)
             if nxt is not None:
                 step.scratch[NORMED_STREAM] = xn

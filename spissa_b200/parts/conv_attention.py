@@ -14,7 +14,7 @@ added to the sum of the exponentials).
 Keys and values may have different sizes per head (``v_head_dim``). The last taps − 1 projected rows of a sequence are
 its state beside the paged keys and values; the convolution, the rotation and the norm run in 32-bit on the unrounded
 projections in one kernel that also writes the cache (the values already times ``out_scale``). The attention itself is
-the grouped-query mixer's: its tensor-core kernels where key and value sizes agree, else the generic one.
+the grouped-query mixer's: its tensor-core kernels where they take the sizes, else the generic one.
 """
 from __future__ import annotations
 
@@ -23,7 +23,7 @@ import math
 import torch
 
 from ..csrc import lib as K
-from .attention import GQAAttention
+from .attention import GQAAttention, attend_paged, attention_modules
 from .base import CacheBundle, KVCacheRequest, Mixer, StateRequest, WeightSpec
 from .linear import Linear
 from .registry import register_part
@@ -34,7 +34,6 @@ from ..phases import phase
 class ConvAttention(GQAAttention):
     graph_safe = True
     kernel_modules = ("hybrid",)
-    kernel_modules_bf16 = ("attention",)
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, v_head_dim: int | None = None,
                  conv_taps: int | None = None, scale: float | None = None, qk_norm_eps: float | None = None,
@@ -55,6 +54,7 @@ class ConvAttention(GQAAttention):
         if self.value_from_key and self.v_head_dim != self.head_dim:
             raise ValueError(f"{prefix}: values that are the keys have the keys' size")
         self.sink_logit = None if sink_logit is None else float(sink_logit)
+        self.kernel_modules_bf16 = attention_modules(self.head_dim, self.v_head_dim)
         self.conv = None
 
     @property
@@ -114,11 +114,6 @@ class ConvAttention(GQAAttention):
                             d, vd, rd, self.qk_norm_eps or 0.0, v_scale=self.out_scale,
                             unit_rms=self.qk_norm_eps is not None, v_from_k=self.value_from_key)
         with phase("attention_ms"):
-            if vd == d:
-                ctx = self.attend(q, step, kv)
-            else:
-                ctx = torch.empty(x.shape[0], nh * vd, dtype=self.rt.act_dtype, device=x.device)
-                K.attention_generic(q, kv.k_pool, kv.v_pool, ctx, kv, nh, nkv, d, self.window, self.scale, vd=vd,
-                                    sink=self.sink)
+            ctx = attend_paged(q, step, kv, nh, nkv, d, self.window, self.scale, self.sink, self.counters, vd=vd)
         with phase("o_projection+attention_residual_ms"):
             self.o(ctx, out=residual, accumulate=True)

@@ -71,19 +71,26 @@ class Linear:
 
 
 class GatedLinear:
-    """act(x·Wgᵀ) ⊙ (x·Wuᵀ) · mult as one product over the stacked weight (``act``: K.ACT_SILU or K.ACT_GELU).
+    """act(x·Wgᵀ) ⊙ (x·Wuᵀ) · mult as one product over the stacked weight (``act``: K.ACT_SILU or K.ACT_GELU; K.ACT_CLAMPED with
+    its ``limit`` and ``slope``: g·sigmoid(slope·g)·(u + 1), g = min(x·Wgᵀ, limit), u = clamp(x·Wuᵀ, ±limit)).
 
     When the sizes allow, gate and up rows are interleaved in blocks (``block`` gate rows, then
     the ``block`` up rows of the same outputs) so that one tile of the tensor-core kernel holds
     both halves and applies act·up in its epilogue.
     """
 
-    def __init__(self, gate: torch.Tensor, up: torch.Tensor, act: int = K.ACT_SILU, mult: float = 1.0):
+    def __init__(self, gate: torch.Tensor, up: torch.Tensor, act: int = K.ACT_SILU, mult: float = 1.0, limit: float = 0.0,
+                 slope: float = 0.0):
         I = gate.shape[0]
         self.act, self.mult = act, float(mult)
+        self.limit, self.slope = float(limit), float(slope)
+        if act == K.ACT_CLAMPED and self.mult != 1.0:
+            raise ValueError("the clamped unit takes no factor")
         self.intermediate = I
         self.block = 128 if I % 128 == 0 else 64 if I % 64 == 0 else 0
         fused = self.block and gate.dtype == torch.bfloat16 and gate.shape[1] % 8 == 0
+        if act == K.ACT_CLAMPED and not self.limit > 0:
+            fused = 0                                    # the epilogues are built for positive limits
         if fused:
             h = self.block
             g = gate.reshape(I // h, h, -1)
@@ -96,12 +103,15 @@ class GatedLinear:
 
     def __call__(self, x: torch.Tensor, act_dtype) -> torch.Tensor:
         out = torch.empty(x.shape[0], self.intermediate, dtype=act_dtype, device=x.device)
+        kw = dict(act=self.act, mult=self.mult, limit=self.limit, slope=self.slope)
         if self.block and x.shape[0] <= GATED_GEMV_TOKENS and K.gemv_supported(x, self.weight):
-            K.gemv(x, self.weight, out, K.TC_SILU_MUL, self.block, self.act, self.mult)
+            K.gemv(x, self.weight, out, K.TC_SILU_MUL, self.block, **kw)
         elif self.block and x.shape[0] <= STREAM_TOKENS and K.tc_stream_supported(x, self.weight, K.TC_SILU_MUL, self.block):
-            K.tc_stream(x, self.weight, out, K.TC_SILU_MUL, self.block, self.act, self.mult)
+            K.tc_stream(x, self.weight, out, K.TC_SILU_MUL, self.block, **kw)
         elif self.block and K.tc_gemm_supported(x, self.weight):
-            K.tc_gemm(x, self.weight, out, K.TC_SILU_MUL, 2 * self.block, self.act, self.mult)
+            K.tc_gemm(x, self.weight, out, K.TC_SILU_MUL, 2 * self.block, **kw)
+        elif self.act == K.ACT_CLAMPED:
+            K.clamped_glu(self.plain(x, out_dtype=torch.float32), out, self.limit, self.slope)     # the clamps read unrounded products
         else:
             gu = self.plain(x, out_dtype=act_dtype)
             K.gated_mul(gu, out, self.act, self.mult)

@@ -185,15 +185,15 @@ class ClampedGLU(FeedForward):
 
     def bind(self, tensors, rt):
         super().bind(tensors, rt)
-        self.gate_up = Linear(torch.cat([tensors[self.names["gate"]], tensors[self.names["up"]]], dim=0))
+        g, u = tensors[self.names["gate"]], tensors[self.names["up"]]
+        if g.dtype != u.dtype:
+            raise ValueError(f"{self.prefix}: gate and up projections must share a storage type")
+        self.gate_up = GatedLinear(g, u, K.ACT_CLAMPED, limit=self.limit, slope=self.slope)
         self.down = Linear(tensors[self.names["down"]])
 
     def forward(self, x, step, residual):
-        with phase("gate_projection+up_projection_ms"):
-            gu = self.gate_up(x, out_dtype=torch.float32)
-        with phase("activation_ms"):
-            act = torch.empty(x.shape[0], self.intermediate_size, dtype=self.rt.act_dtype, device=x.device)
-            K.clamped_glu(gu, act, self.limit, self.slope)
+        with phase("gate_projection+up_projection+activation_multiply_ms"):
+            act = self.gate_up(x, self.rt.act_dtype)
         with phase("down_projection+mlp_residual_ms"):
             self.down(act, out=residual, accumulate=True)
 

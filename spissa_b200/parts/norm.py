@@ -23,6 +23,7 @@ from .registry import register_part
 @register_part("norm", "rmsnorm")
 class RMSNorm(Norm):
     graph_safe = True
+    centered = False                  # the mean stays in (what a kernel that applies this norm inside another pass must know)
 
     def __init__(self, size: int, eps: float, prefix: str = "", weight_name: str = "weight", around_zero: bool = False,
                  weight_scale: float = 1.0):
@@ -113,6 +114,7 @@ class LayerNorm(Norm):
     sum (how the final norm of a model with several residual streams takes them in)."""
     graph_safe = True
     kernel_modules = ("hybrid",)
+    centered = True
 
     def __init__(self, size: int, eps: float, prefix: str = "", weight_name: str = "weight", streams: int = 1):
         super().__init__(prefix)
@@ -131,6 +133,15 @@ class LayerNorm(Norm):
         if self.weight is None:
             return None
         return dict(kind="layernorm", weight=self.weight, eps=self.eps, size=self.size)
+
+    def multiplier(self) -> torch.Tensor:
+        """The weight as float32 [size] (for a kernel that applies this norm inside another pass)."""
+        if self.weight.dtype == torch.float32:
+            return self.weight
+        self.weight32 = getattr(self, "weight32", None)
+        if self.weight32 is None:
+            self.weight32 = self.weight.float().contiguous()
+        return self.weight32
 
     def forward(self, h: torch.Tensor, rows: torch.Tensor | None = None) -> torch.Tensor:
         n = h.shape[0] if rows is None else rows.shape[0]

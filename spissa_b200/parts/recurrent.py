@@ -23,6 +23,13 @@ gelu branch, both of size ``width``:
     y += Wo (S_t ⊙ y_t) · out_scale.
 The convolution's last inputs are a second state, a ring of ``taps`` rows (row p mod taps holds position p's input).
 
+mLSTM (the matrix memory of xLSTM): linear attention with an exponential input gate, a forget gate and a normaliser.
+    q, k [heads·dim], v, g [heads·vdim] = projections of x (no bias), q times dim^(−1/2);  per head, with c = gate_cap:
+    i = c·tanh((Wi x + bi) / c),  f = ln sigmoid(c·tanh((Wf x + bf) / c));  m_t = max(f + m_{t-1}, i)  (m₀ = 0);
+    S_t = e^{f + m_{t-1} − m_t} S_{t-1} + e^{i − m_t} k vᵀ,  n_t likewise with k alone  (S₀ = 0, n₀ = 0);
+    o = S_tᵀ q / (max(|n_t · q|, e^{−m_t}) + 1e-6),  ô = o / sqrt(mean(o²) + eps) per head;
+    y_t = Wo · ( concat_h(ô) ⊙ w ⊙ sigmoid(g) )   (w over all heads).
+
 All states are 32-bit and belong to the sequence's slot; the recurrences run in 32-bit on the unrounded
 projections, which are one matrix product over the stacked weights.
 """
@@ -227,5 +234,56 @@ class RGLRU(Mixer):
             ring = cache.get("conv")
             K.rglru(p, self.w, ring.state if ring is not None else None, cache["state"].state, y, step, self.width, self.taps,
                     self.parts, self.out_scale)
+        with phase("o_projection+mixer_residual_ms"):
+            self.o(y, out=residual, accumulate=True)
+
+
+@register_part("mixer", "mlstm")
+class MLSTM(Mixer):
+    graph_safe = True
+    kernel_modules = ("mlstm",)
+
+    def __init__(self, hidden_size: int, num_heads: int, dim: int, vdim: int, gate_cap: float, eps: float, prefix: str = "",
+                 names: dict | None = None):
+        super().__init__(prefix)
+        self.hidden_size, self.num_heads, self.dim, self.vdim = int(hidden_size), int(num_heads), int(dim), int(vdim)
+        self.gate_cap, self.eps = float(gate_cap), float(eps)
+        if not self.gate_cap > 0:
+            raise ValueError(f"{prefix}: the cap of the gates must be positive")
+        n = dict(q="q", k="k", v="v", g="g", o="o", i="i", ib="i.b", f="f", fb="f.b", norm="norm")
+        n.update(names or {})
+        self.names = {k: prefix + v for k, v in n.items()}
+        self.proj = self.o = self.w = None
+
+    def weight_specs(self):
+        H, nh, d, vd, n = self.hidden_size, self.num_heads, self.dim, self.vdim, self.names
+        return [WeightSpec(n["q"], (nh * d, H)), WeightSpec(n["k"], (nh * d, H)), WeightSpec(n["v"], (nh * vd, H)),
+                WeightSpec(n["g"], (nh * vd, H)), WeightSpec(n["o"], (H, nh * vd)), WeightSpec(n["norm"], (nh * vd,), init="ones"),
+                WeightSpec(n["i"], (nh, H)), WeightSpec(n["ib"], (nh,)), WeightSpec(n["f"], (nh, H)), WeightSpec(n["fb"], (nh,))]
+
+    def cache_request(self):
+        return CacheBundle.of(state=StateRequest((self.num_heads, self.dim, self.vdim), torch.float32),
+                              nm=StateRequest((self.num_heads, self.dim + 1), torch.float32))
+
+    def bind(self, tensors, rt):
+        super().bind(tensors, rt)
+        n = self.names
+        parts = [tensors[n[k]] for k in ("q", "k", "v", "g", "i", "f")]
+        if len({p.dtype for p in parts}) != 1:
+            raise ValueError(f"{self.prefix}: the projections of one input must share a storage type")
+        rows = sum(p.shape[0] for p in parts)
+        if rows % 4:                                     # the kernels' 16-byte pieces want rows of a multiple of four numbers
+            parts.append(torch.zeros(4 - rows % 4, self.hidden_size, dtype=parts[0].dtype, device=parts[0].device))
+        self.proj = Linear(torch.cat(parts, dim=0))
+        self.o = Linear(tensors[n["o"]])
+        self.w = {k: tensors[n[k]].float().contiguous() for k in ("ib", "fb", "norm")}
+
+    def forward(self, x, step, cache, residual):
+        with phase("mixer_projection_ms"):
+            p = self.proj(x, out_dtype=torch.float32)              # the gates and the memory read unrounded products
+        with phase("mlstm_ms"):
+            y = torch.empty(x.shape[0], self.num_heads * self.vdim, dtype=self.rt.act_dtype, device=x.device)
+            K.mlstm(p, self.w, cache["state"].state, cache["nm"].state, y, step, self.num_heads, self.dim, self.vdim,
+                    self.gate_cap, self.eps)
         with phase("o_projection+mixer_residual_ms"):
             self.o(y, out=residual, accumulate=True)
