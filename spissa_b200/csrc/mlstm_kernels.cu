@@ -68,8 +68,8 @@ template <int CT>
 __global__ void __launch_bounds__(MG_WARPS * 32) mlstm_gates_kernel(MlArgs a) {
     constexpr int PL = CT / 32;
     __shared__ double sumF[MG_WARPS], topA[MG_WARPS], m0s[MG_WARPS], m_run;
-    sp_allow_dependents();
     sp_wait_for_predecessor();
+    sp_allow_dependents();               // in this order: whoever starts from here on may read the projections at once
     const int s = blockIdx.x, h = blockIdx.y;
     const int slot = a.seq_slot[s];
     if (slot < 0 || slot >= a.n_slots) return;
@@ -212,8 +212,8 @@ __global__ void __launch_bounds__(256) mlstm_sum_kernel(MlArgs a) {
 // of the value columns leave as sums of two bfloat16 numbers, the high one in the lower half of a word, the low one above it.
 template <bool PACK>
 __global__ void __launch_bounds__(256) mlstm_scan_kernel(MlArgs a, int ct) {
-    sp_allow_dependents();
     sp_wait_for_predecessor();
+    sp_allow_dependents();               // whoever starts from here on may read the projections and the gates at once
     const int s = blockIdx.x, h = blockIdx.y;
     const int x = blockIdx.z * 256 + threadIdx.x;
     if (x >= a.d * a.vc) return;
@@ -355,15 +355,29 @@ __device__ __forceinline__ void load8(const float* p, bool in, float (&f)[8]) {
 }
 __device__ __forceinline__ void proxy_fence() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
 
-// a chunk's values, columns c0 .. c0 + nb - 1 of head h, as boxes of 64 columns: one row per token (the product's K)
-__device__ __forceinline__ void fill_values(const MlArgs& a, uint8_t* dst, int h, int t0, int n, int c0, int nb) {
-#pragma unroll 8
-    for (int u = 0; u < 16; ++u) {
-        const int x = threadIdx.x + 256 * u, j = x >> 5, c = x & 31, col = c0 + 8 * c;
-        if (8 * c >= nb) continue;
-        float f[8];
-        load8(a.proj + (size_t)(t0 + j) * a.ld + 2 * a.H * a.d + (size_t)h * a.vd + col, j < n && col < a.vd, f);
-        *(uint4*)(dst + (c >> 3) * BOX + sw_at(j, c & 7)) = pack8(f);
+// A chunk's values, columns c0 .. c0 + nb - 1 of head h, as boxes of 64 columns with one row per token (the product's K):
+// sixteen pieces of eight numbers per thread, pieces U0 .. U0 + N - 1 of them. All of a batch's loads come before its stores,
+// which the compiler would not let them pass.
+template <int N>
+__device__ __forceinline__ void load_values(const MlArgs& a, float4 (&r)[2 * N], int u0, int h, int t0, int n, int c0, int nb) {
+#pragma unroll
+    for (int u = 0; u < N; ++u) {
+        const int x = threadIdx.x + 256 * (u0 + u), j = x >> 5, col = c0 + 8 * (x & 31);
+        const float4* p = (const float4*)(a.proj + (size_t)(t0 + j) * a.ld + 2 * a.H * a.d + (size_t)h * a.vd + col);
+        const bool in = j < n && col < a.vd;
+        r[2 * u] = in ? p[0] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        r[2 * u + 1] = in ? p[1] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    }
+}
+__device__ __forceinline__ uint4 pack8(const float4& a, const float4& b) {
+    return make_uint4(pack_bf16(a.x, a.y), pack_bf16(a.z, a.w), pack_bf16(b.x, b.y), pack_bf16(b.z, b.w));
+}
+template <int N>
+__device__ __forceinline__ void store_values(uint8_t* dst, const float4 (&r)[2 * N], int u0, int nb) {
+#pragma unroll
+    for (int u = 0; u < N; ++u) {
+        const int x = threadIdx.x + 256 * (u0 + u), j = x >> 5, c = x & 31;
+        if (8 * c < nb) *(uint4*)(dst + (c >> 3) * BOX + sw_at(j, c & 7)) = pack8(r[2 * u], r[2 * u + 1]);
     }
 }
 
@@ -394,7 +408,6 @@ __global__ void __launch_bounds__(256) mlstm_sum_tc_kernel(MlArgs a) {
     tc_fence_after();
     const uint32_t tmem = tmem_slot;
     sp_allow_dependents();
-    sp_wait_for_predecessor();
     int s, t0 = 0, n = 0;
     const bool live = ml_chunk_of(a, blockIdx.x, TK, s, t0, n);
     const int h = blockIdx.y, cb = (a.vd + 255) / 256;
@@ -402,27 +415,39 @@ __global__ void __launch_bounds__(256) mlstm_sum_tc_kernel(MlArgs a) {
     const int nb = (min(256, a.vd - c0) + 15) / 16 * 16;
     float* out = a.cs + ((size_t)blockIdx.x * a.H + h) * a.d * a.vc;
     if (live) {
+        // keys and values come from the projections, which are complete when this kernel starts; the gates are waited for
         const int c8 = threadIdx.x & 15, tg = threadIdx.x >> 4, e = e0 + 8 * c8;
-        float ns[8] = {};
-#pragma unroll 4
+        float4 kr[16], vr[16];
+#pragma unroll
         for (int u = 0; u < 8; ++u) {
             const int j = tg + 16 * u;
             const bool in = j < n && e < a.d;
-            float f[8];
-            load8(a.proj + (size_t)(t0 + j) * a.ld + (size_t)(a.H + h) * a.d + e, in, f);
-            const float w = in ? a.we[(size_t)h * a.T + t0 + j] : 0.0f;
+            const float4* p = (const float4*)(a.proj + (size_t)(t0 + j) * a.ld + (size_t)(a.H + h) * a.d + e);
+            kr[2 * u] = in ? p[0] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            kr[2 * u + 1] = in ? p[1] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        }
+        load_values<8>(a, vr, 0, h, t0, n, c0, nb);
+        store_values<8>(vs, vr, 0, nb);
+        load_values<8>(a, vr, 8, h, t0, n, c0, nb);
+        sp_wait_for_predecessor();
+        float ns[8] = {}, w[8];
+#pragma unroll
+        for (int u = 0; u < 8; ++u) w[u] = tg + 16 * u < n ? a.we[(size_t)h * a.T + t0 + tg + 16 * u] : 0.0f;
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+            float f[8] = {kr[2 * u].x, kr[2 * u].y, kr[2 * u].z, kr[2 * u].w, kr[2 * u + 1].x, kr[2 * u + 1].y, kr[2 * u + 1].z, kr[2 * u + 1].w};
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
-                f[i] *= w;
+                f[i] *= w[u];
                 ns[i] += f[i];
             }
             const uint4 hi = pack8(f);
             low_parts(f, hi);
-            const uint32_t at = (uint32_t)((c8 >> 3) * BOX) + sw_at(j, c8 & 7);
+            const uint32_t at = (uint32_t)((c8 >> 3) * BOX) + sw_at(tg + 16 * u, c8 & 7);
             *(uint4*)(kh + at) = hi;
             *(uint4*)(kl + at) = pack8(f);
         }
-        fill_values(a, vs, h, t0, n, c0, nb);
+        store_values<8>(vs, vr, 8, nb);
 #pragma unroll
         for (int i = 0; i < 8; ++i) part[tg][8 * c8 + i] = ns[i];
         proxy_fence();
@@ -474,6 +499,8 @@ __global__ void __launch_bounds__(256) mlstm_sum_tc_kernel(MlArgs a) {
 // rows. With one column block the denominator, the unit rms, weight and gate follow here, else the raw outputs leave.
 // grid (chunks, H, column blocks of 256)
 constexpr int OT_STAGE = 2 * BOX + 2 * 32768;
+constexpr int OT_LD = 260;                    // floats of a row of outputs in shared memory (rows 16 bytes apart in the banks)
+static_assert(TK * OT_LD * 4 <= 2 * OT_STAGE, "the outputs reuse the operands' stages");
 __global__ void __launch_bounds__(256) mlstm_out_tc_kernel(MlArgs a) {
     extern __shared__ uint8_t smem_raw[];
     __shared__ __align__(8) uint64_t bar_free[2], bar_a, bar_o;
@@ -502,7 +529,6 @@ __global__ void __launch_bounds__(256) mlstm_out_tc_kernel(MlArgs a) {
     const uint32_t tmem = tmem_slot;
     constexpr uint32_t COL_A = 0, COL_PH = 128, COL_PL = 192, COL_O = 256;
     sp_allow_dependents();
-    sp_wait_for_predecessor();
     int s, t0 = 0, n = 0;
     const bool live = ml_chunk_of(a, blockIdx.x, TK, s, t0, n);
     if (live) {
@@ -512,40 +538,76 @@ __global__ void __launch_bounds__(256) mlstm_out_tc_kernel(MlArgs a) {
         const uint32_t lanes = (uint32_t)((warp & 3) * 32) << 16;
         const float qscale = 1.0f / sqrtf((float)d);
         const bool mine = row < n;
-        const size_t at = (size_t)h * a.T + t0 + (mine ? row : 0);
-        const float2 M = a.M2[at];
-        const float rq = a.r[at] * qscale, em = a.em[at];
-        if (threadIdx.x < TK) aj[threadIdx.x] = (int)threadIdx.x < n ? a.a2[(size_t)h * a.T + t0 + threadIdx.x] : make_float2(0.0f, 0.0f);
         const float* cs = a.cs + ((size_t)blockIdx.x * a.H + h) * d * a.vc;
         const uint32_t id_a = umma_idesc_bf16(TK, TK), id_o = umma_idesc_bf16_bmn(TK, nb);
         const int nE = (d + 63) / 64;
         bool ok = true;
         float dot = 0.0f;
-        for (int eb = 0; eb < nE; ++eb) {
-            uint8_t *q = sm + (eb & 1) * OT_STAGE, *k = q + BOX, *sh = q + 2 * BOX, *sl = sh + 32768;
-            if (eb >= 2) ok = mbar_wait_flag(smem_u32(&bar_free[eb & 1]), (uint32_t)((eb >> 1) - 1) & 1u, a.status, 152, &gave_up) && ok;
+        // 512 bytes of operands per thread: q, k and the start state of a block of key dims, in the end the values; the next
+        // ones are asked for before the products of the ones at hand begin
+        float4 buf[32];
+        const float4 z4 = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        auto load_qk = [&](int eb) {
 #pragma unroll
             for (int u = 0; u < 4; ++u) {
-                const int x = threadIdx.x + 256 * u, j = x >> 3, c = x & 7, e = eb * 64 + 8 * c;
-                const float* src = a.proj + (size_t)(t0 + j) * a.ld + (size_t)h * d + e;
-                float f[8], g[8];
-                load8(src, j < n && e < d, f);
-                load8(src + (size_t)a.H * d, j < n && e < d, g);
-                *(uint4*)(q + sw_at(j, c)) = pack8(f);
-                *(uint4*)(k + sw_at(j, c)) = pack8(g);
+                const int x = threadIdx.x + 256 * u, j = x >> 3, e = eb * 64 + 8 * (x & 7);
+                const bool in = j < n && e < d;
+                const float4 *pq = (const float4*)(a.proj + (size_t)(t0 + j) * a.ld + (size_t)h * d + e), *pk = (const float4*)((const float*)pq + (size_t)a.H * d);
+                buf[4 * u] = in ? pq[0] : z4;
+                buf[4 * u + 1] = in ? pq[1] : z4;
+                buf[4 * u + 2] = in ? pk[0] : z4;
+                buf[4 * u + 3] = in ? pk[1] : z4;
             }
+        };
+        auto load_state = [&](int eb) {
 #pragma unroll
             for (int u = 0; u < 8; ++u) {
-                const int x = threadIdx.x + 256 * u, r = x >> 5, c = x & 31, e = eb * 64 + r, col = c0 + 8 * c;
-                if (8 * c >= nb) continue;
+                const int x = threadIdx.x + 256 * u, e = eb * 64 + (x >> 5), col = c0 + 8 * (x & 31);
                 const bool in = e < d && col < a.vd;
-                const uint4 z = make_uint4(0u, 0u, 0u, 0u);
-                const uint4 w0 = in ? *(const uint4*)(cs + (size_t)e * a.vc + col) : z, w1 = in ? *(const uint4*)(cs + (size_t)e * a.vc + col + 4) : z;
+                const float4* p = (const float4*)(cs + (size_t)e * a.vc + col);
+                buf[16 + 2 * u] = in ? p[0] : z4;
+                buf[17 + 2 * u] = in ? p[1] : z4;
+            }
+        };
+        auto store_qk = [&](uint8_t* q, uint8_t* k) {
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                const int x = threadIdx.x + 256 * u;
+                *(uint4*)(q + sw_at(x >> 3, x & 7)) = pack8(buf[4 * u], buf[4 * u + 1]);
+                *(uint4*)(k + sw_at(x >> 3, x & 7)) = pack8(buf[4 * u + 2], buf[4 * u + 3]);
+            }
+        };
+        auto store_state = [&](uint8_t* sh, uint8_t* sl) {
+#pragma unroll
+            for (int u = 0; u < 8; ++u) {
+                const int x = threadIdx.x + 256 * u, r = x >> 5, c = x & 31;
+                if (8 * c >= nb) continue;
+                const uint4 w0 = *(const uint4*)&buf[16 + 2 * u], w1 = *(const uint4*)&buf[17 + 2 * u];
                 const uint32_t to = (uint32_t)((c >> 3) * 8192) + sw_at(r, c & 7);
                 *(uint4*)(sh + to) = make_uint4(__byte_perm(w0.x, w0.y, 0x5410), __byte_perm(w0.z, w0.w, 0x5410), __byte_perm(w1.x, w1.y, 0x5410), __byte_perm(w1.z, w1.w, 0x5410));
                 *(uint4*)(sl + to) = make_uint4(__byte_perm(w0.x, w0.y, 0x7632), __byte_perm(w0.z, w0.w, 0x7632), __byte_perm(w1.x, w1.y, 0x7632), __byte_perm(w1.z, w1.w, 0x7632));
             }
+        };
+        // the projections and the gates are complete when this kernel starts; the start states are waited for
+        load_qk(0);
+        const size_t at = (size_t)h * a.T + t0 + (mine ? row : 0);
+        const float2 M = a.M2[at];
+        const float rq = a.r[at] * qscale, em = a.em[at];
+        if (threadIdx.x < TK) aj[threadIdx.x] = (int)threadIdx.x < n ? a.a2[(size_t)h * a.T + t0 + threadIdx.x] : make_float2(0.0f, 0.0f);
+        sp_wait_for_predecessor();
+        load_state(0);
+        for (int eb = 0; eb < nE; ++eb) {
+            uint8_t *q = sm + (eb & 1) * OT_STAGE, *k = q + BOX, *sh = q + 2 * BOX, *sl = sh + 32768;
+            if (eb >= 2) ok = mbar_wait_flag(smem_u32(&bar_free[eb & 1]), (uint32_t)((eb >> 1) - 1) & 1u, a.status, 152, &gave_up) && ok;
             if (threadIdx.x < 64) nvec[eb & 1][threadIdx.x] = eb * 64 + (int)threadIdx.x < d ? cs[(size_t)(eb * 64 + threadIdx.x) * a.vc + a.vd] : 0.0f;
+            store_qk(q, k);
+            store_state(sh, sl);
+            if (eb + 1 < nE) {
+                load_qk(eb + 1);
+                load_state(eb + 1);
+            } else {
+                load_values<16>(a, buf, 0, h, t0, n, c0, nb);
+            }
             proxy_fence();
             __syncthreads();
             if (threadIdx.x == 0) {
@@ -575,7 +637,7 @@ __global__ void __launch_bounds__(256) mlstm_out_tc_kernel(MlArgs a) {
         // the values go where block nE - 2 was
         uint8_t* vs = sm + (nE & 1) * OT_STAGE;
         if (nE >= 2) ok = mbar_wait_flag(smem_u32(&bar_free[nE & 1]), (uint32_t)((nE - 2) >> 1) & 1u, a.status, 152, &gave_up) && ok;
-        fill_values(a, vs, h, t0, n, c0, nb);
+        store_values<16>(vs, buf, 0, nb);
         proxy_fence();
         ok = mbar_wait_flag(smem_u32(&bar_a), 0, a.status, 153, &gave_up) && ok;
         tc_fence_after();
@@ -646,33 +708,42 @@ __global__ void __launch_bounds__(256) mlstm_out_tc_kernel(MlArgs a) {
             __syncthreads();
             f = inv_den / sqrtf((ss_s[0][row] + ss_s[1][row]) / (float)a.vd + a.eps);
         }
-        const float* g = a.proj + (size_t)(t0 + row) * a.ld + 2 * a.H * d + (size_t)(a.H + h) * a.vd + c0;
-        const float* nw = (const float*)a.nw + (size_t)h * a.vd + c0;
         float* raw = a.raw + ((size_t)(t0 + row) * a.H + h) * a.vc;
         if (!whole && ok && mine && c0 == 0 && hh == 0) raw[a.vd] = qn;
+        // the rows pass through shared memory (all products have read theirs), so that gates and outputs move as whole lines
+        float* rows = (float*)sm;
 #pragma unroll 1
         for (int c = hh * 32; c < nb; c += 64) {
             uint32_t x[32];
             tc_ld_32x32(tmem + lanes + COL_O + c, x);
             tc_ld_wait();
-            if (!ok || !mine) continue;
 #pragma unroll
-            for (int i = 0; i < 32; i += 8) {
-                if (c + i >= nv) break;
+            for (int i = 0; i < 32; i += 4)
+                *(float4*)(rows + row * OT_LD + c + i) = make_float4(__uint_as_float(x[i]) * f, __uint_as_float(x[i + 1]) * f,
+                                                                     __uint_as_float(x[i + 2]) * f, __uint_as_float(x[i + 3]) * f);
+        }
+        __syncthreads();
+        const int col = lane * 8;
+        if (ok && col < nv) {
+            float wv[8];
+            load8((const float*)a.nw + (size_t)h * a.vd + c0 + col, true, wv);
+#pragma unroll 4
+            for (int u = 0; u < TK / 8; ++u) {
+                const int j = warp + 8 * u;
+                if (j >= n) break;
+                const size_t to = (size_t)(t0 + j) * a.H + h;
                 float y[8];
-#pragma unroll
-                for (int v = 0; v < 8; ++v) y[v] = __uint_as_float(x[i + v]);
+                load8(rows + j * OT_LD + col, true, y);
                 if (!whole) {
-                    *(float4*)(raw + c0 + c + i) = make_float4(y[0], y[1], y[2], y[3]);
-                    *(float4*)(raw + c0 + c + i + 4) = make_float4(y[4], y[5], y[6], y[7]);
+                    *(float4*)(a.raw + to * a.vc + c0 + col) = make_float4(y[0], y[1], y[2], y[3]);
+                    *(float4*)(a.raw + to * a.vc + c0 + col + 4) = make_float4(y[4], y[5], y[6], y[7]);
                     continue;
                 }
-                float gv[8], wv[8];
-                load8(g + c + i, true, gv);
-                load8(nw + c + i, true, wv);
+                float gv[8];
+                load8(a.proj + (size_t)(t0 + j) * a.ld + 2 * a.H * d + (size_t)(a.H + h) * a.vd + col, true, gv);
 #pragma unroll
-                for (int v = 0; v < 8; ++v) y[v] = y[v] * f * wv[v] / (1.0f + expf(-gv[v]));
-                *(uint4*)((__nv_bfloat16*)a.out + ((size_t)(t0 + row) * a.H + h) * a.vd + c + i) = pack8(y);
+                for (int v = 0; v < 8; ++v) y[v] = y[v] * wv[v] / (1.0f + expf(-gv[v]));
+                *(uint4*)((__nv_bfloat16*)a.out + to * a.vd + col) = pack8(y);
             }
         }
     }
@@ -687,16 +758,13 @@ __global__ void __launch_bounds__(256) mlstm_out_tc_kernel(MlArgs a) {
 // ============================================================== one token per sequence
 // A cluster of CTAs per (head, sequence) shares the value columns out; each streams its columns of S once (on their way
 // into L2 before the projections are there), all compute n · q, the first one writes n
-// and m once everybody has read them, and the squares of the head's outputs meet in distributed shared memory.
-__device__ __forceinline__ void cluster_sync_all() {
-    asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
-}
-__device__ __forceinline__ float peer_shared_f32(const float* p, uint32_t rank) {
-    uint32_t addr = smem_u32(p), remote;
-    float v;
-    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(addr), "r"(rank));
-    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(remote) : "memory");
-    return v;
+// and m once everybody has read them, and every CTA sends the squares of its outputs to all others' shared memory.
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
+__device__ __forceinline__ void store_peer_f32(float* p, uint32_t rank, float v) {
+    uint32_t remote;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(smem_u32(p)), "r"(rank));
+    asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(remote), "f"(v) : "memory");
 }
 
 constexpr int MS_COLS = 32;        // value columns of a CTA and pass
@@ -704,12 +772,13 @@ constexpr int MS_COLS = 32;        // value columns of a CTA and pass
 template <int VEC>
 __global__ void __launch_bounds__(256) mlstm_step_kernel(MlArgs a, int cz) {
     constexpr int XT = MS_COLS / VEC, ROWS = 256 / XT, AHEAD = 4;
+    constexpr int PARTS = VEC == 4 ? 8 : ROWS;            // partial sums of a column that meet in shared memory
     extern __shared__ __align__(16) float sm[];
     float* qs = sm;                      // [d]
-    float* ks = qs + a.d;                // [d]
-    float* red = ks + a.d;               // [ROWS][32]
-    float* oc = red + ROWS * MS_COLS;    // [column passes][32] this CTA's outputs
-    __shared__ float scratch[32], ssq;
+    float* ks = qs + ((a.d + 3) & ~3);   // [d]
+    float* red = ks + ((a.d + 3) & ~3);  // [PARTS][32]
+    float* oc = red + PARTS * MS_COLS;   // [column passes][32] this CTA's outputs
+    __shared__ float scratch[32], ssq[8];
     const int rank = blockIdx.x, h = blockIdx.y, s = blockIdx.z;
     const int x = threadIdx.x % XT, y = threadIdx.x / XT;
     const int d = a.d, vd = a.vd, Hd = a.H * d, Hv = a.H * vd;
@@ -732,6 +801,7 @@ __global__ void __launch_bounds__(256) mlstm_step_kernel(MlArgs a, int cz) {
         }
     };
     sp_allow_dependents();
+    if (cz > 1) cluster_arrive();                         // everybody has started: waited for before anything is sent
     for (int e = threadIdx.x; e < d; e += 256)            // the first pass's columns on their way into L2
         if (rank * MS_COLS < vd) asm volatile("prefetch.global.L2 [%0];" ::"l"(gS + (size_t)e * vd + rank * MS_COLS));
     sp_wait_for_predecessor();
@@ -750,6 +820,14 @@ __global__ void __launch_bounds__(256) mlstm_step_kernel(MlArgs a, int cz) {
         qs[e] = q;
         ks[e] = take * k;
         nq = fmaf(fmaf(keep, gn[e], take * k), q, nq);
+    }
+    // the output's gate and weight of the first pass, asked for ahead of their use
+    const float* g = row + 2 * Hd + Hv + (size_t)h * vd;
+    const int own = rank * MS_COLS + threadIdx.x;
+    float gate = 0.0f, weight = 0.0f;
+    if (threadIdx.x < MS_COLS && own < vd) {
+        gate = g[own];
+        weight = sp_ld_dt(a.nw, a.w_dt, (size_t)h * vd + own);
     }
     nq = sp_block_sum(nq, scratch);
     const float inv_den = 1.0f / (fmaxf(fabsf(nq), expf(-m1)) + 1e-6f);
@@ -778,44 +856,56 @@ __global__ void __launch_bounds__(256) mlstm_step_kernel(MlArgs a, int cz) {
                 else gS[(size_t)e * vd + col] = st[u][0];
             }
         }
+        if (VEC == 4) {                                         // the four rows that a warp holds of a column
 #pragma unroll
-        for (int c = 0; c < VEC; ++c) red[y * MS_COLS + x * VEC + c] = part[c];
+            for (int c = 0; c < VEC; ++c) {
+                part[c] += __shfl_xor_sync(0xffffffffu, part[c], 8);
+                part[c] += __shfl_xor_sync(0xffffffffu, part[c], 16);
+            }
+            if ((threadIdx.x & 31) < 8) *(float4*)(red + (threadIdx.x >> 5) * MS_COLS + x * 4) = make_float4(part[0], part[VEC > 1 ? 1 : 0], part[VEC > 2 ? 2 : 0], part[VEC > 3 ? 3 : 0]);
+        } else {
+            red[y * MS_COLS + x] = part[0];
+        }
         __syncthreads();
         if (threadIdx.x < MS_COLS) {
             float o = 0.0f;
-            for (int r = 0; r < ROWS; ++r) o += red[r * MS_COLS + threadIdx.x];
+#pragma unroll
+            for (int r = 0; r < PARTS; ++r) o += red[r * MS_COLS + threadIdx.x];
             o *= inv_den;
             oc[p * MS_COLS + threadIdx.x] = o;
             ss = fmaf(o, o, ss);                                // columns beyond vd hold zeros
         }
-        __syncthreads();
+        if (p + 1 < passes) __syncthreads();
     }
-    if (threadIdx.x < 32) {
-        ss = sp_warp_sum(ss);
-        if (threadIdx.x == 0) ssq = ss;
-    }
-    __syncthreads();
-    float sum = ssq;
+    if (threadIdx.x < 32) ss = sp_warp_sum(ss);
+    float sum = 0.0f;
     if (cz > 1) {
-        cluster_sync_all();                                     // every CTA has read n and m and left its squares
-        sum = 0.0f;
-        for (int c = 0; c < cz; ++c) sum += peer_shared_f32(&ssq, (uint32_t)c);
+        cluster_wait();
+        if ((int)threadIdx.x < cz) store_peer_f32(&ssq[rank], threadIdx.x, ss);
+        cluster_arrive();                                       // every CTA has read n and m and sent its squares
+        cluster_wait();
+        for (int c = 0; c < cz; ++c) sum += ssq[c];
+    } else {
+        if (threadIdx.x == 0) ssq[0] = ss;
+        __syncthreads();
+        sum = ssq[0];
     }
     const float f = 1.0f / sqrtf(sum / (float)vd + a.eps);
-    const float* g = row + 2 * Hd + Hv + (size_t)h * vd;
     if (live) {
         for (int p = 0; p < passes; ++p) {
             const int col = (p * cz + rank) * MS_COLS + threadIdx.x;
-            if (threadIdx.x < MS_COLS && col < vd)
-                sp_st_dt(a.out, a.out_dt, (size_t)t * Hv + (size_t)h * vd + col,
-                         oc[p * MS_COLS + threadIdx.x] * f * sp_ld_dt(a.nw, a.w_dt, (size_t)h * vd + col) / (1.0f + expf(-g[col])));
+            if (threadIdx.x >= MS_COLS || col >= vd) break;
+            if (p) {
+                gate = g[col];
+                weight = sp_ld_dt(a.nw, a.w_dt, (size_t)h * vd + col);
+            }
+            sp_st_dt(a.out, a.out_dt, (size_t)t * Hv + (size_t)h * vd + col, oc[p * MS_COLS + threadIdx.x] * f * weight / (1.0f + expf(-gate)));
         }
         if (rank == 0) {
             for (int e = threadIdx.x; e < d; e += 256) gn[e] = fmaf(keep, gn[e], ks[e]);
             if (threadIdx.x == 0) gn[d] = m1;
         }
     }
-    if (cz > 1) cluster_sync_all();                             // nobody leaves while a peer still reads its squares
 }
 
 long long up4(long long n) { return (n + 3) / 4 * 4; }
@@ -853,8 +943,7 @@ SP_API int sp_mlstm(const float* proj, int ld, const void* ib, const void* fb, c
         cz = cz >= 8 ? 8 : cz >= 4 ? 4 : cz >= 2 ? 2 : 1;
         const int passes = (vd + MS_COLS * cz - 1) / (MS_COLS * cz);
         const bool vec = vd % 4 == 0 && ((uintptr_t)S & 15) == 0;
-        const int rows = vec ? 32 : 8;
-        const size_t smem = ((size_t)2 * d + (size_t)(rows + passes) * MS_COLS) * sizeof(float);
+        const size_t smem = ((size_t)2 * up4(d) + (size_t)(8 + passes) * MS_COLS) * sizeof(float);
         if (smem > 48 * 1024) SP_FAIL("mlstm (step): heads of %d x %d are beyond this kernel's range", d, vd);
         if (vec) SP_CHECK_CALL("mlstm_step", sp_launch_cluster(mlstm_step_kernel<4>, dim3(cz, H, B), dim3(256), smem, stream, -cz, a, cz));
         else SP_CHECK_CALL("mlstm_step", sp_launch_cluster(mlstm_step_kernel<1>, dim3(cz, H, B), dim3(256), smem, stream, -cz, a, cz));

@@ -158,9 +158,91 @@ __global__ void __launch_bounds__(256) stream_norm_add_kernel(NormAddArgs a) {
     }
 }
 
-// The same with layer norms: (v − mean) / sqrt(mean((v − mean)²) + eps) ⊙ w for the output and for the next reader. Rows of
-// up to NV · 1,024 numbers stay in registers between the passes (NV 0: any width, re-read).
+// The same with layer norms: (v − mean) / sqrt(mean((v − mean)²) + eps) ⊙ w for the output and for the next reader.
+// Widths of 512 · NV: a block of 128 threads per row, the row in registers, mean and squared deviations of equal parts merged
+// pair by pair (each part's are its own, so nothing cancels): one exchange through shared memory per norm.
+struct MeanDev { float mean, dev; };              // of n numbers: their mean, the sum of their squared deviations from it
+__device__ __forceinline__ MeanDev merge_equal(MeanDev a, MeanDev b, float n) {      // n: numbers in each part
+    const float d = b.mean - a.mean;
+    return MeanDev{0.5f * (a.mean + b.mean), a.dev + b.dev + 0.5f * n * d * d};
+}
+template <int N>
+__device__ __forceinline__ MeanDev block_mean_dev(const float4 (&v)[N], MeanDev* red) {
+    float s = 0.0f;
+#pragma unroll
+    for (int i = 0; i < N; ++i) s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+    MeanDev m{s * (1.0f / (4 * N)), 0.0f};
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+        const float p = v[i].x - m.mean, q = v[i].y - m.mean, r = v[i].z - m.mean, u = v[i].w - m.mean;
+        m.dev += (p * p + q * q) + (r * r + u * u);
+    }
+    float n = 4.0f * N;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1, n *= 2.0f)
+        m = merge_equal(m, MeanDev{__shfl_xor_sync(0xffffffffu, m.mean, o), __shfl_xor_sync(0xffffffffu, m.dev, o)}, n);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = m;
+    __syncthreads();
+    return merge_equal(merge_equal(red[0], red[1], n), merge_equal(red[2], red[3], n), 2.0f * n);
+}
+
 template <int NV>
+__global__ void __launch_bounds__(128) stream_layernorm_add_rows_kernel(NormAddArgs a) {
+    __shared__ MeanDev red[2][4];
+    sp_allow_dependents();
+    sp_wait_for_predecessor();
+    const int t = blockIdx.x;
+    if (t >= a.T) return;
+    float4* __restrict__ xr = (float4*)(a.x + (size_t)t * a.W) + threadIdx.x;
+    float4* __restrict__ yr = (float4*)(a.y + (size_t)t * a.W) + threadIdx.x;
+    const float4* __restrict__ w1 = (const float4*)a.w_post + threadIdx.x;
+    float4 v[NV], x[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) v[i] = yr[128 * i];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) x[i] = xr[128 * i];
+    const float invW = 1.0f / (float)a.W;
+    const MeanDev m = block_mean_dev<NV>(v, red[0]);
+    const float f = a.mult / sqrtf(m.dev * invW + a.eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const float4 w = __ldg(w1 + 128 * i);
+        x[i].x = fmaf((v[i].x - m.mean) * f, w.x, x[i].x); x[i].y = fmaf((v[i].y - m.mean) * f, w.y, x[i].y);
+        x[i].z = fmaf((v[i].z - m.mean) * f, w.z, x[i].z); x[i].w = fmaf((v[i].w - m.mean) * f, w.w, x[i].w);
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        xr[128 * i] = x[i];
+        yr[128 * i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    }
+    if (a.next_mode == 0) return;
+    MeanDev m2{0.0f, 0.0f};
+    float g = 1.0f;
+    if (a.next_mode == 1) {
+        m2 = block_mean_dev<NV>(x, red[1]);
+        g = 1.0f / sqrtf(m2.dev * invW + a.eps);
+    }
+    const float4* __restrict__ w2 = (const float4*)a.w_next + threadIdx.x;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        float4 o = x[i];
+        if (a.next_mode == 1) {
+            const float4 w = __ldg(w2 + 128 * i);
+            o.x = (o.x - m2.mean) * g * w.x; o.y = (o.y - m2.mean) * g * w.y; o.z = (o.z - m2.mean) * g * w.z; o.w = (o.w - m2.mean) * g * w.w;
+        }
+        const size_t at = (size_t)t * a.W + (threadIdx.x + 128 * i) * 4;
+        if (a.out_dt == SP_DT_F32) {
+            *(float4*)((float*)a.out + at) = o;
+        } else {
+            __nv_bfloat162 p0 = __floats2bfloat162_rn(o.x, o.y), p1 = __floats2bfloat162_rn(o.z, o.w);
+            uint2 pk;
+            pk.x = *(uint32_t*)&p0; pk.y = *(uint32_t*)&p1;
+            *(uint2*)((__nv_bfloat16*)a.out + at) = pk;
+        }
+    }
+}
+
+// any width: the mean first, then the squared deviations
 __global__ void __launch_bounds__(256) stream_layernorm_add_kernel(NormAddArgs a) {
     __shared__ float red[32];
     sp_allow_dependents();
@@ -170,74 +252,6 @@ __global__ void __launch_bounds__(256) stream_layernorm_add_kernel(NormAddArgs a
     float* xr = a.x + (size_t)t * a.W;
     float* yr = a.y + (size_t)t * a.W;
     const float invW = 1.0f / (float)a.W;
-    if (NV > 0) {
-        constexpr int N = NV > 0 ? NV : 1;
-        float4 v[N], x[N];
-        float sum = 0.0f;
-#pragma unroll
-        for (int i = 0; i < N; ++i) {
-            const int c = (i * 256 + threadIdx.x) * 4;
-            v[i] = x[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-            if (c < a.W) {
-                v[i] = *(const float4*)(yr + c);
-                x[i] = *(const float4*)(xr + c);
-                *(float4*)(yr + c) = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-            }
-            sum += (v[i].x + v[i].y) + (v[i].z + v[i].w);
-        }
-        const float mean = sp_block_sum(sum, red) * invW;
-        float ss = 0.0f;
-#pragma unroll
-        for (int i = 0; i < N; ++i) {
-            if ((i * 256 + threadIdx.x) * 4 >= a.W) continue;
-            v[i].x -= mean; v[i].y -= mean; v[i].z -= mean; v[i].w -= mean;
-            ss = fmaf(v[i].x, v[i].x, ss); ss = fmaf(v[i].y, v[i].y, ss); ss = fmaf(v[i].z, v[i].z, ss); ss = fmaf(v[i].w, v[i].w, ss);
-        }
-        const float f = a.mult / sqrtf(sp_block_sum(ss, red) * invW + a.eps);
-        sum = 0.0f;
-#pragma unroll
-        for (int i = 0; i < N; ++i) {
-            const int c = (i * 256 + threadIdx.x) * 4;
-            if (c >= a.W) continue;
-            const float4 w = *(const float4*)(a.w_post + c);
-            x[i].x = fmaf(v[i].x * f, w.x, x[i].x); x[i].y = fmaf(v[i].y * f, w.y, x[i].y);
-            x[i].z = fmaf(v[i].z * f, w.z, x[i].z); x[i].w = fmaf(v[i].w * f, w.w, x[i].w);
-            *(float4*)(xr + c) = x[i];
-            sum += (x[i].x + x[i].y) + (x[i].z + x[i].w);
-        }
-        if (a.next_mode == 0) return;
-        float m2 = 0.0f, g = 1.0f;
-        if (a.next_mode == 1) {
-            m2 = sp_block_sum(sum, red) * invW;
-            ss = 0.0f;
-#pragma unroll
-            for (int i = 0; i < N; ++i) {
-                if ((i * 256 + threadIdx.x) * 4 >= a.W) continue;
-                const float p = x[i].x - m2, q = x[i].y - m2, r = x[i].z - m2, u = x[i].w - m2;
-                ss = fmaf(p, p, ss); ss = fmaf(q, q, ss); ss = fmaf(r, r, ss); ss = fmaf(u, u, ss);
-            }
-            g = 1.0f / sqrtf(sp_block_sum(ss, red) * invW + a.eps);
-        }
-#pragma unroll
-        for (int i = 0; i < N; ++i) {
-            const int c = (i * 256 + threadIdx.x) * 4;
-            if (c >= a.W) continue;
-            float4 o = x[i];
-            if (a.next_mode == 1) {
-                const float4 w = *(const float4*)(a.w_next + c);
-                o.x = (o.x - m2) * (g * w.x); o.y = (o.y - m2) * (g * w.y); o.z = (o.z - m2) * (g * w.z); o.w = (o.w - m2) * (g * w.w);
-            }
-            if (a.out_dt == SP_DT_F32) {
-                *(float4*)((float*)a.out + (size_t)t * a.W + c) = o;
-            } else {
-                __nv_bfloat162 p0 = __floats2bfloat162_rn(o.x, o.y), p1 = __floats2bfloat162_rn(o.z, o.w);
-                uint2 pk;
-                pk.x = *(uint32_t*)&p0; pk.y = *(uint32_t*)&p1;
-                *(uint2*)((__nv_bfloat16*)a.out + (size_t)t * a.W + c) = pk;
-            }
-        }
-        return;
-    }
     float sum = 0.0f, ss = 0.0f;
     for (int c = threadIdx.x; c < a.W; c += blockDim.x) sum += yr[c];
     const float mean = sp_block_sum(sum, red) * invW;
@@ -259,7 +273,7 @@ __global__ void __launch_bounds__(256) stream_layernorm_add_kernel(NormAddArgs a
         g = 1.0f / sqrtf(sp_block_sum(ss, red) * invW + a.eps);
     }
     for (int c = threadIdx.x; c < a.W; c += blockDim.x)
-        sp_st_dt(a.out, a.out_dt, (size_t)t * a.W + c, a.next_mode == 1 ? (xr[c] - m2) * (g * a.w_next[c]) : xr[c]);
+        sp_st_dt(a.out, a.out_dt, (size_t)t * a.W + c, a.next_mode == 1 ? (xr[c] - m2) * g * a.w_next[c] : xr[c]);
 }
 
 SP_API int sp_stream_norm_add(float* x, float* y, const float* w_post, const float* w_next, void* out, int out_dt,
@@ -270,12 +284,10 @@ SP_API int sp_stream_norm_add(float* x, float* y, const float* w_post, const flo
     NormAddArgs a{x, y, w_post, w_next, out, out_dt, next_mode, T, W, mult, eps};
     const bool vec = (W % 4) == 0 && ((((uintptr_t)x | (uintptr_t)y | (uintptr_t)w_post | (uintptr_t)w_next | (uintptr_t)out) & 15) == 0);
     if (centered) {
-        const dim3 g(T), b(256);
-        if (vec && W <= 1024) SP_CHECK_CALL("stream_norm_add", sp_launch_dependent(stream_layernorm_add_kernel<1>, g, b, 0, stream, a));
-        else if (vec && W <= 2048) SP_CHECK_CALL("stream_norm_add", sp_launch_dependent(stream_layernorm_add_kernel<2>, g, b, 0, stream, a));
-        else if (vec && W <= 4096) SP_CHECK_CALL("stream_norm_add", sp_launch_dependent(stream_layernorm_add_kernel<4>, g, b, 0, stream, a));
-        else if (vec && W <= 8192) SP_CHECK_CALL("stream_norm_add", sp_launch_dependent(stream_layernorm_add_kernel<8>, g, b, 0, stream, a));
-        else SP_CHECK_CALL("stream_norm_add", sp_launch_dependent(stream_layernorm_add_kernel<0>, g, b, 0, stream, a));
+#define SP_LN_ROWS(NV) if (vec && W == 512 * NV) { SP_CHECK_CALL("stream_norm_add", sp_launch_dependent(stream_layernorm_add_rows_kernel<NV>, dim3(T), dim3(128), 0, stream, a)); return 0; }
+        SP_LN_ROWS(1) SP_LN_ROWS(2) SP_LN_ROWS(3) SP_LN_ROWS(4) SP_LN_ROWS(5) SP_LN_ROWS(6) SP_LN_ROWS(8) SP_LN_ROWS(10)
+#undef SP_LN_ROWS
+        SP_CHECK_CALL("stream_norm_add", sp_launch_dependent(stream_layernorm_add_kernel, dim3(T), dim3(256), 0, stream, a));
         return 0;
     }
     if (vec) SP_CHECK_CALL("stream_norm_add", sp_launch_dependent(stream_norm_add_kernel<4>, dim3(T), dim3(256), 0, stream, a));
@@ -527,6 +539,82 @@ __global__ void __launch_bounds__(NR_WARPS * 32) qkv_norm_rot_store_kernel(NormR
     }
 }
 
+// The same where a head is one float4 per lane (d at most 128, pairs half apart, multiples of four): a warp asks for four
+// heads' values at once, ahead of the angles, and a pair's other half comes from another lane.
+template <typename TO, typename TC>
+__global__ void __launch_bounds__(NR_WARPS * 32) qkv_norm_rot_rows_kernel(NormRotArgs a) {
+    extern __shared__ __align__(16) float cs[];          // [2][rd/2]
+    constexpr int HB = 4;
+    sp_allow_dependents();
+    sp_wait_for_predecessor();
+    const int t = blockIdx.x;
+    if (t >= a.T) return;
+    const int half = a.rd >> 1, d = a.d, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int i = lane * 4, heads = a.nh + a.nkv;
+    const bool in = i < d;
+    const float* src = a.proj + (size_t)t * a.ld;
+    const float4 z = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    float4 v[HB];
+    auto load = [&](int h0) {
+#pragma unroll
+        for (int u = 0; u < HB; ++u) {
+            const int h = h0 + u * NR_WARPS;
+            v[u] = (in && h < heads) ? *(const float4*)(src + h * d + i) : z;
+        }
+    };
+    load(warp);
+    const int pos = a.pl.positions[t];
+    const float4 wq = a.qw && in ? ld4_dt(a.qw, a.w_dt, i) : z, wk = a.kw && in ? ld4_dt(a.kw, a.w_dt, i) : z;
+    int page = 0;
+    const bool place_ok = a.nkv > 0 && page_of(a.pl, t, pos, page);
+    const int off = pos % a.pl.page_size;
+    pair_angles(cs, a.freq, half, pos, a.rot_mult);
+    __syncthreads();
+    // the lane's four dims: their cos and sin, and the lane that holds their partners
+    const bool turns = i < a.rd, lo = i < half;
+    float4 c4 = make_float4(1.0f, 1.0f, 1.0f, 1.0f), s4 = z;
+    if (turns) {
+        c4 = *(const float4*)(cs + (lo ? i : i - half));
+        s4 = *(const float4*)(cs + half + (lo ? i : i - half));
+        if (lo) { s4.x = -s4.x; s4.y = -s4.y; s4.z = -s4.z; s4.w = -s4.w; }
+    }
+    const int peer = turns ? (lo ? lane + half / 4 : lane - half / 4) : lane;
+    TO* q_out = (TO*)a.q_out + (size_t)t * a.nh * d;
+    for (int h0 = warp; h0 < heads; h0 += HB * NR_WARPS) {
+        if (h0 != warp) load(h0);
+#pragma unroll
+        for (int u = 0; u < HB; ++u) {
+            const int h = h0 + u * NR_WARPS;
+            if (h >= heads) break;
+            const bool is_q = h < a.nh;
+            if (a.bias && in) { const float4 b = ld4_dt(a.bias, a.b_dt, (size_t)h * d + i); v[u].x += b.x; v[u].y += b.y; v[u].z += b.z; v[u].w += b.w; }
+            if (is_q ? a.qw != nullptr : a.kw != nullptr) {
+                const float ss = sp_warp_sum((v[u].x * v[u].x + v[u].y * v[u].y) + (v[u].z * v[u].z + v[u].w * v[u].w));
+                const float inv = 1.0f / sqrtf(ss / (float)d + a.eps);
+                const float4 w = is_q ? wq : wk;
+                v[u].x = v[u].x * inv * w.x; v[u].y = v[u].y * inv * w.y; v[u].z = v[u].z * inv * w.z; v[u].w = v[u].w * inv * w.w;
+            }
+            const float4 o = make_float4(__shfl_sync(0xffffffffu, v[u].x, peer), __shfl_sync(0xffffffffu, v[u].y, peer),
+                                         __shfl_sync(0xffffffffu, v[u].z, peer), __shfl_sync(0xffffffffu, v[u].w, peer));
+            if (!in) continue;
+            if (turns) {
+                v[u].x = v[u].x * c4.x + o.x * s4.x; v[u].y = v[u].y * c4.y + o.y * s4.y;
+                v[u].z = v[u].z * c4.z + o.z * s4.z; v[u].w = v[u].w * c4.w + o.w * s4.w;
+            }
+            if (is_q) st4(q_out, (size_t)h * d + i, v[u]);
+            else if (place_ok) st4((TC*)a.kpool, (((size_t)page * a.nkv + (h - a.nh)) * a.pl.page_size + off) * d + i, v[u]);
+        }
+    }
+    if (!place_ok) return;
+    const int v0 = heads * d;
+    for (int e = threadIdx.x * 4; e < a.nkv * a.vd; e += blockDim.x * 4) {
+        const int g = e / a.vd, r = e - g * a.vd;
+        float4 x = *(const float4*)(src + v0 + e);
+        if (a.bias) { const float4 b = ld4_dt(a.bias, a.b_dt, (size_t)v0 + e); x.x += b.x; x.y += b.y; x.z += b.z; x.w += b.w; }
+        st4((TC*)a.vpool, (((size_t)page * a.nkv + g) * a.pl.page_size + off) * a.vd + r, x);
+    }
+}
+
 SP_API int sp_qkv_norm_rot_store(const float* proj, int ld, const void* bias, int b_dt, const void* qw, const void* kw, int w_dt,
                                  void* q_out, int q_dt, void* kpool, void* vpool, int c_dt, const float* freq,
                                  const int* token_seq, const int* positions, const int* seq_row, const int* page_table,
@@ -543,7 +631,8 @@ SP_API int sp_qkv_norm_rot_store(const float* proj, int ld, const void* bias, in
                      ((((uintptr_t)proj | (uintptr_t)bias | (uintptr_t)q_out | (uintptr_t)kpool | (uintptr_t)vpool) & 15) == 0);
     const size_t smem = (size_t)(((rd + 3) & ~3) + NR_WARPS * ((d + 3) & ~3)) * sizeof(float);
     if (smem > 48 * 1024) SP_FAIL("qkv_norm_rot_store: heads of %d are beyond this kernel's range", d);
-#define NR_LAUNCH(TO, TC) do { if (vec) SP_CHECK_CALL("qkv_norm_rot_store", sp_launch_dependent(qkv_norm_rot_store_kernel<TO, TC, true>, dim3(T), dim3(NR_WARPS * 32), smem, stream, a)); \
+#define NR_LAUNCH(TO, TC) do { if (vec && d <= 128) SP_CHECK_CALL("qkv_norm_rot_store", sp_launch_dependent(qkv_norm_rot_rows_kernel<TO, TC>, dim3(T), dim3(NR_WARPS * 32), (size_t)(rd > 0 ? rd : 4) * sizeof(float), stream, a)); \
+    else if (vec) SP_CHECK_CALL("qkv_norm_rot_store", sp_launch_dependent(qkv_norm_rot_store_kernel<TO, TC, true>, dim3(T), dim3(NR_WARPS * 32), smem, stream, a)); \
     else SP_CHECK_CALL("qkv_norm_rot_store", sp_launch_dependent(qkv_norm_rot_store_kernel<TO, TC, false>, dim3(T), dim3(NR_WARPS * 32), smem, stream, a)); } while (0)
     if (q_dt == SP_DT_F32 && c_dt == SP_DT_F32) NR_LAUNCH(float, float);
     else if (q_dt == SP_DT_BF16 && c_dt == SP_DT_BF16) NR_LAUNCH(__nv_bfloat16, __nv_bfloat16);
