@@ -61,19 +61,21 @@ __device__ __forceinline__ bool ml_chunk_of(const MlArgs& a, int x, int ct, int&
 }
 
 // ============================================================== the gates of a prompt step
-// One block per (sequence, head); a warp takes a chunk, a lane CT / 32 neighbouring tokens. Running sums and maxima in
-// 64-bit; what the products read are exponentials of differences, each rounded once.
-constexpr int MG_WARPS = 16;
+// One block per (sequence, head); a warp takes 64 tokens, a lane two neighbouring ones, CT / 64 warps share a chunk; one warp
+// carries the maximum from chunk to chunk (max-plus scan). Running sums and maxima in 64-bit; what the products read are
+// exponentials of differences, each rounded once.
+constexpr int MG_WARPS = 32;
 template <int CT>
 __global__ void __launch_bounds__(MG_WARPS * 32) mlstm_gates_kernel(MlArgs a) {
-    constexpr int PL = CT / 32;
-    __shared__ double sumF[MG_WARPS], topA[MG_WARPS], m0s[MG_WARPS], m_run;
+    static_assert(CT == 64 || CT == 128, "one or two warps of 64 tokens share a chunk");
+    constexpr int WPC = CT / 64, CHUNKS = MG_WARPS / WPC;       // warps of a chunk, chunks of a pass
+    __shared__ double sumF[MG_WARPS], topA[MG_WARPS], m0s[CHUNKS], m_run;
     sp_wait_for_predecessor();
     sp_allow_dependents();               // in this order: whoever starts from here on may read the projections at once
     const int s = blockIdx.x, h = blockIdx.y;
     const int slot = a.seq_slot[s];
     if (slot < 0 || slot >= a.n_slots) return;
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, part = warp % WPC;
     const int first = a.seq_start[s], cnt = a.seq_start[s + 1] - first;
     int chunk0 = 0;
     for (int b = 0; b < s; ++b) chunk0 += (a.seq_start[b + 1] - a.seq_start[b] + CT - 1) / CT;
@@ -81,78 +83,89 @@ __global__ void __launch_bounds__(MG_WARPS * 32) mlstm_gates_kernel(MlArgs a) {
     float* m_state = a.nm + ((size_t)slot * a.H + h) * (a.d + 1) + a.d;
     if (threadIdx.x == 0) m_run = *m_state;
     const float ib = sp_ld_dt(a.ib, a.w_dt, h), fb = sp_ld_dt(a.fb, a.w_dt, h);
-    const int gi = 2 * a.H * a.d + 2 * a.H * a.vd + h;
-    for (int c0 = 0; c0 < nc; c0 += MG_WARPS) {
-        const int c = c0 + warp;
-        double F[PL], A[PL], top[PL];
-        if (c < nc) {
-            double run = 0.0;
-            float iv[PL], fv[PL];
+    const float* gates = a.proj + 2 * a.H * a.d + 2 * a.H * a.vd + h;
+    for (int c0 = 0; c0 < nc; c0 += CHUNKS) {
+        const int t = c0 * CT + warp * 64 + lane * 2;            // the lane's first token
+        float iv[2], fv[2];
 #pragma unroll
-            for (int u = 0; u < PL; ++u) {
-                const int t = c * CT + lane * PL + u;
-                const float* row = a.proj + (size_t)(first + min(t, cnt - 1)) * a.ld + gi;
-                iv[u] = t < cnt ? ml_input_gate(row[0] + ib, a.cap) : -INFINITY;
-                fv[u] = t < cnt ? ml_log_forget(row[a.H] + fb, a.cap) : 0.0f;
+        for (int u = 0; u < 2; ++u) {
+            const float* row = gates + (size_t)(first + min(t + u, cnt - 1)) * a.ld;
+            iv[u] = row[0];
+            fv[u] = row[a.H];
+        }
+        double F[2], A[2], top[2];
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+            iv[u] = t + u < cnt ? ml_input_gate(iv[u] + ib, a.cap) : -INFINITY;
+            fv[u] = t + u < cnt ? ml_log_forget(fv[u] + fb, a.cap) : 0.0f;
+        }
+        double inc = (double)fv[0] + (double)fv[1];              // inclusive over the lanes
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const double up = __shfl_up_sync(0xffffffffu, inc, o);
+            if (lane >= o) inc += up;
+        }
+        F[1] = inc;
+        F[0] = inc - (double)fv[1];
+        A[0] = (double)iv[0] - F[0];
+        A[1] = (double)iv[1] - F[1];
+        double mx = fmax(A[0], A[1]);
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const double up = __shfl_up_sync(0xffffffffu, mx, o);
+            if (lane >= o) mx = fmax(mx, up);
+        }
+        double before = __shfl_up_sync(0xffffffffu, mx, 1);
+        if (lane == 0) before = -INFINITY;
+        top[0] = fmax(before, A[0]);
+        top[1] = mx;
+        if (lane == 31) { sumF[warp] = inc; topA[warp] = mx; }
+        __syncthreads();
+        if (warp == 0) {
+            // chunk by chunk m ← max(m + S, T), S the chunk's sum of f, T = S + its largest a
+            double S = 0.0, T = -INFINITY;
+            if (lane < CHUNKS && c0 + lane < nc) {
+#pragma unroll
+                for (int w = 0; w < WPC; ++w) {
+                    T = fmax(T, topA[lane * WPC + w] - S);
+                    S += sumF[lane * WPC + w];
+                }
+                T += S;
             }
-#pragma unroll
-            for (int u = 0; u < PL; ++u) { run += (double)fv[u]; F[u] = run; }
-            double base = run;                           // inclusive over lanes, then exclusive
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
-                const double up = __shfl_up_sync(0xffffffffu, base, o);
-                if (lane >= o) base += up;
+                const double s1 = __shfl_up_sync(0xffffffffu, S, o), t1 = __shfl_up_sync(0xffffffffu, T, o);
+                if (lane >= o) {
+                    T = fmax(t1 + S, T);
+                    S += s1;
+                }
             }
-            const double total = __shfl_sync(0xffffffffu, base, 31);
-            double ex = __shfl_up_sync(0xffffffffu, base, 1);
-            if (lane == 0) ex = 0.0;
-            double mx = -INFINITY;
-#pragma unroll
-            for (int u = 0; u < PL; ++u) {
-                F[u] += ex;
-                A[u] = (double)iv[u] - F[u];
-                mx = fmax(mx, A[u]);
-                top[u] = mx;
-            }
-            double inc = mx;
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const double up = __shfl_up_sync(0xffffffffu, inc, o);
-                if (lane >= o) inc = fmax(inc, up);
-            }
-            double em = __shfl_up_sync(0xffffffffu, inc, 1);
-            if (lane == 0) em = -INFINITY;
-#pragma unroll
-            for (int u = 0; u < PL; ++u) top[u] = fmax(top[u], em);
-            const double all = __shfl_sync(0xffffffffu, inc, 31);
-            if (lane == 0) { sumF[warp] = total; topA[warp] = all; }
+            const double m_in = m_run, m_end = fmax(m_in + S, T);
+            const double m_before = __shfl_up_sync(0xffffffffu, m_end, 1);
+            if (lane < CHUNKS) m0s[lane] = lane == 0 ? m_in : m_before;
+            if (lane == 31) m_run = m_end;                       // lanes beyond the last chunk add nothing
         }
         __syncthreads();
-        if (threadIdx.x == 0) {
-            double m = m_run;
-            for (int w = 0; w < MG_WARPS && c0 + w < nc; ++w) {
-                m0s[w] = m;
-                m = sumF[w] + fmax(m, topA[w]);
-            }
-            m_run = m;
-        }
-        __syncthreads();
+        const int c = c0 + warp / WPC;
         if (c < nc) {
-            const double m0 = m0s[warp], ML = fmax(m0, topA[warp]);
+            // of the chunk: the sum and the largest a in front of this warp's tokens, the largest of all
+            const int w0 = warp - part;
+            const double S = part ? sumF[w0] : 0.0, ahead = part ? topA[w0] : -INFINITY;
+            const double all = WPC == 2 ? fmax(topA[w0], topA[w0 + WPC - 1] - sumF[w0]) : topA[w0];
+            const double m0 = m0s[warp / WPC], ML = fmax(m0, all);
 #pragma unroll
-            for (int u = 0; u < PL; ++u) {
-                const int t = c * CT + lane * PL + u;
-                if (t >= cnt) break;
-                const size_t at = (size_t)h * a.T + first + t;
-                const double M = fmax(m0, top[u]);
-                const float ah = (float)A[u], mh = (float)M;
-                a.a2[at] = make_float2(ah, (float)(A[u] - (double)ah));
+            for (int u = 0; u < 2; ++u) {
+                if (t + u >= cnt) break;
+                const size_t at = (size_t)h * a.T + first + t + u;
+                const double aj = A[u] - S, M = fmax(m0, fmax(ahead, top[u] - S));
+                const float ah = (float)aj, mh = (float)M;
+                a.a2[at] = make_float2(ah, (float)(aj - (double)ah));
                 a.M2[at] = make_float2(mh, (float)(M - (double)mh));
                 a.r[at] = expf((float)(m0 - M));
-                a.we[at] = expf((float)(A[u] - ML));
-                a.em[at] = expf((float)(-(F[u] + M)));
+                a.we[at] = expf((float)(aj - ML));
+                a.em[at] = expf((float)(-(F[u] + S + M)));
             }
-            if (lane == 0) a.ce[(size_t)h * a.n_chunks + chunk0 + c] = expf((float)(m0 - ML));
+            if (lane == 0 && part == 0) a.ce[(size_t)h * a.n_chunks + chunk0 + c] = expf((float)(m0 - ML));
         }
         __syncthreads();
     }
@@ -335,6 +348,7 @@ __global__ void __launch_bounds__(128) mlstm_finish_kernel(MlArgs a) {
 // 128-byte swizzle (rows of 64 numbers, 16-byte pieces exchanged by the row's low bits).
 constexpr int TK = 128;
 constexpr int BOX = TK * 128;                 // bytes of 128 rows of 64 numbers
+constexpr int OT_LD = 260;                    // floats of a row of results in shared memory (rows 16 bytes apart in the banks)
 
 __device__ __forceinline__ uint32_t sw_at(int row, int piece) { return (uint32_t)(row * 128 + ((piece ^ (row & 7)) << 4)); }
 __device__ __forceinline__ uint4 pack8(const float (&f)[8]) {
@@ -356,13 +370,13 @@ __device__ __forceinline__ void load8(const float* p, bool in, float (&f)[8]) {
 __device__ __forceinline__ void proxy_fence() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
 
 // A chunk's values, columns c0 .. c0 + nb - 1 of head h, as boxes of 64 columns with one row per token (the product's K):
-// sixteen pieces of eight numbers per thread, pieces U0 .. U0 + N - 1 of them. All of a batch's loads come before its stores,
+// 4,096 pieces of eight numbers over the THREADS of a block, a thread's pieces u0 .. u0 + N - 1. All of a batch's loads come before its stores,
 // which the compiler would not let them pass.
-template <int N>
+template <int N, int THREADS = 256>
 __device__ __forceinline__ void load_values(const MlArgs& a, float4 (&r)[2 * N], int u0, int h, int t0, int n, int c0, int nb) {
 #pragma unroll
     for (int u = 0; u < N; ++u) {
-        const int x = threadIdx.x + 256 * (u0 + u), j = x >> 5, col = c0 + 8 * (x & 31);
+        const int x = threadIdx.x + THREADS * (u0 + u), j = x >> 5, col = c0 + 8 * (x & 31);
         const float4* p = (const float4*)(a.proj + (size_t)(t0 + j) * a.ld + 2 * a.H * a.d + (size_t)h * a.vd + col);
         const bool in = j < n && col < a.vd;
         r[2 * u] = in ? p[0] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
@@ -372,11 +386,11 @@ __device__ __forceinline__ void load_values(const MlArgs& a, float4 (&r)[2 * N],
 __device__ __forceinline__ uint4 pack8(const float4& a, const float4& b) {
     return make_uint4(pack_bf16(a.x, a.y), pack_bf16(a.z, a.w), pack_bf16(b.x, b.y), pack_bf16(b.z, b.w));
 }
-template <int N>
+template <int N, int THREADS = 256>
 __device__ __forceinline__ void store_values(uint8_t* dst, const float4 (&r)[2 * N], int u0, int nb) {
 #pragma unroll
     for (int u = 0; u < N; ++u) {
-        const int x = threadIdx.x + 256 * (u0 + u), j = x >> 5, c = x & 31;
+        const int x = threadIdx.x + THREADS * (u0 + u), j = x >> 5, c = x & 31;
         if (8 * c < nb) *(uint4*)(dst + (c >> 3) * BOX + sw_at(j, c & 7)) = pack8(r[2 * u], r[2 * u + 1]);
     }
 }
@@ -471,17 +485,24 @@ __global__ void __launch_bounds__(256) mlstm_sum_tc_kernel(MlArgs a) {
         }
         const bool ok = mbar_wait_flag(smem_u32(&bar), 0, a.status, 151, &gave_up);
         tc_fence_after();
-        const int e = e0 + (warp & 3) * 32 + lane;
+        // through shared memory (the products have read theirs), so that the sums leave as whole lines
+        float* rows = (float*)sm;
         for (int c = (warp >> 2) * 32; c < nb; c += 64) {
             uint32_t r[32];
             tc_ld_32x32(tmem + ((uint32_t)((warp & 3) * 32) << 16) + c, r);
             tc_ld_wait();
-            if (!ok || e >= a.d) continue;
 #pragma unroll
             for (int i = 0; i < 32; i += 4)
-                if (c0 + c + i < a.vd)
-                    *(float4*)(out + (size_t)e * a.vc + c0 + c + i) =
-                        make_float4(__uint_as_float(r[i]), __uint_as_float(r[i + 1]), __uint_as_float(r[i + 2]), __uint_as_float(r[i + 3]));
+                *(float4*)(rows + ((warp & 3) * 32 + lane) * OT_LD + c + i) =
+                    make_float4(__uint_as_float(r[i]), __uint_as_float(r[i + 1]), __uint_as_float(r[i + 2]), __uint_as_float(r[i + 3]));
+        }
+        __syncthreads();
+        if (ok) {
+#pragma unroll 4
+            for (int x = threadIdx.x; x < TK * 64; x += 256) {
+                const int e = x >> 6, c = (x & 63) * 4;
+                if (e0 + e < a.d && c0 + c < a.vd && c < nb) *(float4*)(out + (size_t)(e0 + e) * a.vc + c0 + c) = *(const float4*)(rows + e * OT_LD + c);
+            }
         }
     }
     tc_fence_before();
@@ -495,19 +516,19 @@ __global__ void __launch_bounds__(256) mlstm_sum_tc_kernel(MlArgs a) {
 // Outputs of a chunk, up to 256 value columns. Blocks of 64 key dims pass through two shared-memory stages (q, k, the start
 // state's high and low part): A = q kᵀ and O = q · S₀ gather in tensor memory; the rows of O take e^{m₀ − M_i}, A turns into
 // the pair weights (high and low part, as an operand in tensor memory), the values follow into the stage that is free, and O
-// gathers the chunk's own share. A thread owns a row (token) and every other group of 32 columns; warps w and w + 4 share
-// rows. With one column block the denominator, the unit rms, weight and gate follow here, else the raw outputs leave.
+// gathers the chunk's own share. A thread owns a row (token) and every fourth group of 32 columns; warps whose
+// numbers are equal modulo 4 share rows. With one column block the denominator, the unit rms, weight and gate follow here, else the raw outputs leave.
 // grid (chunks, H, column blocks of 256)
+constexpr int OT_THREADS = 512;
 constexpr int OT_STAGE = 2 * BOX + 2 * 32768;
-constexpr int OT_LD = 260;                    // floats of a row of outputs in shared memory (rows 16 bytes apart in the banks)
 static_assert(TK * OT_LD * 4 <= 2 * OT_STAGE, "the outputs reuse the operands' stages");
-__global__ void __launch_bounds__(256) mlstm_out_tc_kernel(MlArgs a) {
+__global__ void __launch_bounds__(OT_THREADS) mlstm_out_tc_kernel(MlArgs a) {
     extern __shared__ uint8_t smem_raw[];
     __shared__ __align__(8) uint64_t bar_free[2], bar_a, bar_o;
     __shared__ uint32_t tmem_slot;
     __shared__ int gave_up;
     __shared__ float2 aj[TK];
-    __shared__ float nvec[2][64], qn_s[2][TK], ss_s[2][TK];
+    __shared__ float nvec[2][64], qn_s[4][TK], ss_s[4][TK];
     uint8_t* sm = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (threadIdx.x == 0) {
@@ -543,14 +564,14 @@ __global__ void __launch_bounds__(256) mlstm_out_tc_kernel(MlArgs a) {
         const int nE = (d + 63) / 64;
         bool ok = true;
         float dot = 0.0f;
-        // 512 bytes of operands per thread: q, k and the start state of a block of key dims, in the end the values; the next
+        // 256 bytes of operands per thread: q, k and the start state of a block of key dims, in the end the values; the next
         // ones are asked for before the products of the ones at hand begin
-        float4 buf[32];
+        float4 buf[16];
         const float4 z4 = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         auto load_qk = [&](int eb) {
 #pragma unroll
-            for (int u = 0; u < 4; ++u) {
-                const int x = threadIdx.x + 256 * u, j = x >> 3, e = eb * 64 + 8 * (x & 7);
+            for (int u = 0; u < 2; ++u) {
+                const int x = threadIdx.x + OT_THREADS * u, j = x >> 3, e = eb * 64 + 8 * (x & 7);
                 const bool in = j < n && e < d;
                 const float4 *pq = (const float4*)(a.proj + (size_t)(t0 + j) * a.ld + (size_t)h * d + e), *pk = (const float4*)((const float*)pq + (size_t)a.H * d);
                 buf[4 * u] = in ? pq[0] : z4;
@@ -561,28 +582,28 @@ __global__ void __launch_bounds__(256) mlstm_out_tc_kernel(MlArgs a) {
         };
         auto load_state = [&](int eb) {
 #pragma unroll
-            for (int u = 0; u < 8; ++u) {
-                const int x = threadIdx.x + 256 * u, e = eb * 64 + (x >> 5), col = c0 + 8 * (x & 31);
+            for (int u = 0; u < 4; ++u) {
+                const int x = threadIdx.x + OT_THREADS * u, e = eb * 64 + (x >> 5), col = c0 + 8 * (x & 31);
                 const bool in = e < d && col < a.vd;
                 const float4* p = (const float4*)(cs + (size_t)e * a.vc + col);
-                buf[16 + 2 * u] = in ? p[0] : z4;
-                buf[17 + 2 * u] = in ? p[1] : z4;
+                buf[8 + 2 * u] = in ? p[0] : z4;
+                buf[9 + 2 * u] = in ? p[1] : z4;
             }
         };
         auto store_qk = [&](uint8_t* q, uint8_t* k) {
 #pragma unroll
-            for (int u = 0; u < 4; ++u) {
-                const int x = threadIdx.x + 256 * u;
+            for (int u = 0; u < 2; ++u) {
+                const int x = threadIdx.x + OT_THREADS * u;
                 *(uint4*)(q + sw_at(x >> 3, x & 7)) = pack8(buf[4 * u], buf[4 * u + 1]);
                 *(uint4*)(k + sw_at(x >> 3, x & 7)) = pack8(buf[4 * u + 2], buf[4 * u + 3]);
             }
         };
         auto store_state = [&](uint8_t* sh, uint8_t* sl) {
 #pragma unroll
-            for (int u = 0; u < 8; ++u) {
-                const int x = threadIdx.x + 256 * u, r = x >> 5, c = x & 31;
+            for (int u = 0; u < 4; ++u) {
+                const int x = threadIdx.x + OT_THREADS * u, r = x >> 5, c = x & 31;
                 if (8 * c >= nb) continue;
-                const uint4 w0 = *(const uint4*)&buf[16 + 2 * u], w1 = *(const uint4*)&buf[17 + 2 * u];
+                const uint4 w0 = *(const uint4*)&buf[8 + 2 * u], w1 = *(const uint4*)&buf[9 + 2 * u];
                 const uint32_t to = (uint32_t)((c >> 3) * 8192) + sw_at(r, c & 7);
                 *(uint4*)(sh + to) = make_uint4(__byte_perm(w0.x, w0.y, 0x5410), __byte_perm(w0.z, w0.w, 0x5410), __byte_perm(w1.x, w1.y, 0x5410), __byte_perm(w1.z, w1.w, 0x5410));
                 *(uint4*)(sl + to) = make_uint4(__byte_perm(w0.x, w0.y, 0x7632), __byte_perm(w0.z, w0.w, 0x7632), __byte_perm(w1.x, w1.y, 0x7632), __byte_perm(w1.z, w1.w, 0x7632));
@@ -606,7 +627,7 @@ __global__ void __launch_bounds__(256) mlstm_out_tc_kernel(MlArgs a) {
                 load_qk(eb + 1);
                 load_state(eb + 1);
             } else {
-                load_values<16>(a, buf, 0, h, t0, n, c0, nb);
+                load_values<8, OT_THREADS>(a, buf, 0, h, t0, n, c0, nb);
             }
             proxy_fence();
             __syncthreads();
@@ -621,12 +642,12 @@ __global__ void __launch_bounds__(256) mlstm_out_tc_kernel(MlArgs a) {
                 tc_commit(smem_u32(&bar_free[eb & 1]));
                 if (eb == nE - 1) tc_commit(smem_u32(&bar_a));
             }
-            // q · n of the row, half of the block's dims each
+            // q · n of the row, a quarter of the block's dims each
 #pragma unroll
-            for (int c = 0; c < 4; ++c) {
-                const uint4 w = *(const uint4*)(q + sw_at(row, hh * 4 + c));
+            for (int c = 0; c < 2; ++c) {
+                const uint4 w = *(const uint4*)(q + sw_at(row, hh * 2 + c));
                 const uint32_t v[4] = {w.x, w.y, w.z, w.w};
-                const float* nr = &nvec[eb & 1][hh * 32 + c * 8];
+                const float* nr = &nvec[eb & 1][hh * 16 + c * 8];
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
                     dot = fmaf(__uint_as_float(v[i] << 16), nr[2 * i], dot);
@@ -637,35 +658,34 @@ __global__ void __launch_bounds__(256) mlstm_out_tc_kernel(MlArgs a) {
         // the values go where block nE - 2 was
         uint8_t* vs = sm + (nE & 1) * OT_STAGE;
         if (nE >= 2) ok = mbar_wait_flag(smem_u32(&bar_free[nE & 1]), (uint32_t)((nE - 2) >> 1) & 1u, a.status, 152, &gave_up) && ok;
-        store_values<16>(vs, buf, 0, nb);
+        store_values<8, OT_THREADS>(vs, buf, 0, nb);
         proxy_fence();
         ok = mbar_wait_flag(smem_u32(&bar_a), 0, a.status, 153, &gave_up) && ok;
         tc_fence_after();
         float qn = dot * rq;
         {
-            uint32_t x[64], ph[32], pl[32];
-            tc_ld_32x32(tmem + lanes + COL_A + hh * 64, x);
-            tc_ld_32x32(tmem + lanes + COL_A + hh * 64 + 32, x + 32);
+            uint32_t x[32], ph[16], pl[16];
+            tc_ld_32x32(tmem + lanes + COL_A + hh * 32, x);
             tc_ld_wait();
 #pragma unroll
-            for (int i = 0; i < 64; i += 2) {
+            for (int i = 0; i < 32; i += 2) {
                 float w[2];
 #pragma unroll
                 for (int v = 0; v < 2; ++v) {
-                    const int j = hh * 64 + i + v;
+                    const int j = hh * 32 + i + v;
                     const float2 e = aj[j];
-                    w[v] = (mine && j <= row) ? __uint_as_float(x[i + v]) * qscale * expf((e.x - M.x) + (e.y - M.y)) : 0.0f;
+                    w[v] = (mine && j <= row) ? __uint_as_float(x[i + v]) * qscale * __expf((e.x - M.x) + (e.y - M.y)) : 0.0f;
                     qn += w[v];
                 }
                 const uint32_t hi = pack_bf16(w[0], w[1]);
                 ph[i >> 1] = hi;
                 pl[i >> 1] = pack_bf16(w[0] - __uint_as_float(hi << 16), w[1] - __uint_as_float(hi & 0xffff0000u));
             }
-            tc_st_32x32(tmem + lanes + COL_PH + hh * 32, ph);
-            tc_st_32x32(tmem + lanes + COL_PL + hh * 32, pl);
+            tc_st_32x16(tmem + lanes + COL_PH + hh * 16, ph);
+            tc_st_32x16(tmem + lanes + COL_PL + hh * 16, pl);
         }
 #pragma unroll 1
-        for (int c = hh * 32; c < nb; c += 64) {
+        for (int c = hh * 32; c < nb; c += 128) {
             uint32_t x[32];
             tc_ld_32x32(tmem + lanes + COL_O + c, x);
             tc_ld_wait();
@@ -685,7 +705,7 @@ __global__ void __launch_bounds__(256) mlstm_out_tc_kernel(MlArgs a) {
                     tc_mma_bf16_ts(tmem + COL_O, tmem + (lo ? COL_PL : COL_PH) + 8 * k, umma_desc_mn_sw128(smem_u32(vs) + k * 2048, BOX), id_o, 1u);
             tc_commit(smem_u32(&bar_o));
         }
-        qn = qn_s[0][row] + qn_s[1][row];
+        qn = (qn_s[0][row] + qn_s[1][row]) + (qn_s[2][row] + qn_s[3][row]);
         const bool whole = gridDim.z == 1;
         const float inv_den = 1.0f / (fmaxf(fabsf(qn), em) + 1e-6f);
         ok = mbar_wait_flag(smem_u32(&bar_o), 0, a.status, 154, &gave_up) && ok;
@@ -694,7 +714,7 @@ __global__ void __launch_bounds__(256) mlstm_out_tc_kernel(MlArgs a) {
         if (whole) {
             float ss = 0.0f;
 #pragma unroll 1
-            for (int c = hh * 32; c < nb; c += 64) {
+            for (int c = hh * 32; c < nb; c += 128) {
                 uint32_t x[32];
                 tc_ld_32x32(tmem + lanes + COL_O + c, x);
                 tc_ld_wait();
@@ -706,14 +726,14 @@ __global__ void __launch_bounds__(256) mlstm_out_tc_kernel(MlArgs a) {
             }
             ss_s[hh][row] = ss;
             __syncthreads();
-            f = inv_den / sqrtf((ss_s[0][row] + ss_s[1][row]) / (float)a.vd + a.eps);
+            f = inv_den / sqrtf(((ss_s[0][row] + ss_s[1][row]) + (ss_s[2][row] + ss_s[3][row])) / (float)a.vd + a.eps);
         }
         float* raw = a.raw + ((size_t)(t0 + row) * a.H + h) * a.vc;
         if (!whole && ok && mine && c0 == 0 && hh == 0) raw[a.vd] = qn;
         // the rows pass through shared memory (all products have read theirs), so that gates and outputs move as whole lines
         float* rows = (float*)sm;
 #pragma unroll 1
-        for (int c = hh * 32; c < nb; c += 64) {
+        for (int c = hh * 32; c < nb; c += 128) {
             uint32_t x[32];
             tc_ld_32x32(tmem + lanes + COL_O + c, x);
             tc_ld_wait();
@@ -728,8 +748,8 @@ __global__ void __launch_bounds__(256) mlstm_out_tc_kernel(MlArgs a) {
             float wv[8];
             load8((const float*)a.nw + (size_t)h * a.vd + c0 + col, true, wv);
 #pragma unroll 4
-            for (int u = 0; u < TK / 8; ++u) {
-                const int j = warp + 8 * u;
+            for (int u = 0; u < TK / 16; ++u) {
+                const int j = warp + 16 * u;
                 if (j >= n) break;
                 const size_t to = (size_t)(t0 + j) * a.H + h;
                 float y[8];
@@ -742,7 +762,7 @@ __global__ void __launch_bounds__(256) mlstm_out_tc_kernel(MlArgs a) {
                 float gv[8];
                 load8(a.proj + (size_t)(t0 + j) * a.ld + 2 * a.H * d + (size_t)(a.H + h) * a.vd + col, true, gv);
 #pragma unroll
-                for (int v = 0; v < 8; ++v) y[v] = y[v] * wv[v] / (1.0f + expf(-gv[v]));
+                for (int v = 0; v < 8; ++v) y[v] = __fdividef(y[v] * wv[v], 1.0f + __expf(-gv[v]));
                 *(uint4*)((__nv_bfloat16*)a.out + to * a.vd + col) = pack8(y);
             }
         }
@@ -964,7 +984,7 @@ SP_API int sp_mlstm(const float* proj, int ld, const void* ib, const void* fb, c
     a.cs = p; p += up4((long long)n_chunks * H * d * a.vc);
     a.raw = p;
     static SpPerDevice ready;
-    const int smem = (2 * 64 * MP + 64 * 64) * (int)sizeof(float), sum_smem = 8 * BOX + 1024, out_smem = 2 * OT_STAGE + 1024;
+    const int smem = (2 * 64 * MP + 64 * 64) * (int)sizeof(float), sum_smem = TK * OT_LD * 4 + 1024, out_smem = 2 * OT_STAGE + 1024;
     if (!ready.done()) {
         if (cudaFuncSetAttribute(mlstm_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess ||
             cudaFuncSetAttribute(mlstm_sum_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, sum_smem) != cudaSuccess ||
@@ -978,7 +998,7 @@ SP_API int sp_mlstm(const float* proj, int ld, const void* ib, const void* fb, c
         SP_CHECK_CALL("mlstm_gates", sp_launch_dependent(mlstm_gates_kernel<TK>, dim3(B, H), dim3(MG_WARPS * 32), 0, stream, a));
         SP_CHECK_CALL("mlstm_sum_tc", sp_launch_dependent(mlstm_sum_tc_kernel, dim3(n_chunks, H, cb * eb), dim3(256), (size_t)sum_smem, stream, a));
         SP_CHECK_CALL("mlstm_scan", sp_launch_dependent(mlstm_scan_kernel<true>, scan_grid, dim3(256), 0, stream, a, TK));
-        SP_CHECK_CALL("mlstm_out_tc", sp_launch_dependent(mlstm_out_tc_kernel, dim3(n_chunks, H, cb), dim3(256), (size_t)out_smem, stream, a));
+        SP_CHECK_CALL("mlstm_out_tc", sp_launch_dependent(mlstm_out_tc_kernel, dim3(n_chunks, H, cb), dim3(OT_THREADS), (size_t)out_smem, stream, a));
         if (cb > 1) {
             mlstm_finish_kernel<<<dim3(T, H), 128, 0, stream>>>(a);
             SP_CHECK_LAUNCH("mlstm_finish");
