@@ -1599,7 +1599,8 @@ def mlstm(proj, w: dict, state, nm, out, step, H, d, vd, cap, eps):
         # a prompt of some length on the tensor cores (gates, the chunks' sums, their start states, outputs with their norms
         # and gates), short portions and the 32-bit mode in FFMA products (the norms and gates in a kernel of their own)
         tc = step.max_new >= CHUNKED_FROM and bool(lib.sp_mlstm_tc_supported(
-            c_void_p(_ptr(proj)), proj.shape[1], c_void_p(_ptr(w["norm"])), w_dt, c_void_p(_ptr(out)), dt_code(out), int(d), int(vd)))
+            c_void_p(_ptr(proj)), proj.shape[1], c_void_p(_ptr(w["norm"])), w_dt, c_void_p(_ptr(state)), c_void_p(_ptr(out)),
+            dt_code(out), int(d), int(vd)))
         mode = 2 if tc else 0
         launches += 3 if tc and vd <= 256 else 4
         n_chunks = query_tiles(step.host["new_counts"], int(lib.sp_mlstm_chunk_tokens(int(tc))))

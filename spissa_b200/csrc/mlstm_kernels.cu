@@ -221,12 +221,10 @@ __global__ void __launch_bounds__(256) mlstm_sum_kernel(MlArgs a) {
 }
 
 // the chunks' start states one after the other, element by element (the sums turn into start states in place); grid
-// (sequences, H, blocks of 256 elements of [d][vc]). ``ct``: tokens of a chunk. PACK: the start states
-// of the value columns leave as sums of two bfloat16 numbers, the high one in the lower half of a word, the low one above it.
-template <bool PACK>
+// (sequences, H, blocks of 256 elements of [d][vc]). ``ct``: tokens of a chunk.
 __global__ void __launch_bounds__(256) mlstm_scan_kernel(MlArgs a, int ct) {
+    sp_allow_dependents();
     sp_wait_for_predecessor();
-    sp_allow_dependents();               // whoever starts from here on may read the projections and the gates at once
     const int s = blockIdx.x, h = blockIdx.y;
     const int x = blockIdx.z * 256 + threadIdx.x;
     if (x >= a.d * a.vc) return;
@@ -251,17 +249,59 @@ __global__ void __launch_bounds__(256) mlstm_scan_kernel(MlArgs a, int ct) {
 #pragma unroll
         for (int u = 0; u < 8; ++u)
             if (k0 + u < nc) {
-                if (PACK && col < a.vd) {
-                    const __nv_bfloat16 hi = __float2bfloat16_rn(S);
-                    const __nv_bfloat162 both = __halves2bfloat162(hi, __float2bfloat16_rn(S - __bfloat162float(hi)));
-                    cs[(size_t)(k0 + u) * step] = __uint_as_float(*(const uint32_t*)&both);
-                } else {
-                    cs[(size_t)(k0 + u) * step] = S;
-                }
+                cs[(size_t)(k0 + u) * step] = S;
                 S = fmaf(dv[u], S, own[u]);
             }
     }
     *st = S;
+}
+
+// The same for the tensor-core form, four columns at a time (vd a multiple of four: the group that begins at column vd is n);
+// the start states of the value columns leave as sums of two bfloat16 numbers, the high one in the lower half of a word, the
+// low one above it. grid (sequences, H, blocks of 128 groups of [d][vc / 4])
+__device__ __forceinline__ float pack_high_low(float v) {
+    const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+    const __nv_bfloat162 both = __halves2bfloat162(hi, __float2bfloat16_rn(v - __bfloat162float(hi)));
+    return __uint_as_float(*(const uint32_t*)&both);
+}
+__global__ void __launch_bounds__(128) mlstm_scan_packed_kernel(MlArgs a, int ct) {
+    sp_wait_for_predecessor();
+    sp_allow_dependents();               // whoever starts from here on may read the projections and the gates at once
+    const int s = blockIdx.x, h = blockIdx.y, groups = a.vc / 4;
+    const int x = blockIdx.z * 128 + threadIdx.x;
+    if (x >= a.d * groups) return;
+    const int slot = a.seq_slot[s];
+    if (slot < 0 || slot >= a.n_slots) return;
+    int first = 0;
+    for (int b = 0; b < s; ++b) first += (a.seq_start[b + 1] - a.seq_start[b] + ct - 1) / ct;
+    const int nc = (a.seq_start[s + 1] - a.seq_start[s] + ct - 1) / ct;
+    const int e = x / groups, col = (x - e * groups) * 4;
+    const bool value = col < a.vd;
+    float* st = value ? a.S + (((size_t)slot * a.H + h) * a.d + e) * a.vd + col : a.nm + ((size_t)slot * a.H + h) * (a.d + 1) + e;
+    float4 S = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (value) S = *(const float4*)st;
+    else S.x = *st;
+    const size_t step = (size_t)a.H * a.d * groups;
+    float4* cs = (float4*)a.cs + (size_t)first * step + (size_t)h * a.d * groups + x;
+    const float* ce = a.ce + (size_t)h * a.n_chunks + first;
+    for (int k0 = 0; k0 < nc; k0 += 8) {
+        float4 own[8];
+        float dv[8];
+#pragma unroll
+        for (int u = 0; u < 8; ++u)
+            if (k0 + u < nc) { own[u] = cs[(size_t)(k0 + u) * step]; dv[u] = ce[k0 + u]; }
+#pragma unroll
+        for (int u = 0; u < 8; ++u)
+            if (k0 + u < nc) {
+                cs[(size_t)(k0 + u) * step] = value ? make_float4(pack_high_low(S.x), pack_high_low(S.y), pack_high_low(S.z), pack_high_low(S.w)) : S;
+                S.x = fmaf(dv[u], S.x, own[u].x);
+                S.y = fmaf(dv[u], S.y, own[u].y);
+                S.z = fmaf(dv[u], S.z, own[u].z);
+                S.w = fmaf(dv[u], S.w, own[u].w);
+            }
+    }
+    if (value) *(float4*)st = S;
+    else *st = S.x;
 }
 
 // outputs; grid (chunks, H, column blocks of 64)
@@ -933,8 +973,8 @@ long long up4(long long n) { return (n + 3) / 4 * 4; }
 }  // namespace
 
 // Whether a prompt step with these operands can run on the tensor cores (bfloat16 outputs, 16-byte pieces everywhere).
-SP_API int sp_mlstm_tc_supported(const void* proj, int ld, const void* nw, int w_dt, const void* out, int out_dt, int d, int vd) {
-    return out_dt == SP_DT_BF16 && w_dt == SP_DT_F32 && d % 8 == 0 && vd % 8 == 0 && ld % 4 == 0 &&
+SP_API int sp_mlstm_tc_supported(const void* proj, int ld, const void* nw, int w_dt, const float* state, const void* out, int out_dt, int d, int vd) {
+    return out_dt == SP_DT_BF16 && w_dt == SP_DT_F32 && (((uintptr_t)state) & 15) == 0 && d % 8 == 0 && vd % 8 == 0 && ld % 4 == 0 &&
            ((((uintptr_t)proj | (uintptr_t)nw | (uintptr_t)out) & 15) == 0);
 }
 SP_API int sp_mlstm_chunk_tokens(int tensor_cores) { return tensor_cores ? TK : MC; }
@@ -971,7 +1011,7 @@ SP_API int sp_mlstm(const float* proj, int ld, const void* ib, const void* fb, c
         return 0;
     }
     if (!scratch || ((uintptr_t)scratch & 15)) SP_FAIL("mlstm: a prompt step needs scratch that starts on 16 bytes");
-    if (mode == 2 && !sp_mlstm_tc_supported(proj, ld, nw, w_dt, out, out_dt, d, vd)) SP_FAIL("mlstm: the tensor-core form does not take these operands");
+    if (mode == 2 && !sp_mlstm_tc_supported(proj, ld, nw, w_dt, S, out, out_dt, d, vd)) SP_FAIL("mlstm: the tensor-core form does not take these operands");
     const long long HT = up4((long long)H * T);
     a.vc = (int)up4(vd + 1);
     float* p = scratch;
@@ -997,7 +1037,7 @@ SP_API int sp_mlstm(const float* proj, int ld, const void* ib, const void* fb, c
         const int cb = (vd + 255) / 256, eb = (d + TK - 1) / TK;
         SP_CHECK_CALL("mlstm_gates", sp_launch_dependent(mlstm_gates_kernel<TK>, dim3(B, H), dim3(MG_WARPS * 32), 0, stream, a));
         SP_CHECK_CALL("mlstm_sum_tc", sp_launch_dependent(mlstm_sum_tc_kernel, dim3(n_chunks, H, cb * eb), dim3(256), (size_t)sum_smem, stream, a));
-        SP_CHECK_CALL("mlstm_scan", sp_launch_dependent(mlstm_scan_kernel<true>, scan_grid, dim3(256), 0, stream, a, TK));
+        SP_CHECK_CALL("mlstm_scan", sp_launch_dependent(mlstm_scan_packed_kernel, dim3(B, H, (d * (a.vc / 4) + 127) / 128), dim3(128), 0, stream, a, TK));
         SP_CHECK_CALL("mlstm_out_tc", sp_launch_dependent(mlstm_out_tc_kernel, dim3(n_chunks, H, cb), dim3(OT_THREADS), (size_t)out_smem, stream, a));
         if (cb > 1) {
             mlstm_finish_kernel<<<dim3(T, H), 128, 0, stream>>>(a);
@@ -1009,7 +1049,7 @@ SP_API int sp_mlstm(const float* proj, int ld, const void* ib, const void* fb, c
     const int nb = (vd + 64) / 64, eb = (d + 63) / 64;
     mlstm_sum_kernel<<<dim3(n_chunks, H, nb * eb), 256, 0, stream>>>(a);
     SP_CHECK_LAUNCH("mlstm_sum");
-    SP_CHECK_CALL("mlstm_scan", sp_launch_dependent(mlstm_scan_kernel<false>, scan_grid, dim3(256), 0, stream, a, MC));
+    SP_CHECK_CALL("mlstm_scan", sp_launch_dependent(mlstm_scan_kernel, scan_grid, dim3(256), 0, stream, a, MC));
     mlstm_out_kernel<<<dim3(n_chunks, H, nb), 256, smem, stream>>>(a);
     SP_CHECK_LAUNCH("mlstm_out");
     mlstm_finish_kernel<<<dim3(T, H), 128, 0, stream>>>(a);
