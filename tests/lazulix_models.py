@@ -7,7 +7,7 @@ import torch
 from plain.llama_plain import read_model_folder
 
 
-def mem(heads, dim, vdim, cap=12.0):
+def mem(heads, dim, vdim, cap=11.0):
     return dict(heads=heads, dim=dim, vdim=vdim, gate_cap=cap)
 
 
@@ -152,7 +152,7 @@ def key_needle_model(kind="attention", heads=2, kv=1, dim=16, vdim=8, shared=Fal
 def memory_needle_model(heads=2, dim=8, vdim=12, slow=True):
     """A matrix memory into which token ``NEEDLE`` alone writes something large (its input gate opens wide). ``slow``: forget
     gates so open that it is still there hundreds of tokens later; else the memory forgets at once."""
-    cfg = model(32, 64, [layer("mlstm", mem(heads, dim, vdim, 12.0))], scale=1.0)
+    cfg = model(32, 64, [layer("mlstm", mem(heads, dim, vdim, 13.0))], scale=1.0)
 
     def patch(w):
         _mark_embedding(w, 32)

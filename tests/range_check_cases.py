@@ -122,6 +122,33 @@ def main() -> int:
     code, kp = streamed(bad)
     assert code == 401 and bool((kp[bad] == 9.0).all())
     assert any(bool((kp[p] != 9.0).any()) for p in other)
+
+    # key and value rows of two sizes: the decode attention's table, and the kernels that place q, k and v head by head
+    d, vd = 40, 24
+    assert K.range_checked("attention_kv") and K.range_checked("sandwich")
+    kp2 = torch.ones(meta.n_pages, nkv, 64, d, dtype=torch.bfloat16, device=DEV)
+    vp2 = torch.ones(meta.n_pages, nkv, 64, vd, dtype=torch.bfloat16, device=DEV)
+    q2, out2 = torch.randn(B, nh * d, device=DEV).bfloat16(), torch.empty(B, nh * vd, dtype=torch.bfloat16, device=DEV)
+
+    def decode_kv():
+        ct, nc = K.flash_decode_plan(B, nkv, max(lengths))
+        scratch = torch.empty(K.flash_decode_scratch_floats(B, nh, vd, nc), device=DEV)
+        K.flash_decode(q2, kp2, vp2, out2, meta, meta.seq_len, nh, nkv, d, None, scale, ct, nc, scratch, vd=vd)
+    assert code_of(decode_kv) == 0
+    meta.declared_pages = top_page
+    assert code_of(decode_kv) == 401
+    meta.declared_pages = None
+    for d2 in (40, 10):                                            # with 16-byte accesses and without
+        row = torch.randn(T, (nh + nkv) * d2 + nkv * vd, device=DEV)
+        qo2 = torch.empty(T, nh * d2, dtype=torch.bfloat16, device=DEV)
+        for declared, want in ((None, 0), (bad, 401)):
+            kp = torch.full((wmeta.n_pages, nkv, 64, d2), 9.0, dtype=torch.bfloat16, device=DEV)
+            vp = torch.full((wmeta.n_pages, nkv, 64, vd), -9.0, dtype=torch.bfloat16, device=DEV)
+            wmeta.declared_pages = declared
+            assert code_of(lambda: K.qkv_norm_rot_store(row, None, qo2, kp, vp, wmeta, None, nh, nkv, d2, vd, 0)) == want
+            wmeta.declared_pages = None
+            assert any(bool((kp[p] != 9.0).any()) for p in other)
+            assert bool((kp[bad] == 9.0).all()) == bool((vp[bad] == -9.0).all()) == (want == 401)
     print("range check cases ok")
     return 0
 
